@@ -32,12 +32,16 @@ _SIGNATURES = {
     "ce_add_residual": (_i, [_p, _p, _i, _ll, _p]),
     "ce_swiglu": (_i, [_p, _p, _i, _i, _i, _p]),
     "ce_reluglu": (_i, [_p, _p, _i, _i, _i, _p]),
+    # gate_up, out, dtype, bias, limit, alpha, T, I, stream
+    "ce_clamp_glu": (_i, [_p, _p, _i, _p, _f, _f, _i, _i, _p]),
     # in, out, dtype, T, I, ldo, stream
     "ce_relu2": (_i, [_p, _p, _i, _i, _i, _i, _p]),
     # x, w, b, out, out_dtype, rows, R, H, eps, stream
     "ce_layernorm": (_i, [_p, _p, _p, _p, _i, _p, _i, _i, _f, _p]),
     # y, w, x, T, H, eps, stream
     "ce_rmsnorm_add": (_i, [_p, _p, _p, _p, _i, _i, _f, _p]),
+    # y, bias, w, x, w2, h, h_dtype, T, H, eps, eps2, stream
+    "ce_rmsnorm_add_norm": (_i, [_p] * 6 + [_i] * 3 + [_f, _f, _p]),
     # x, n, cap, stream
     "ce_tanh_cap": (_i, [_p, _ll, _f, _p]),
     # src, out, out_dtype, T, ld, off, L, stream
@@ -47,11 +51,11 @@ _SIGNATURES = {
     # rows, dtype, stride, off, n, first, first_stride, first_off, lam, T, stream
     "ce_value_mix": (_i, [_p, _i, _i, _i, _i, _p, _i, _i, _f, _i, _p]),
     # proj, wq, wkv, cq, k_pool, dtype, cos, sin, positions, seq_of_token, seq_slot, block_table, status,
-    # T, ld, off_q, qr, off_kv, r, dr, rd, page_size, max_pages, num_pages, max_pos, write_kv, eps, stream
-    "ce_latent_prepare": (_i, [_p] * 5 + [_i] + [_p] * 7 + [_i] * 13 + [_f, _p]),
+    # T, ld, off_q, qr, off_kv, r, dr, rd, page_size, max_pages, num_pages, max_pos, write_kv, eps, pairing, stream
+    "ce_latent_prepare": (_i, [_p] * 5 + [_i] + [_p] * 7 + [_i] * 13 + [_f, _i, _p]),
     # src, src_stride, src_head, src_off, dst, dst_stride, dst_head, dst_off, dtype, cos, sin, positions, status,
-    # T, H, dr, rd, max_pos, stream
-    "ce_rope_part": (_i, [_p, _i, _i, _i, _p, _i, _i, _i, _i, _p, _p, _p, _p, _i, _i, _i, _i, _i, _p]),
+    # T, H, dr, rd, max_pos, pairing, stream
+    "ce_rope_part": (_i, [_p, _i, _i, _i, _p, _i, _i, _i, _i, _p, _p, _p, _p, _i, _i, _i, _i, _i, _i, _p]),
     # in, in_stride, in_head, W, out, out_stride, out_head, gate, gate_stride, gate_head, dtype, M, H, N, K, stream
     "ce_head_matmul": (_i, [_p, _i, _i, _p, _p, _i, _i, _p, _i, _i, _i, _i, _i, _i, _i, _p]),
     # q, k_pool, v_pool, gate, out, dtype, positions, seq_of_token, seq_slot, block_table, status, T, nh, nkv, d, dv,
@@ -67,17 +71,19 @@ _SIGNATURES = {
     # q_stride, q_head, ldk, ldv, gate_stride, page_size, max_pages, num_pages, window, keep_first, scale, softcap, sinks,
     # out_scale, stream
     "ce_masked_attention_mma": (_i, [_p] * 11 + [_i] * 16 + [_f, _f, _p, _f, _p]),
-    "ce_gated_delta_prep_width": (_i, [_i, _i, _i, _i]),
+    # H, G, d, dv, decay_mode
+    "ce_gated_delta_prep_width": (_i, [_i] * 5),
     # proj, dec, gz, taps, a_log, dt_bias, norm_w, prep, raw, state, kept, out, out_dtype, seq_of_token, seq_slot, q_start,
     # T, B, ld, off_conv, off_b, H, G, d, dv, K, eps, ld_dec, ld_gz, decay_mode, operands, rule, gate_act, out_scale,
-    # cos, sin, positions, status, rd, max_pos, stage, stream
-    "ce_gated_delta": (_i, [_p] * 12 + [_i] + [_p] * 3 + [_i] * 10 + [_f] + [_i] * 6 + [_f] + [_p] * 4 + [_i, _i, _i, _p]),
+    # cos, sin, positions, status, rd, max_pos, conv_bias, skip, m_state, cap, write_mode, ones, norm_all, parts, stage, stream
+    "ce_gated_delta": (_i, [_p] * 12 + [_i] + [_p] * 3 + [_i] * 10 + [_f] + [_i] * 6 + [_f] + [_p] * 4 + [_i, _i] + [_p] * 3 + [_f]
+                       + [_i] * 5 + [_p]),
     # q, k_pool, v_pool, out, dtype, positions, seq_of_token, seq_slot, block_table, status,
     # T, nh, nkv, d, q_stride, page_size, max_pages, num_pages, window, scale, stream
     "ce_attention_generic": (_i, [_p, _p, _p, _p, _i, _p, _p, _p, _p, _p,
                                   _i, _i, _i, _i, _i, _i, _i, _i, _i, _f, _p]),
-    # A, W, C, dtype, M, N, K, lda, ldc, mode, stream
-    "ce_gemm_plain": (_i, [_p, _p, _p, _i, _i, _i, _i, _i, _i, _i, _p]),
+    # A, W, C, dtype, M, N, K, lda, ldc, mode, bias, limit, alpha, stream
+    "ce_gemm_plain": (_i, [_p, _p, _p, _i, _i, _i, _i, _i, _i, _i, _p, _f, _f, _p]),
     "ce_sample": (_i, [_p, _i, _i, _p, _p, _p]),
     "ce_argmax": (_i, [_p, _i, _i, _p, _p]),
     "ce_apply_penalties": (_i, [_p, _i, _p, _i, _p, _p]),
@@ -104,13 +110,13 @@ _SIGNATURES = {
     # q, k_pool, v_pool, gate, out, positions, seq_slot, q_start, block_table, tiles, status, n_tiles, nh, nkv, d, dv,
     # q_stride, gate_stride, page_size, max_pages, num_pages, window, chunk, scale, lambda, eps, out_scale, stream
     "ce_diff_attention_mma": (_i, [_p] * 11 + [_i] * 12 + [_f] * 4 + [_p]),
-    # z, ids, weights, sgate, T, ld, E, top, groups, keep, scale, stream
-    "ce_moe_route": (_i, [_p] * 4 + [_i] * 6 + [_f, _p]),
+    # z, ids, weights, sgate, T, ld, E, top, groups, keep, scale, correction, scoring, group_score, renormalize, stream
+    "ce_moe_route": (_i, [_p] * 4 + [_i] * 6 + [_f, _p, _i, _i, _i, _p]),
     "ce_moe_max_tiles": (_i, [_i, _i, _i]),
     # ids, n_pairs, top, E, BM, max_rows, row_token, pair_row, tile_expert, n_tiles, stream
     "ce_moe_align": (_i, [_p] + [_i] * 5 + [_p] * 5),
-    # in, W, out, row_token, tile_expert, n_tiles, dtype, max_tiles, BM, N, K, ldi, ldo, act, n_rows, stream
-    "ce_moe_matmul": (_i, [_p] * 6 + [_i] * 9 + [_p]),
+    # in, W, out, row_token, tile_expert, n_tiles, dtype, max_tiles, BM, N, K, ldi, ldo, act, limit, alpha, n_rows, stream
+    "ce_moe_matmul": (_i, [_p] * 6 + [_i] * 8 + [_f, _f, _i, _p]),
     # in, ldi, K, elsize, row_token, n_tiles, BM, out, max_rows, stream
     "ce_moe_gather": (_i, [_p, _i, _i, _i, _p, _p, _i, _p, _i, _p]),
     # rows, dtype, ld, pair_row, weights, shared, sgate, y, T, top, W, accumulate, stream

@@ -73,6 +73,19 @@ __device__ __forceinline__ float ce_exp2_fast(float x) {
     return y;
 }
 
+// The clamped gated activation: g = min(gate, limit), u = up cut to [-limit, limit]; g sigmoid(alpha g) (u + 1).
+__device__ __forceinline__ float ce_clamp_glu(float g, float u, float limit, float alpha) {
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    return g / (1.0f + expf(-alpha * g)) * (u + 1.0f);
+}
+// the same with the approximate exponential and reciprocal, for results that are rounded to bfloat16 right after
+__device__ __forceinline__ float ce_clamp_glu_fast(float g, float u, float limit, float alpha) {
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    return __fdividef(g, 1.0f + __expf(-alpha * g)) * (u + 1.0f);
+}
+
 template <typename T> struct CeType;
 template <> struct CeType<float> {
     static __device__ __forceinline__ float load(const float* p) { return *p; }

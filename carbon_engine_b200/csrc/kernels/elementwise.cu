@@ -512,6 +512,33 @@ extern "C" int ce_swiglu(const void* gu, void* out, int dtype, int T, int I, cud
     return gated_act(gu, out, dtype, T, I, 0, stream);
 }
 
+// out[t, i] = the clamped gated activation of gu[t, i] + bias[i] and gu[t, I + i] + bias[I + i] (bias float32 [2I] or null)
+template <typename T>
+__global__ void clamp_glu_kernel(const T* __restrict__ gu, T* __restrict__ out, const float* __restrict__ bias, float limit, float alpha,
+                                 int I, size_t total) {
+    ce_pdl_begin();
+    size_t stride = (size_t)gridDim.x * blockDim.x;
+    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += stride) {
+        size_t t = i / I, c = i - t * I;
+        float g = CeType<T>::load(gu + t * 2 * I + c) + (bias ? bias[c] : 0.f);
+        float u = CeType<T>::load(gu + t * 2 * I + I + c) + (bias ? bias[I + c] : 0.f);
+        CeType<T>::store(out + i, ce_clamp_glu(g, u, limit, alpha));
+    }
+}
+
+extern "C" int ce_clamp_glu(const void* gu, void* out, int dtype, const float* bias, float limit, float alpha, int T, int I,
+                            cudaStream_t stream) {
+    size_t total = (size_t)T * I;
+    if (total == 0) return CE_OK;
+    if (!gu || !out) return ce_fail(CE_ERR_ARG, "ce_clamp_glu: null pointer");
+    int blocks = (int)((total + 255) / 256 < 148 * 16 ? (total + 255) / 256 : 148 * 16);
+    ce_note("clamp_glu_kernel");
+    if (dtype == CE_F32) ce_launch(clamp_glu_kernel<float>, blocks, 256, 0, stream, (const float*)gu, (float*)out, bias, limit, alpha, I, total);
+    else if (dtype == CE_BF16) ce_launch(clamp_glu_kernel<__nv_bfloat16>, blocks, 256, 0, stream, (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, bias, limit, alpha, I, total);
+    else return ce_fail(CE_ERR_ARG, "ce_clamp_glu: unknown dtype %d", dtype);
+    return ce_check_launch("ce_clamp_glu");
+}
+
 // out[t, i] = relu(in[t, i])^2: the epilogue of a library product for the activation of the small experts
 template <typename T>
 __global__ void relu2_kernel(const T* __restrict__ in, T* __restrict__ out, int I, int ldo, size_t total) {

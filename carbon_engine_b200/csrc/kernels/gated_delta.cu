@@ -3,27 +3,40 @@
 //
 //     S <- diag(g_t) S;    u_t = beta_t (v_t - S^T k_t);    S <- S + k_t u_t^T;    o_t = S^T q_t
 //
-// (the read-out sees the token's own write), and the plain decaying sum of outer products, "retention" (rule 1): the same
-// with u_t = v_t.  The options are arguments, so that the family's mixers share the four kernels:
+// (the read-out sees the token's own write), and the plain decaying sum of outer products (rule 1: retention, state-space
+// duality, matrix memories): the same with u_t = beta_t v_t.  The options are arguments, so that the family's mixers share
+// the kernels:
 //   decay     0: one per head and key channel from logits [T, H d];  1: one per head from logits [T, H];
-//             2: a constant per head (``a_log`` then holds the constants themselves, nothing is learned per token)
+//             2: a constant per head (``a_log`` then holds the constants themselves, nothing is learned per token);
+//             3: exponential gates: log input gate i = cap tanh((z_i + b_i) / cap), log forget gate
+//                f = logsigmoid(cap tanh((z_f + b_f) / cap)), a running maximum m_t = max(f + m_(t-1), i) per head (m starts
+//                at 0), decay exp(f + m_(t-1) - m_t), beta exp(i - m_t)
 //   operands  0: short convolution, SiLU, unit q and k (below);  1: no convolution: q and k are rotated over their first
-//             ``rd`` elements by the token's position (element i with i + rd/2), k times d^-1/2, v as projected
-//   gate      0: sigmoid, 1: SiLU of the gate logits;  the weight after the root mean square may be absent;  the stored
-//             result is multiplied by ``out_scale`` (the mixer's weight in a sum of mixers)
+//             ``rd`` elements by the token's position (element i with i + rd/2), k times d^-1/2, v as projected;
+//             2: short convolution and SiLU only;  3: q times d^-1/2, k and v as projected
+//   write     0: beta = sigmoid of a projection;  1: beta is the step size itself, softplus(z + bias) of the decay's logits
+//             (rotated operands write with beta 1, exponential gates with their own beta)
+//   ones      1: one more value channel whose value is always 1 (the decayed sum of the written keys, a normalizer): the head's
+//             output is divided by max(|its read-out|, exp(-m_t)) + 1e-6
+//   gate      0: sigmoid, 1: SiLU of the gate logits;  the weight after the root mean square may be absent, of size dv or of
+//             all heads' size;  the stored result is multiplied by ``out_scale`` (the mixer's weight in a sum of mixers)
+//   parts     0: the order after the read-out is root mean square per head, weight, gate;  n > 0: skip D_h v_t is added, the
+//             gate comes first, and the root mean square is taken in n equal parts of all heads' values together
 // With the convolution:  q, k and v come out of a short causal convolution over time per channel
 // followed by SiLU; q and k are then brought to unit length per head (q also times d^-1/2); the decay is
 // g_t = exp(-exp(A_h) softplus(z_t + bias)) with z_t the token's decay logits (a product of their own);
 // beta_t = sigmoid of a projection, one per head.  Query/key head of value head h: h / (H / G).  Afterwards every
 // head's o_t is divided by its root mean square, multiplied by a weight of size dv and by sigmoid(gate logits).
 //
-// Four kernels, all float32:
+// The kernels, all float32:
 //   prepare     every token on its own: convolution (the inputs before a portion's first token come from the
 //               request's kept rows), SiLU, unit q and k, decay, beta                       (parallel over tokens)
 //   keep        the last taps-1 convolution inputs of every sequence go to its kept rows   (parallel over channels)
 //   walk        one block per (head, sequence, slice of value channels) walks the sequence's tokens of this step
 //               in order, from the state its slot holds, and stores the state back           (the recurrence)
 //   finish      every (token, head): root mean square, weight, gate, one rounding at the store   (parallel)
+// and, with exponential gates, between prepare and walk, scan: the running maximum of every (sequence, head) in token order.
+// A step in which every sequence brings one token has no keep and no scan: prepare does their work.
 //
 // The columns of S (value channels) are independent of one another, so a slice of GD_COLS columns is a block of
 // its own and a column lives in the registers of 16 neighbouring lanes (32 for more than 128 key channels, so that a
@@ -41,15 +54,15 @@ __device__ __forceinline__ float gd_softplus(float z) { return z > 20.f ? z : lo
 
 struct GatedDeltaArgs {
     const float* proj;           // [T, ld]: the convolution's inputs q | k | v from off_conv (C = 2 G d + H dv columns), beta logits at off_b
-    const float* dec;            // decay logits before the bias, rows of ld_dec: [T, H*d] (decay 0) or [T, H] (decay 1); unused with decay 2
+    const float* dec;            // decay logits before the bias, rows of ld_dec: [T, H*d] (decay 0), [T, H] (decay 1), [T, 2 H] (decay 3: input gates, then forget gates); unused with decay 2
     const float* gz;             // [T, H*dv] gate logits, rows of ld_gz
-    const float* taps;           // [C, K] convolution weights, the last column the current token's (operands 0)
-    const float* a_log;          // [H]; with decay 2 the heads' constant decays themselves
-    const float* dt_bias;        // [H*d] (decay 0) or [H] (decay 1)
-    const float* norm_w;         // [dv] or null
-    float* prep;                 // [T, P]: q (G d) | k (G d) | v (H dv) | decay (H d) | beta (H); P padded to a multiple of 4
-    float* raw;                  // [T, H*dv] o_t before the norm
-    float* state;                // [slots, H, d, dv]
+    const float* taps;           // [C, K] convolution weights, the last column the current token's (operands 0 and 2)
+    const float* a_log;          // [H]; with decay 2 the heads' constant decays themselves; unused with decay 3
+    const float* dt_bias;        // [H*d] (decay 0), [H] (decay 1) or [2 H] (decay 3: input gates, then forget gates)
+    const float* norm_w;         // [dv], [H*dv] (norm_all) or null
+    float* prep;                 // [T, P]: q (G d) | k (G d) | v (H dv) | decay (H d, or H with one per head) | beta (H) | running maximum (H, decay 3); P padded to a multiple of 4
+    float* raw;                  // [T, H*(dv + ones)] o_t before the norm; the heads' extra channels follow all heads' values
+    float* state;                // [slots, H, d*(dv + ones)]: d rows of dv, then the extra channel's d numbers
     float* kept;                 // [slots, K-1, C] the convolution inputs of the last K-1 tokens, oldest first
     void* out;                   // [T, H*dv]
     const int* seq_of_token;
@@ -65,7 +78,15 @@ struct GatedDeltaArgs {
     const int* positions;        // [T]
     int* status;
     int rd, max_pos;
+    const float* conv_bias;      // [C] or null: added to the convolution before SiLU
+    const float* skip;           // [H] (parts > 0): y_t = o_t + skip_h v_t
+    float* m_state;              // [slots, H] the running maximum (decay 3)
+    float cap;                   // of the exponential gates' logits
+    int write_mode, ones, norm_all, parts, single;       // single: every sequence of the step brings exactly one token
 };
+
+// One decay per head: the walk stages one number a token instead of a vector.
+__device__ __host__ __forceinline__ bool gd_head_decay(int decay_mode) { return decay_mode != 0; }
 
 // A token's heads of q, of k (unit vectors) and of v are dealt to the warps of gridDim.y blocks in turn (one block a token
 // in a long step; in a step of few tokens a block per handful of heads, so that the step is not eight blocks' work); the
@@ -79,6 +100,7 @@ __global__ void gated_delta_prepare_kernel(GatedDeltaArgs a) {
     int b = a.seq_of_token[t];
     int rel = t - a.q_start[b];                     // tokens of the same sequence before this one in the step
     const float* kept = a.kept + (size_t)a.seq_slot[b] * (K - 1) * C;
+    float* kept_rw = a.kept + (size_t)a.seq_slot[b] * (K - 1) * C;
     float* pw = a.prep + (size_t)t * a.P;
     float q_scale = rsqrtf((float)d);
     int nthr = blockDim.x * gridDim.y, thr = blockIdx.y * blockDim.x + threadIdx.x;
@@ -104,18 +126,37 @@ __global__ void gated_delta_prepare_kernel(GatedDeltaArgs a) {
         }
         for (int e = thr; e < H * dv; e += nthr) pw[nqk + e] = row[nqk + e];
         float* decay1 = pw + C;
-        for (int e = thr; e < H * d; e += nthr) decay1[e] = a.a_log[e / d];
-        for (int h = thr; h < H; h += nthr) decay1[H * d + h] = 1.0f;
+        for (int h = thr; h < H; h += nthr) { decay1[h] = a.a_log[h]; decay1[H + h] = 1.0f; }
+        return;
+    }
+    if (a.operands == 3) {
+        const float* row = a.proj + (size_t)t * a.ld + a.off_conv;
+        for (int e = thr; e < C; e += nthr) pw[e] = e < G * d ? row[e] * q_scale : row[e];
+        float* gates = pw + C;                      // f (then the decay) | i (then beta) | running maximum
+        const float* z = a.dec + (size_t)t * a.ld_dec;
+        for (int h = thr; h < H; h += nthr) {
+            float i = __fmul_rn(a.cap, tanhf((z[h] + a.dt_bias[h]) / a.cap));
+            float f = -gd_softplus(-__fmul_rn(a.cap, tanhf((z[H + h] + a.dt_bias[H + h]) / a.cap)));
+            if (!a.single) { gates[h] = f; gates[H + h] = i; continue; }
+            float* ms = a.m_state + (size_t)a.seq_slot[b] * H + h;
+            float fm = __fadd_rn(f, *ms), m = fmaxf(fm, i);
+            gates[h] = expf(__fsub_rn(fm, m));
+            gates[H + h] = expf(__fsub_rn(i, m));
+            gates[2 * H + h] = m;
+            *ms = m;
+        }
         return;
     }
     // convolution + SiLU of channel c at this token
     auto conv = [&](int c) -> float {
-        float y = 0.f;
+        float y = a.conv_bias ? a.conv_bias[c] : 0.f;
         for (int j = 0; j < K; ++j) {
             int back = K - 1 - j;                   // how many tokens before this one
             float x = back <= rel ? a.proj[(size_t)(t - back) * a.ld + a.off_conv + c]
                                   : kept[(size_t)(K - 1 + rel - back) * C + c];
             y = fmaf(a.taps[(size_t)c * K + j], x, y);
+            // a single token: the kept rows move up by one behind the read (row j has just been read; no other thread touches the channel)
+            if (a.single && j > 0) kept_rw[(size_t)(j - 1) * C + c] = x;
         }
         return y / (1.0f + expf(-y));
     };
@@ -124,7 +165,7 @@ __global__ void gated_delta_prepare_kernel(GatedDeltaArgs a) {
         bool is_v = hh >= 2 * G;
         int size = is_v ? dv : d;
         int c0 = is_v ? 2 * G * d + (hh - 2 * G) * dv : hh * d;
-        if (is_v) {
+        if (is_v || a.operands == 2) {
             for (int c = lane; c < size; c += 32) pw[c0 + c] = conv(c0 + c);
             continue;
         }
@@ -143,15 +184,65 @@ __global__ void gated_delta_prepare_kernel(GatedDeltaArgs a) {
     if (a.decay_mode == 0) {
         for (int e = thr; e < H * d; e += nthr)
             decay[e] = expf(-expf(a.a_log[e / d]) * gd_softplus(a.dec[(size_t)t * a.ld_dec + e] + a.dt_bias[e]));
-    } else if (a.decay_mode == 1) {          // one decay per head, written to all its key channels
-        for (int e = thr; e < H * d; e += nthr) {
-            int h = e / d;
-            decay[e] = expf(-expf(a.a_log[h]) * gd_softplus(a.dec[(size_t)t * a.ld_dec + h] + a.dt_bias[h]));
-        }
-    } else {
-        for (int e = thr; e < H * d; e += nthr) decay[e] = a.a_log[e / d];
+        for (int h = thr; h < H; h += nthr) decay[H * d + h] = gd_sigmoid(a.proj[(size_t)t * a.ld + a.off_b + h]);
+        return;
     }
-    for (int h = thr; h < H; h += nthr) decay[H * d + h] = gd_sigmoid(a.proj[(size_t)t * a.ld + a.off_b + h]);
+    for (int h = thr; h < H; h += nthr) {
+        float step = a.decay_mode == 1 ? gd_softplus(a.dec[(size_t)t * a.ld_dec + h] + a.dt_bias[h]) : 0.f;
+        decay[h] = a.decay_mode == 1 ? expf(-expf(a.a_log[h]) * step) : a.a_log[h];
+        decay[H + h] = a.write_mode == 1 ? step : gd_sigmoid(a.proj[(size_t)t * a.ld + a.off_b + h]);
+    }
+}
+
+// The running maximum of the exponential gates, token after token: a block per (sequence, 32 heads).  The chain is one addition
+// and one maximum a token; one warp walks it, a head a lane, over a chunk of tokens in shared memory, and all warps fetch the
+// chunk's gates before and take the exponentials after.
+#define GD_SCAN_TOKENS 64
+__global__ void __launch_bounds__(256) gated_delta_scan_kernel(GatedDeltaArgs a) {
+    ce_pdl_begin();
+    __shared__ float fs[GD_SCAN_TOKENS][32], is[GD_SCAN_TOKENS][32], ms[GD_SCAN_TOKENS + 1][32];
+    int b = blockIdx.x, h0 = blockIdx.y * 32, tid = threadIdx.x, H = a.H;
+    int t_begin = a.q_start[b], n = a.q_start[b + 1] - t_begin;
+    if (n <= 0) return;
+    size_t off = (size_t)2 * a.G * a.d + (size_t)H * a.dv;
+    float* m_state = a.m_state + (size_t)a.seq_slot[b] * H;
+    if (tid < 32) ms[0][tid] = h0 + tid < H ? m_state[h0 + tid] : 0.f;
+    for (int c0 = 0; c0 < n; c0 += GD_SCAN_TOKENS) {
+        int nt = min(GD_SCAN_TOKENS, n - c0);
+        for (int e = tid; e < nt * 32; e += 256) {
+            int tok = e >> 5, h = e & 31;
+            const float* g = a.prep + (size_t)(t_begin + c0 + tok) * a.P + off + h0 + h;
+            bool in = h0 + h < H;
+            fs[tok][h] = in ? g[0] : 0.f;
+            is[tok][h] = in ? g[H] : 0.f;
+        }
+        __syncthreads();
+        if (tid < 32) {
+            float m = ms[0][tid];
+#pragma unroll 8
+            for (int tok = 0; tok < nt; ++tok) {
+                m = fmaxf(__fadd_rn(fs[tok][tid], m), is[tok][tid]);
+                ms[tok + 1][tid] = m;
+            }
+        }
+        __syncthreads();
+        for (int e = tid; e < nt * 32; e += 256) {
+            int tok = e >> 5, h = e & 31;
+            if (h0 + h >= H) continue;
+            float* g = a.prep + (size_t)(t_begin + c0 + tok) * a.P + off + h0 + h;
+            float m = ms[tok + 1][h], fm = __fadd_rn(fs[tok][h], ms[tok][h]);
+            g[0] = expf(__fsub_rn(fm, m));
+            g[H] = expf(__fsub_rn(is[tok][h], m));
+            g[2 * H] = m;
+        }
+        __syncthreads();
+        if (tid < 32) {
+            float m = ms[nt][tid];
+            ms[0][tid] = m;
+            if (c0 + nt >= n && h0 + tid < H) m_state[h0 + tid] = m;
+        }
+        __syncthreads();
+    }
 }
 
 // One thread per (sequence, channel): the kept rows move up by the portion's length and take the portion's last inputs.
@@ -179,36 +270,42 @@ __device__ __forceinline__ void gd_cp16(float* dst, const float* src) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(s), "l"(src));
 }
 
-// Copies of one tile of tokens into a buffer: three vectors of d per token (decay, key, query; rows padded to DP floats),
-// BC values (the block's value channels) and beta.
-template <int DP, bool VEC, int BC>
+// Copies of one tile of tokens into a buffer: key, query and, with a decay per key channel (HD false), decay, vectors of d per
+// token (rows padded to DP floats); then per token BC values (the block's value channels), beta and the head's decay.
+template <int DP, bool VEC, int BC, bool HD>
 __device__ __forceinline__ void gd_stage(const GatedDeltaArgs& a, float* buf, int t0, int n_tok, int h, int col0, int ncols) {
+    constexpr int NV = HD ? 2 : 3, VS = BC + 2;
     int d = a.d, G = a.G, H = a.H, tid = threadIdx.x, nthr = blockDim.x;
     int g = h / (H / G);
     int C = 2 * G * d + H * a.dv;
-    int offs[3] = {C + h * d, G * d + g * d, g * d};          // decay, key, query within a prep row
-    float* vbuf = buf + 3 * GD_TILE * DP;
+    int offs[3] = {G * d + g * d, g * d, C + h * d};          // key, query, decay within a prep row
+    int off_beta = C + (HD ? H : H * d) + h;
+    float* vbuf = buf + NV * GD_TILE * DP;
     if (VEC) {
         constexpr int DP4 = DP / 4;
-        for (int e = tid; e < 3 * GD_TILE * DP4; e += nthr) {
+        for (int e = tid; e < NV * GD_TILE * DP4; e += nthr) {
             int which = e / (GD_TILE * DP4), tok = (e / DP4) % GD_TILE, c = (e % DP4) * 4;
             if (tok < n_tok && c < d) gd_cp16(buf + (which * GD_TILE + tok) * DP + c, a.prep + (size_t)(t0 + tok) * a.P + offs[which] + c);
         }
     } else {
-        for (int e = tid; e < 3 * GD_TILE * DP; e += nthr) {
+        for (int e = tid; e < NV * GD_TILE * DP; e += nthr) {
             int which = e / (GD_TILE * DP), tok = (e / DP) % GD_TILE, c = e % DP;
             if (tok < n_tok && c < d) gd_cp4(buf + (which * GD_TILE + tok) * DP + c, a.prep + (size_t)(t0 + tok) * a.P + offs[which] + c);
         }
     }
-    for (int e = tid; e < GD_TILE * (BC + 1); e += nthr) {
-        int tok = e / (BC + 1), c = e % (BC + 1);
+    for (int e = tid; e < GD_TILE * VS; e += nthr) {
+        int tok = e / VS, c = e % VS;
         if (tok >= n_tok) continue;
         const float* row = a.prep + (size_t)(t0 + tok) * a.P;
-        if (c < ncols) gd_cp4(vbuf + tok * (BC + 1) + c, row + 2 * G * d + h * a.dv + col0 + c);
-        else if (c == BC) gd_cp4(vbuf + tok * (BC + 1) + c, row + C + H * d + h);
+        if (c < ncols) gd_cp4(vbuf + tok * VS + c, row + 2 * G * d + h * a.dv + col0 + c);
+        else if (c == BC) gd_cp4(vbuf + tok * VS + c, row + off_beta);
+        else if (HD && c == BC + 1) gd_cp4(vbuf + tok * VS + c, row + C + h);
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
 }
+
+// Where row r of value channel j of a head's state lies: d rows of dv, then the extra channel's d numbers.
+__device__ __forceinline__ size_t gd_at(int r, int j, int d, int dv) { return j < dv ? (size_t)r * dv + j : (size_t)d * dv + r; }
 
 // A thread's rows: for m < RPT / 4 the four rows (m * GD_R + g) * 4 .. + 3, so that the lanes of a column read
 // consecutive float4 of a staged vector at a time (no bank conflicts; the other column of the warp reads the same
@@ -220,74 +317,78 @@ __device__ __forceinline__ void gd_stage(const GatedDeltaArgs& a, float* buf, in
 // chains' latencies overlap; every column's arithmetic is the same whatever NC is.
 // (Registers: with one column a thread four blocks of 128 threads share an SM, as many as the grid of a long prompt brings; with
 // two columns the grid is half as large and a thread may hold twice the registers, which spares it the spills.)
-template <int RPT, bool VEC, int GD_R, bool DELTA, int NC>
+template <int RPT, bool VEC, int GD_R, bool DELTA, int NC, bool HD>
 __global__ void __launch_bounds__(GD_R * GD_COLS, (NC == 1 ? 512 : 256) / (GD_R * GD_COLS)) gated_delta_walk_kernel(GatedDeltaArgs a, int n_buf) {
     ce_pdl_begin();
     extern __shared__ __align__(16) float gd_smem[];
-    constexpr int R4 = RPT / 4, BC = GD_COLS * NC;
+    constexpr int R4 = RPT / 4, BC = GD_COLS * NC, NV = HD ? 2 : 3, VS = BC + 2;
     int d = a.d, dv = a.dv;
     int h = blockIdx.x, b = blockIdx.y, col0 = blockIdx.z * BC, tid = threadIdx.x;
     int t_begin = a.q_start[b], t_end = a.q_start[b + 1];
     if (t_end <= t_begin) return;
-    int ncols = min(BC, dv - col0);
+    int ncols = max(0, min(BC, dv - col0)), all_cols = min(BC, dv + a.ones - col0);       // value channels; with the extra one
     constexpr bool delta = DELTA;              // false: the plain sum of outer products, whose write needs no dot product
     int jj = (tid / GD_R) * NC, g = tid % GD_R;          // this thread's columns: col0 + jj .. + NC - 1
     bool owner[NC];
-    float* sp = a.state + ((size_t)a.seq_slot[b] * a.H + h) * d * dv;
+    float* sp = a.state + ((size_t)a.seq_slot[b] * a.H + h) * d * (dv + a.ones);
     float S[NC][RPT];
 #pragma unroll
     for (int n = 0; n < NC; ++n) {
-        owner[n] = jj + n < ncols;
+        owner[n] = jj + n < all_cols;
 #pragma unroll
         for (int m = 0; m < RPT; ++m) {
             int row = ((m >> 2) * GD_R + g) * 4 + (m & 3);
-            S[n][m] = (owner[n] && row < d) ? sp[(size_t)row * dv + col0 + jj + n] : 0.f;
+            S[n][m] = (owner[n] && row < d) ? sp[gd_at(row, col0 + jj + n, d, dv)] : 0.f;
         }
     }
     // a row of the staged vectors is padded to GD_R * RPT floats, so that every thread reads whole float4
     constexpr int dp = GD_R * RPT;
-    int buf_floats = 3 * GD_TILE * dp + GD_TILE * (BC + 1);
+    int buf_floats = NV * GD_TILE * dp + GD_TILE * VS;
     buf_floats = (buf_floats + 3) / 4 * 4;
     // the padding of every staged row stays zero (rows of tokens a tile does not have are read ahead but never used)
     if (dp > d)
-        for (int e = tid; e < n_buf * 3 * GD_TILE * (dp - d); e += blockDim.x) {
+        for (int e = tid; e < n_buf * NV * GD_TILE * (dp - d); e += blockDim.x) {
             int row = e / (dp - d), c = d + e % (dp - d);
-            gd_smem[(row / (3 * GD_TILE)) * buf_floats + (row % (3 * GD_TILE)) * dp + c] = 0.f;
+            gd_smem[(row / (NV * GD_TILE)) * buf_floats + (row % (NV * GD_TILE)) * dp + c] = 0.f;
         }
     __syncthreads();
     int n_tiles = (t_end - t_begin + GD_TILE - 1) / GD_TILE;
-    gd_stage<dp, VEC, BC>(a, gd_smem, t_begin, min(GD_TILE, t_end - t_begin), h, col0, ncols);
+    gd_stage<dp, VEC, BC, HD>(a, gd_smem, t_begin, min(GD_TILE, t_end - t_begin), h, col0, ncols);
     for (int tile = 0; tile < n_tiles; ++tile) {
         int t0 = t_begin + tile * GD_TILE, n_tok = min(GD_TILE, t_end - t0);
         float* buf = gd_smem + (tile & (n_buf - 1)) * buf_floats;
         if (tile + 1 < n_tiles && n_buf == 2) {
-            gd_stage<dp, VEC, BC>(a, gd_smem + ((tile + 1) & 1) * buf_floats, t0 + GD_TILE, min(GD_TILE, t_end - t0 - GD_TILE), h, col0, ncols);
+            gd_stage<dp, VEC, BC, HD>(a, gd_smem + ((tile + 1) & 1) * buf_floats, t0 + GD_TILE, min(GD_TILE, t_end - t0 - GD_TILE), h, col0, ncols);
             asm volatile("cp.async.wait_group 1;" ::: "memory");
         } else {
-            if (tile > 0 && n_buf == 1) gd_stage<dp, VEC, BC>(a, buf, t0, n_tok, h, col0, ncols);     // one buffer: a tile is staged when its turn comes
+            if (tile > 0 && n_buf == 1) gd_stage<dp, VEC, BC, HD>(a, buf, t0, n_tok, h, col0, ncols);     // one buffer: a tile is staged when its turn comes
             asm volatile("cp.async.wait_group 0;" ::: "memory");
         }
         __syncthreads();
-        const float* vbuf = buf + 3 * GD_TILE * dp;
+        const float* vbuf = buf + NV * GD_TILE * dp;
         // The sum over rows of S^T q is not needed by the next token: every thread keeps its part for each token of
         // the tile, and the butterflies of all tokens run together after the walk (their latencies overlap).
         float part[NC][GD_TILE];
-        float4 w[R4], kw[R4], k[R4], q[R4];
-        float vj[NC], beta;
+        float4 w[HD ? 1 : R4], kw[R4], k[R4], q[R4];         // with one decay per head every element of w is w1
+        float vj[NC], beta, w1 = 1.f;
         auto lo2 = [](const float4& v) { return make_float2(v.x, v.y); };
         auto hi2 = [](const float4& v) { return make_float2(v.z, v.w); };
         auto fetch = [&](int tok) {                 // a token's vectors; nothing here depends on the state
+            if (HD) w1 = vbuf[tok * VS + BC + 1];
 #pragma unroll
             for (int m = 0; m < R4; ++m) {
-                w[m] = *reinterpret_cast<const float4*>(buf + (0 * GD_TILE + tok) * dp + (m * GD_R + g) * 4);
-                k[m] = *reinterpret_cast<const float4*>(buf + (1 * GD_TILE + tok) * dp + (m * GD_R + g) * 4);
-                q[m] = *reinterpret_cast<const float4*>(buf + (2 * GD_TILE + tok) * dp + (m * GD_R + g) * 4);
-                float2 a0 = __fmul2_rn(lo2(k[m]), lo2(w[m])), a1 = __fmul2_rn(hi2(k[m]), hi2(w[m]));
-                kw[m] = make_float4(a0.x, a0.y, a1.x, a1.y);
+                k[m] = *reinterpret_cast<const float4*>(buf + (0 * GD_TILE + tok) * dp + (m * GD_R + g) * 4);
+                q[m] = *reinterpret_cast<const float4*>(buf + (1 * GD_TILE + tok) * dp + (m * GD_R + g) * 4);
+                if (!HD) w[m] = *reinterpret_cast<const float4*>(buf + (2 * GD_TILE + tok) * dp + (m * GD_R + g) * 4);
+                if (delta) {
+                    float2 wl = HD ? make_float2(w1, w1) : lo2(w[HD ? 0 : m]), wh = HD ? make_float2(w1, w1) : hi2(w[HD ? 0 : m]);
+                    float2 a0 = __fmul2_rn(lo2(k[m]), wl), a1 = __fmul2_rn(hi2(k[m]), wh);
+                    kw[m] = make_float4(a0.x, a0.y, a1.x, a1.y);
+                }
             }
 #pragma unroll
-            for (int n = 0; n < NC; ++n) vj[n] = owner[n] ? vbuf[tok * (BC + 1) + jj + n] : 0.f;
-            beta = vbuf[tok * (BC + 1) + BC];
+            for (int n = 0; n < NC; ++n) vj[n] = jj + n < ncols ? vbuf[tok * VS + jj + n] : owner[n] ? 1.f : 0.f;
+            beta = vbuf[tok * VS + BC];
         };
         fetch(0);
         // The arithmetic on the state runs on pairs of rows (fma.f32x2: two IEEE operations an instruction, the same results):
@@ -313,8 +414,8 @@ __global__ void __launch_bounds__(GD_R * GD_COLS, (NC == 1 ? 512 : 256) / (GD_R 
                             p01 = __ffma2_rn(lo2(kw[m]), s01, p01);
                             p23 = __ffma2_rn(hi2(kw[m]), s23, p23);
                         }
-                        dS[n][2 * m] = __fmul2_rn(lo2(w[m]), s01);
-                        dS[n][2 * m + 1] = __fmul2_rn(hi2(w[m]), s23);
+                        dS[n][2 * m] = __fmul2_rn(HD ? make_float2(w1, w1) : lo2(w[HD ? 0 : m]), s01);
+                        dS[n][2 * m + 1] = __fmul2_rn(HD ? make_float2(w1, w1) : hi2(w[HD ? 0 : m]), s23);
                     }
                     dot[n] = (p01.x + p01.y) + (p23.x + p23.y);
                 }
@@ -347,7 +448,7 @@ __global__ void __launch_bounds__(GD_R * GD_COLS, (NC == 1 ? 512 : 256) / (GD_R 
                 }
 #pragma unroll
                 for (int n = 0; n < NC; ++n) {
-                    float u = delta ? beta_now * (v_now[n] - dot[n]) : v_now[n];         // the plain sum of outer products writes v itself
+                    float u = delta ? beta_now * (v_now[n] - dot[n]) : beta_now * v_now[n];         // the plain sum of outer products writes beta v
                     const float2 uu = make_float2(u, u);
                     float2 q01 = make_float2(0.f, 0.f), q23 = make_float2(0.f, 0.f);
 #pragma unroll
@@ -364,14 +465,21 @@ __global__ void __launch_bounds__(GD_R * GD_COLS, (NC == 1 ? 512 : 256) / (GD_R 
 #pragma unroll
         for (int n = 0; n < NC; ++n) {
 #pragma unroll
-            for (int o = 1; o < GD_R; o <<= 1)
+            for (int s = 0; s < 4; ++s) {
+                // lanes that differ in bit s add their parts; of every two tokens that differ in bit s a lane goes on with the
+                // one whose bit is its own, so that half the values are left and lane g ends with token g (GD_TILE is 16)
+                const bool odd = (g >> s) & 1;
 #pragma unroll
-                for (int tok = 0; tok < GD_TILE; ++tok) part[n][tok] += __shfl_xor_sync(0xffffffffu, part[n][tok], o);
-            // lane g of a column stores token g of the tile (GD_TILE <= GD_R)
-            float mine = part[n][0];
-#pragma unroll
-            for (int tok = 1; tok < GD_TILE; ++tok) mine = g == tok ? part[n][tok] : mine;
-            if (owner[n] && g < n_tok) a.raw[(size_t)(t0 + g) * a.H * dv + h * dv + col0 + jj + n] = mine;
+                for (int i = 0; i < (GD_TILE >> (s + 1)); ++i) {
+                    float mine = odd ? part[n][2 * i + 1] : part[n][2 * i], other = odd ? part[n][2 * i] : part[n][2 * i + 1];
+                    part[n][i] = mine + __shfl_xor_sync(0xffffffffu, other, 1 << s);
+                }
+            }
+            if (GD_R == 32) part[n][0] += __shfl_xor_sync(0xffffffffu, part[n][0], 16);
+            if (owner[n] && g < n_tok) {
+                int j = col0 + jj + n;
+                a.raw[(size_t)(t0 + g) * a.H * (dv + a.ones) + (j < dv ? h * dv + j : a.H * dv + h)] = part[n][0];
+            }
         }
         __syncthreads();             // the buffer is free for the tile after the next
     }
@@ -380,7 +488,7 @@ __global__ void __launch_bounds__(GD_R * GD_COLS, (NC == 1 ? 512 : 256) / (GD_R 
 #pragma unroll
         for (int m = 0; m < RPT; ++m) {
             int row = ((m >> 2) * GD_R + g) * 4 + (m & 3);
-            if (owner[n] && row < d) sp[(size_t)row * dv + col0 + jj + n] = S[n][m];
+            if (owner[n] && row < d) sp[gd_at(row, col0 + jj + n, d, dv)] = S[n][m];
         }
 }
 
@@ -392,41 +500,42 @@ __global__ void __launch_bounds__(GD_R * GD_COLS, (NC == 1 ? 512 : 256) / (GD_R 
 // the lanes for the read-out; quads, then quads of quads, for the dot product).  A token therefore gets the same bits whether
 // it arrives alone or inside a portion.
 #define GD_STEP_COLS 32
-template <int RPT, int GD_R, bool DELTA>
+template <int RPT, int GD_R, bool DELTA, bool HD>
 __global__ void __launch_bounds__(GD_R * GD_STEP_COLS) gated_delta_step_kernel(GatedDeltaArgs a) {
     ce_pdl_begin();
-    constexpr int R4 = RPT / 4, dp = GD_R * RPT;
-    __shared__ __align__(16) float vec[3 * dp];                    // decay, key, query of the token, padded with zeros
+    constexpr int R4 = RPT / 4, dp = GD_R * RPT, NV = HD ? 2 : 3;
+    __shared__ __align__(16) float vec[NV * dp];                   // key, query (and decay) of the token, padded with zeros
     __shared__ float dots[GD_R * GD_STEP_COLS], parts[GD_R * GD_STEP_COLS];
     int d = a.d, dv = a.dv, H = a.H, G = a.G;
     int h = blockIdx.x, b = blockIdx.y, tid = threadIdx.x;
     int c = tid % GD_STEP_COLS, g = tid / GD_STEP_COLS, j = blockIdx.z * GD_STEP_COLS + c;
     int t = a.q_start[b];
     if (a.q_start[b + 1] <= t) return;
-    bool owner = j < dv;
+    bool owner = j < dv + a.ones;
     int C = 2 * G * d + H * dv, kh = h / (H / G);
     const float* row = a.prep + (size_t)t * a.P;
-    int offs[3] = {C + h * d, G * d + kh * d, kh * d};          // decay, key, query within a prep row
-    for (int e = tid; e < 3 * dp; e += blockDim.x) {
+    int offs[3] = {G * d + kh * d, kh * d, C + h * d};          // key, query, decay within a prep row
+    for (int e = tid; e < NV * dp; e += blockDim.x) {
         int which = e / dp, i = e % dp;
         vec[e] = i < d ? row[offs[which] + i] : 0.f;
     }
-    float* sp = a.state + ((size_t)a.seq_slot[b] * H + h) * d * dv;
+    float* sp = a.state + ((size_t)a.seq_slot[b] * H + h) * d * (dv + a.ones);
     float S[RPT];
 #pragma unroll
     for (int m = 0; m < RPT; ++m) {
         int r = ((m >> 2) * GD_R + g) * 4 + (m & 3);
-        S[m] = (owner && r < d) ? sp[(size_t)r * dv + j] : 0.f;
+        S[m] = (owner && r < d) ? sp[gd_at(r, j, d, dv)] : 0.f;
     }
-    float vj = owner ? row[2 * G * d + h * dv + j] : 0.f, beta = row[C + H * d + h];
+    float vj = j < dv ? row[2 * G * d + h * dv + j] : owner ? 1.f : 0.f, beta = row[C + (HD ? H : H * d) + h];
+    const float w1 = HD ? row[C + h] : 1.f;
     __syncthreads();
     float w[RPT], k[RPT], q[RPT], dS[RPT];
     float p0 = 0.f, p1 = 0.f, p2 = 0.f, p3 = 0.f;
 #pragma unroll
     for (int m4 = 0; m4 < R4; ++m4) {
-        const float4 w4 = *reinterpret_cast<const float4*>(vec + 0 * dp + (m4 * GD_R + g) * 4);
-        const float4 k4 = *reinterpret_cast<const float4*>(vec + 1 * dp + (m4 * GD_R + g) * 4);
-        const float4 q4 = *reinterpret_cast<const float4*>(vec + 2 * dp + (m4 * GD_R + g) * 4);
+        const float4 k4 = *reinterpret_cast<const float4*>(vec + 0 * dp + (m4 * GD_R + g) * 4);
+        const float4 q4 = *reinterpret_cast<const float4*>(vec + 1 * dp + (m4 * GD_R + g) * 4);
+        const float4 w4 = HD ? make_float4(w1, w1, w1, w1) : *reinterpret_cast<const float4*>(vec + (NV - 1) * dp + (m4 * GD_R + g) * 4);
         w[4 * m4] = w4.x; w[4 * m4 + 1] = w4.y; w[4 * m4 + 2] = w4.z; w[4 * m4 + 3] = w4.w;
         k[4 * m4] = k4.x; k[4 * m4 + 1] = k4.y; k[4 * m4 + 2] = k4.z; k[4 * m4 + 3] = k4.w;
         q[4 * m4] = q4.x; q[4 * m4 + 1] = q4.y; q[4 * m4 + 2] = q4.z; q[4 * m4 + 3] = q4.w;
@@ -439,7 +548,7 @@ __global__ void __launch_bounds__(GD_R * GD_STEP_COLS) gated_delta_step_kernel(G
 #pragma unroll
         for (int i = 0; i < 4; ++i) dS[4 * m4 + i] = __fmul_rn(w[4 * m4 + i], S[4 * m4 + i]);
     }
-    float u = vj;
+    float u = __fmul_rn(beta, vj);
     if (DELTA) {
         dots[g * GD_STEP_COLS + c] = __fadd_rn(__fadd_rn(p0, p1), __fadd_rn(p2, p3));
         __syncthreads();
@@ -466,7 +575,7 @@ __global__ void __launch_bounds__(GD_R * GD_STEP_COLS) gated_delta_step_kernel(G
 #pragma unroll
     for (int m = 0; m < RPT; ++m) {
         int r = ((m >> 2) * GD_R + g) * 4 + (m & 3);
-        if (owner && r < d) sp[(size_t)r * dv + j] = S[m];
+        if (owner && r < d) sp[gd_at(r, j, d, dv)] = S[m];
     }
     parts[g * GD_STEP_COLS + c] = __fadd_rn(__fadd_rn(q0, q1), __fadd_rn(q2, q3));
     __syncthreads();
@@ -479,7 +588,7 @@ __global__ void __launch_bounds__(GD_R * GD_STEP_COLS) gated_delta_step_kernel(G
         for (int o = 1; o < GD_R; o <<= 1)
 #pragma unroll
             for (int n = 0; n < GD_R; n += 2 * o) tree[n] = __fadd_rn(tree[n], tree[n + o]);
-        a.raw[(size_t)t * H * dv + h * dv + j] = tree[0];
+        a.raw[(size_t)t * H * (dv + a.ones) + (j < dv ? h * dv + j : H * dv + h)] = tree[0];
     }
 }
 
@@ -490,21 +599,55 @@ __global__ void gated_delta_finish_kernel(GatedDeltaArgs a) {
     int t = blockIdx.x, lane = threadIdx.x & 31, nwarp = (blockDim.x >> 5) * gridDim.y;
     int warp = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5);
     int dv = a.dv, n = a.H * dv;
-    const float* o = a.raw + (size_t)t * n;
+    const float* o = a.raw + (size_t)t * a.H * (dv + a.ones);
     const float* gz = a.gz + (size_t)t * a.ld_gz;
     for (int h = warp; h < a.H; h += nwarp) {
+        float den = 1.f;
+        if (a.ones) {
+            float m = a.prep[(size_t)t * a.P + 2 * a.G * a.d + n + 2 * a.H + h];
+            den = fmaxf(fabsf(o[n + h]), expf(-m)) + 1e-6f;
+        }
         float ss = 0.f;
-        for (int c = lane; c < dv; c += 32) ss = fmaf(o[h * dv + c], o[h * dv + c], ss);
+        for (int c = lane; c < dv; c += 32) { float v = o[h * dv + c] / den; ss = fmaf(v, v, ss); }
         for (int k = 16; k > 0; k >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, k);
         float inv = 1.0f / sqrtf(ss / (float)dv + a.eps);
         for (int c = lane; c < dv; c += 32) {
             int col = h * dv + c;
             float z = gz[col], g = gd_sigmoid(z);
             if (a.gate_act == 1) g *= z;
-            float y = o[col] * inv;
-            if (a.norm_w) y *= a.norm_w[c];
+            float y = o[col] / den * inv;
+            if (a.norm_w) y *= a.norm_w[a.norm_all ? col : c];
             CeType<T>::store((T*)a.out + (size_t)t * n + col, y * g * a.out_scale);
         }
+    }
+}
+
+// The other order (parts > 0): a block per (token, part) of all heads' values: y = (o + skip_h v) gate(z), divided by the part's
+// own root mean square, times the weight.
+template <typename T>
+__global__ void gated_delta_part_finish_kernel(GatedDeltaArgs a) {
+    ce_pdl_begin();
+    extern __shared__ float gd_part_smem[];          // the part's values
+    __shared__ float scratch[32];
+    int t = blockIdx.x, n = a.H * a.dv, size = n / a.parts, c0 = blockIdx.y * size;
+    const float* o = a.raw + (size_t)t * n;
+    const float* v = a.prep + (size_t)t * a.P + 2 * a.G * a.d;
+    const float* gz = a.gz + (size_t)t * a.ld_gz;
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < size; i += blockDim.x) {
+        int c = c0 + i;
+        float z = gz[c], g = gd_sigmoid(z);
+        if (a.gate_act == 1) g *= z;
+        float y = (a.skip ? fmaf(a.skip[c / a.dv], v[c], o[c]) : o[c]) * g;
+        gd_part_smem[i] = y;
+        ss = fmaf(y, y, ss);
+    }
+    float inv = 1.0f / sqrtf(ce_block_sum(ss, scratch) / (float)size + a.eps);
+    for (int i = threadIdx.x; i < size; i += blockDim.x) {          // (every thread reads what it wrote)
+        int c = c0 + i;
+        float y = gd_part_smem[i] * inv;
+        if (a.norm_w) y *= a.norm_w[c];
+        CeType<T>::store((T*)a.out + (size_t)t * n + c, y * a.out_scale);
     }
 }
 
@@ -512,20 +655,24 @@ __global__ void gated_delta_finish_kernel(GatedDeltaArgs a) {
 template <int RPT, int R, int NC>
 static void gd_launch_walk_nc(const GatedDeltaArgs& a, int B, bool vec, int n_buf, cudaStream_t stream) {
     constexpr int BC = GD_COLS * NC;
-    size_t floats = 3 * GD_TILE * R * RPT + GD_TILE * (BC + 1);
+    const bool hd = gd_head_decay(a.decay_mode);
+    size_t floats = (hd ? 2 : 3) * GD_TILE * R * RPT + GD_TILE * (BC + 2);
     size_t smem = (size_t)n_buf * ((floats + 3) / 4 * 4) * sizeof(float);
-    dim3 grid(a.H, B, (a.dv + BC - 1) / BC);
+    dim3 grid(a.H, B, (a.dv + a.ones + BC - 1) / BC);
     ce_note("gated_delta_walk_kernel");
     auto go = [&](auto kernel) {
         if (smem > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         ce_launch(kernel, grid, R * GD_COLS, smem, stream, a, n_buf);
     };
-    if (a.rule == 0) {
-        if (vec) go(gated_delta_walk_kernel<RPT, true, R, true, NC>);
-        else go(gated_delta_walk_kernel<RPT, false, R, true, NC>);
-    } else {
-        if (vec) go(gated_delta_walk_kernel<RPT, true, R, false, NC>);
-        else go(gated_delta_walk_kernel<RPT, false, R, false, NC>);
+    if (a.rule == 0 && !hd) {
+        if (vec) go(gated_delta_walk_kernel<RPT, true, R, true, NC, false>);
+        else go(gated_delta_walk_kernel<RPT, false, R, true, NC, false>);
+    } else if (a.rule == 0) {
+        if (vec) go(gated_delta_walk_kernel<RPT, true, R, true, NC, true>);
+        else go(gated_delta_walk_kernel<RPT, false, R, true, NC, true>);
+    } else {                         // (the plain sum of outer products always has one decay per head)
+        if (vec) go(gated_delta_walk_kernel<RPT, true, R, false, NC, true>);
+        else go(gated_delta_walk_kernel<RPT, false, R, false, NC, true>);
     }
 }
 
@@ -544,25 +691,36 @@ static void gd_launch_walk(const GatedDeltaArgs& a, int B, bool vec, int n_buf, 
 }
 
 // Floats of a ``prep`` row for these sizes.
-extern "C" int ce_gated_delta_prep_width(int H, int G, int d, int dv) {
-    return (2 * G * d + H * dv + H * d + H + 3) / 4 * 4;
+extern "C" int ce_gated_delta_prep_width(int H, int G, int d, int dv, int decay_mode) {
+    int gates = decay_mode == 0 ? H * d + H : decay_mode == 3 ? 3 * H : 2 * H;
+    return (2 * G * d + H * dv + gates + 3) / 4 * 4;
 }
 
-// stage: 1 prepare, 2 keep, 3 walk, 4 finish (each one launch, so that each is counted and timed by itself)
+// stage: 1 prepare, 2 keep (or, with exponential gates, scan), 3 walk, 4 finish (each one launch, so that each is counted and timed
+// by itself).  A step of single tokens (T == B) has no stage 2.
 extern "C" int ce_gated_delta(const float* proj, const float* dec, const float* gz, const float* taps, const float* a_log,
                               const float* dt_bias, const float* norm_w, float* prep, float* raw, float* state, float* kept,
                               void* out, int out_dtype, const int* seq_of_token, const int* seq_slot, const int* q_start,
                               int T, int B, int ld, int off_conv, int off_b, int H, int G, int d, int dv, int K, float eps,
                               int ld_dec, int ld_gz, int decay_mode, int operands, int rule, int gate_act, float out_scale,
                               const float* cos_table, const float* sin_table, const int* positions, int* status, int rd, int max_pos,
-                              int stage, cudaStream_t stream) {
+                              const float* conv_bias, const float* skip, float* m_state, float cap, int write_mode, int ones,
+                              int norm_all, int parts, int stage, cudaStream_t stream) {
     if (B == 0 || T == 0) return CE_OK;
     if (stage < 1 || stage > 4) return ce_fail(CE_ERR_ARG, "ce_gated_delta: stage %d", stage);
-    if (decay_mode < 0 || decay_mode > 2 || operands < 0 || operands > 1 || rule < 0 || rule > 1 || gate_act < 0 || gate_act > 1)
+    if (decay_mode < 0 || decay_mode > 3 || operands < 0 || operands > 3 || rule < 0 || rule > 1 || gate_act < 0 || gate_act > 1 ||
+        write_mode < 0 || write_mode > 1 || ones < 0 || ones > 1)
         return ce_fail(CE_ERR_ARG, "ce_gated_delta: decay %d, operands %d, rule %d, gate %d", decay_mode, operands, rule, gate_act);
-    if (!proj || !gz || !a_log || !prep || !raw || !state || !out || !seq_of_token || !seq_slot || !q_start ||
-        (decay_mode != 2 && (!dec || !dt_bias)) || (operands == 0 && (!taps || (K > 1 && !kept))))
+    const bool conv = operands == 0 || operands == 2;
+    if (!proj || !gz || (!a_log && decay_mode != 3) || !prep || !raw || !state || !out || !seq_of_token || !seq_slot || !q_start ||
+        (decay_mode != 2 && (!dec || !dt_bias)) || (conv && (!taps || (K > 1 && !kept))) || (decay_mode == 3 && !m_state))
         return ce_fail(CE_ERR_ARG, "ce_gated_delta: null pointer");
+    if ((operands == 3) != (decay_mode == 3) || (ones && decay_mode != 3) || (decay_mode == 3 && (rule != 1 || K != 1 || !(cap > 0.f))))
+        return ce_fail(CE_ERR_ARG, "ce_gated_delta: exponential gates come with plain operands, the plain sum and a positive cap");
+    if ((decay_mode == 0 && rule == 1) || (write_mode == 1 && decay_mode != 1))
+        return ce_fail(CE_ERR_ARG, "ce_gated_delta: decay %d does not go with rule %d and write %d", decay_mode, rule, write_mode);
+    if (parts < 0 || (parts > 0 && ((H * dv) % parts || ones || H * dv / parts > 48 * 1024)))
+        return ce_fail(CE_ERR_SIZE, "ce_gated_delta: %d values normalised in %d parts", H * dv, parts);
     if (operands == 1) {
         if (K != 1 || decay_mode != 2) return ce_fail(CE_ERR_ARG, "ce_gated_delta: rotated operands come without a convolution and with constant decays");
         if (rd < 0 || rd > d || rd % 2) return ce_fail(CE_ERR_SIZE, "ce_gated_delta: %d rotated elements of %d", rd, d);
@@ -572,10 +730,11 @@ extern "C" int ce_gated_delta(const float* proj, const float* dec, const float* 
     if (H <= 0 || G <= 0 || H % G || B > 65535 || K < 1 || K > 64)
         return ce_fail(CE_ERR_SIZE, "ce_gated_delta: %d heads, %d key heads, %d sequences, %d taps", H, G, B, K);
     if (out_dtype != CE_F32 && out_dtype != CE_BF16) return ce_fail(CE_ERR_ARG, "ce_gated_delta: unknown dtype %d", out_dtype);
-    int P = ce_gated_delta_prep_width(H, G, d, dv);
+    int P = ce_gated_delta_prep_width(H, G, d, dv, decay_mode);
     GatedDeltaArgs a{proj, dec, gz, taps, a_log, dt_bias, norm_w, prep, raw, state, kept, out, seq_of_token, seq_slot, q_start,
                      ld, off_conv, off_b, H, G, d, dv, K, P, eps, ld_dec, ld_gz, decay_mode, operands, rule, gate_act, out_scale,
-                     rd > 0 ? cos_table : nullptr, sin_table, positions, status, rd, max_pos};
+                     rd > 0 ? cos_table : nullptr, sin_table, positions, status, rd, max_pos, conv_bias, skip, m_state, cap,
+                     write_mode, ones, norm_all, parts, T == B ? 1 : 0};
     int heads = 2 * G + H;
     int threads = heads >= 8 ? 256 : 32 * heads;
     if (stage == 1) {
@@ -584,10 +743,26 @@ extern "C" int ce_gated_delta(const float* proj, const float* dec, const float* 
         int split = want < room ? want : room;
         ce_launch(gated_delta_prepare_kernel, dim3(T, split < 1 ? 1 : split), threads, 0, stream, a);
     } else if (stage == 2) {
+        if (T == B) return CE_OK;               // prepare has done it
+        if (decay_mode == 3) {
+            ce_note("gated_delta_scan_kernel");
+            ce_launch(gated_delta_scan_kernel, dim3(B, (H + 31) / 32), 256, 0, stream, a);
+            return ce_check_launch("ce_gated_delta");
+        }
         if (K == 1) return CE_OK;
         size_t total = (size_t)B * (2 * G * d + H * dv), want = (total + 255) / 256;
         ce_note("gated_delta_keep_kernel");
         ce_launch(gated_delta_keep_kernel, (int)(want < 148 * 8 ? want : 148 * 8), 256, 0, stream, a, B);
+    } else if (stage == 4 && parts > 0) {
+        ce_note("gated_delta_part_finish_kernel");
+        int size = H * dv / parts, th = size >= 2048 ? 256 : size >= 512 ? 128 : 64;
+        size_t smem = (size_t)size * sizeof(float);
+        auto go = [&](auto kernel) {
+            if (smem > 40 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+            ce_launch(kernel, dim3(T, parts), th, smem, stream, a);
+        };
+        if (out_dtype == CE_F32) go(gated_delta_part_finish_kernel<float>);
+        else go(gated_delta_part_finish_kernel<__nv_bfloat16>);
     } else if (stage == 4) {
         ce_note("gated_delta_finish_kernel");
         int th = H >= 8 ? 256 : 32 * H;
@@ -605,11 +780,12 @@ extern "C" int ce_gated_delta(const float* proj, const float* dec, const float* 
         int n_buf = T == B ? 1 : 2;             // as many tokens as sequences: every sequence brings exactly one
         static int no_step = getenv("CE_DELTA_NO_STEP") ? 1 : 0;       // (for measurement: single tokens on the walk)
         if (T == B && !no_step) {
-            dim3 grid(H, B, (dv + GD_STEP_COLS - 1) / GD_STEP_COLS);
+            dim3 grid(H, B, (dv + ones + GD_STEP_COLS - 1) / GD_STEP_COLS);
             ce_note("gated_delta_step_kernel");
 #define GD_STEP_CASE(RPT, R)                                                                                      \
-            if (a.rule == 0) ce_launch(gated_delta_step_kernel<RPT, R, true>, grid, R * GD_STEP_COLS, 0, stream, a);  \
-            else ce_launch(gated_delta_step_kernel<RPT, R, false>, grid, R * GD_STEP_COLS, 0, stream, a);
+            if (a.rule == 0 && decay_mode == 0) ce_launch(gated_delta_step_kernel<RPT, R, true, false>, grid, R * GD_STEP_COLS, 0, stream, a);  \
+            else if (a.rule == 0) ce_launch(gated_delta_step_kernel<RPT, R, true, true>, grid, R * GD_STEP_COLS, 0, stream, a);  \
+            else ce_launch(gated_delta_step_kernel<RPT, R, false, true>, grid, R * GD_STEP_COLS, 0, stream, a);
             if (d <= 64) { GD_STEP_CASE(4, 16) } else if (d <= 128) { GD_STEP_CASE(8, 16) } else { GD_STEP_CASE(8, 32) }
 #undef GD_STEP_CASE
             return ce_check_launch("ce_gated_delta");

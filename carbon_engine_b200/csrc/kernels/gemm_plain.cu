@@ -8,20 +8,26 @@
 //
 // Epilogues: store (in the activation dtype or float32), add into the float32 residual stream, or
 // SwiGLU, where W holds the gate rows [0, N) and the up rows [N, 2N) and the output is
-// silu(gate) * up (src/model/layers.rs:625-648), or relu(gate) * up.
+// silu(gate) * up (src/model/layers.rs:625-648), relu(gate) * up, or the clamped gated activation of gate and up rows
+// with an optional bias.
 #include "common.cuh"
 
 #define GP_BM 64
 #define GP_BN 64
 #define GP_BK 16
 
-enum { GP_STORE = 0, GP_STORE_F32 = 1, GP_ACCUM_F32 = 2, GP_SWIGLU = 3, GP_RELUGLU = 4, GP_RELU2 = 5 };     // 4: relu(gate) * up; 5: relu(v)^2
+enum { GP_STORE = 0, GP_STORE_F32 = 1, GP_ACCUM_F32 = 2, GP_SWIGLU = 3, GP_RELUGLU = 4, GP_RELU2 = 5, GP_CLAMPGLU = 6 };     // 4: relu(gate) * up; 5: relu(v)^2; 6: ce_clamp_glu(gate + bias, up + bias)
+
+struct GpGate {
+    const float* bias;           // float32 [2N] or null: gate rows, then up rows (mode 6)
+    float limit, alpha;
+};
 
 template <typename T, int MODE>
 __global__ void __launch_bounds__(256) gemm_plain_kernel(const T* __restrict__ A, const T* __restrict__ W,
-                                                         void* __restrict__ Cv, int M, int N, int K, int lda, int ldc) {
+                                                         void* __restrict__ Cv, int M, int N, int K, int lda, int ldc, GpGate gate) {
     ce_pdl_begin();
-    constexpr int NW = (MODE == GP_SWIGLU || MODE == GP_RELUGLU) ? 2 : 1;
+    constexpr int NW = (MODE == GP_SWIGLU || MODE == GP_RELUGLU || MODE == GP_CLAMPGLU) ? 2 : 1;
     __shared__ float As[GP_BK][GP_BM + 1];
     __shared__ float Ws[NW][GP_BK][GP_BN + 1];
     int tid = threadIdx.x;
@@ -82,6 +88,10 @@ __global__ void __launch_bounds__(256) gemm_plain_kernel(const T* __restrict__ A
             } else if (MODE == GP_RELU2) {
                 float v = fmaxf(acc[0][i][j], 0.f);
                 CeType<T>::store((T*)Cv + o, v * v);
+            } else if (MODE == GP_CLAMPGLU) {
+                float g = acc[0][i][j], u = acc[NW - 1][i][j];
+                if (gate.bias) { g += gate.bias[gn]; u += gate.bias[N + gn]; }
+                CeType<T>::store((T*)Cv + o, ce_clamp_glu(g, u, gate.limit, gate.alpha));
             } else if (MODE == GP_RELUGLU) {
                 CeType<T>::store((T*)Cv + o, fmaxf(acc[0][i][j], 0.f) * acc[NW - 1][i][j]);
             } else {
@@ -94,15 +104,16 @@ __global__ void __launch_bounds__(256) gemm_plain_kernel(const T* __restrict__ A
 
 template <typename T>
 static int launch_plain(const void* A, const void* W, void* C, int M, int N, int K, int lda, int ldc, int mode,
-                        cudaStream_t stream) {
+                        GpGate gate, cudaStream_t stream) {
     dim3 grid((N + GP_BN - 1) / GP_BN, (M + GP_BM - 1) / GP_BM);
     switch (mode) {
-        case GP_STORE: { ce_note("gemm_plain_kernel"); ce_launch(gemm_plain_kernel<T, GP_STORE>, grid, 256, 0, stream, (const T*)A, (const T*)W, C, M, N, K, lda, ldc); } break;
-        case GP_STORE_F32: { ce_note("gemm_plain_kernel"); ce_launch(gemm_plain_kernel<T, GP_STORE_F32>, grid, 256, 0, stream, (const T*)A, (const T*)W, C, M, N, K, lda, ldc); } break;
-        case GP_ACCUM_F32: { ce_note("gemm_plain_kernel"); ce_launch(gemm_plain_kernel<T, GP_ACCUM_F32>, grid, 256, 0, stream, (const T*)A, (const T*)W, C, M, N, K, lda, ldc); } break;
-        case GP_SWIGLU: { ce_note("gemm_plain_kernel"); ce_launch(gemm_plain_kernel<T, GP_SWIGLU>, grid, 256, 0, stream, (const T*)A, (const T*)W, C, M, N, K, lda, ldc); } break;
-        case GP_RELUGLU: { ce_note("gemm_plain_kernel"); ce_launch(gemm_plain_kernel<T, GP_RELUGLU>, grid, 256, 0, stream, (const T*)A, (const T*)W, C, M, N, K, lda, ldc); } break;
-        case GP_RELU2: { ce_note("gemm_plain_kernel"); ce_launch(gemm_plain_kernel<T, GP_RELU2>, grid, 256, 0, stream, (const T*)A, (const T*)W, C, M, N, K, lda, ldc); } break;
+        case GP_STORE: { ce_note("gemm_plain_kernel"); ce_launch(gemm_plain_kernel<T, GP_STORE>, grid, 256, 0, stream, (const T*)A, (const T*)W, C, M, N, K, lda, ldc, gate); } break;
+        case GP_STORE_F32: { ce_note("gemm_plain_kernel"); ce_launch(gemm_plain_kernel<T, GP_STORE_F32>, grid, 256, 0, stream, (const T*)A, (const T*)W, C, M, N, K, lda, ldc, gate); } break;
+        case GP_ACCUM_F32: { ce_note("gemm_plain_kernel"); ce_launch(gemm_plain_kernel<T, GP_ACCUM_F32>, grid, 256, 0, stream, (const T*)A, (const T*)W, C, M, N, K, lda, ldc, gate); } break;
+        case GP_SWIGLU: { ce_note("gemm_plain_kernel"); ce_launch(gemm_plain_kernel<T, GP_SWIGLU>, grid, 256, 0, stream, (const T*)A, (const T*)W, C, M, N, K, lda, ldc, gate); } break;
+        case GP_RELUGLU: { ce_note("gemm_plain_kernel"); ce_launch(gemm_plain_kernel<T, GP_RELUGLU>, grid, 256, 0, stream, (const T*)A, (const T*)W, C, M, N, K, lda, ldc, gate); } break;
+        case GP_RELU2: { ce_note("gemm_plain_kernel"); ce_launch(gemm_plain_kernel<T, GP_RELU2>, grid, 256, 0, stream, (const T*)A, (const T*)W, C, M, N, K, lda, ldc, gate); } break;
+        case GP_CLAMPGLU: { ce_note("gemm_plain_kernel"); ce_launch(gemm_plain_kernel<T, GP_CLAMPGLU>, grid, 256, 0, stream, (const T*)A, (const T*)W, C, M, N, K, lda, ldc, gate); } break;
         default: return ce_fail(CE_ERR_ARG, "ce_gemm_plain: unknown epilogue %d", mode);
     }
     return ce_check_launch("ce_gemm_plain");
@@ -110,12 +121,13 @@ static int launch_plain(const void* A, const void* W, void* C, int M, int N, int
 
 // N is the number of output columns (for SwiGLU: the intermediate width, W having 2N rows).
 extern "C" int ce_gemm_plain(const void* A, const void* W, void* C, int dtype, int M, int N, int K, int lda, int ldc,
-                             int mode, cudaStream_t stream) {
+                             int mode, const float* bias, float limit, float alpha, cudaStream_t stream) {
+    GpGate gate{bias, limit, alpha};
     if (M == 0 || N == 0) return CE_OK;
     if (!A || !W || !C) return ce_fail(CE_ERR_ARG, "ce_gemm_plain: null pointer");
     if (K <= 0) return ce_fail(CE_ERR_SIZE, "ce_gemm_plain: K=%d", K);
     if ((M + GP_BM - 1) / GP_BM > 65535) return ce_fail(CE_ERR_SIZE, "ce_gemm_plain: M=%d is too large", M);
-    if (dtype == CE_F32) return launch_plain<float>(A, W, C, M, N, K, lda, ldc, mode, stream);
-    if (dtype == CE_BF16) return launch_plain<__nv_bfloat16>(A, W, C, M, N, K, lda, ldc, mode, stream);
+    if (dtype == CE_F32) return launch_plain<float>(A, W, C, M, N, K, lda, ldc, mode, gate, stream);
+    if (dtype == CE_BF16) return launch_plain<__nv_bfloat16>(A, W, C, M, N, K, lda, ldc, mode, gate, stream);
     return ce_fail(CE_ERR_ARG, "ce_gemm_plain: unknown dtype %d", dtype);
 }

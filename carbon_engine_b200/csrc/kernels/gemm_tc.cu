@@ -38,8 +38,8 @@ constexpr int UMMA_K = 16;
 constexpr int THREADS = 192;
 constexpr uint32_t SPIN_LIMIT = 1u << 20;     // with the back-off below: about a second at most
 
-enum { TC_STORE = 0, TC_STORE_F32 = 1, TC_ACCUM_F32 = 2, TC_SWIGLU = 3, TC_RELUGLU = 4, TC_RELU2 = 5 };     // 4: relu(gate) * up, laid out and tiled like 3; 5: relu(v)^2 stored like 0
-#define TC_GATED(mode) ((mode) == TC_SWIGLU || (mode) == TC_RELUGLU)
+enum { TC_STORE = 0, TC_STORE_F32 = 1, TC_ACCUM_F32 = 2, TC_SWIGLU = 3, TC_RELUGLU = 4, TC_RELU2 = 5, TC_CLAMPGLU = 6 };     // 4: relu(gate) * up, laid out and tiled like 3; 5: relu(v)^2 stored like 0; 6: the clamped gated activation of gate + bias and up + bias, like 3
+#define TC_GATED(mode) ((mode) == TC_SWIGLU || (mode) == TC_RELUGLU || (mode) == TC_CLAMPGLU)
 
 __device__ __forceinline__ uint32_t smem_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
 
@@ -135,14 +135,23 @@ struct TcArgs {
     int M, N, K, ldo, mode, splits, kblocks_per_split, kblocks, trace;
     int cluster;             // 1: the splits of a tile form a cluster and add their partial sums through shared memory
     int coop;                // 1: every split of a tile adds the partial sums for a share of the tile's tokens (more than 8 tokens)
+    const float* bias;       // mode 6: float32 [2N] (gate rows, then up rows) or null
+    float limit, alpha;      // mode 6
 };
 
 __device__ __forceinline__ float silu_mul(float g, float u) { return g / (1.0f + __expf(-g)) * u; }
 // the same with the approximate reciprocal (the result is rounded to bfloat16 right after)
 __device__ __forceinline__ float silu_mul_fast(float g, float u) { return __fdividef(g, 1.0f + __expf(-g)) * u; }
-// the gated epilogue's activation by mode
-__device__ __forceinline__ float gated_mul(int mode, float g, float u) { return mode == TC_RELUGLU ? fmaxf(g, 0.f) * u : silu_mul(g, u); }
-__device__ __forceinline__ float gated_mul_fast(int mode, float g, float u) { return mode == TC_RELUGLU ? fmaxf(g, 0.f) * u : silu_mul_fast(g, u); }
+// the gated epilogue's activation by mode; bg, bu: the feature's biases (mode 6)
+__device__ __forceinline__ float gated_mul(const TcArgs& a, float g, float u, float bg, float bu) {
+    if (a.mode == TC_CLAMPGLU) return ce_clamp_glu_fast(g + bg, u + bu, a.limit, a.alpha);
+    return a.mode == TC_RELUGLU ? fmaxf(g, 0.f) * u : silu_mul(g, u);
+}
+__device__ __forceinline__ float gated_mul_fast(const TcArgs& a, float g, float u, float bg, float bu) {
+    if (a.mode == TC_CLAMPGLU) return ce_clamp_glu_fast(g + bg, u + bu, a.limit, a.alpha);
+    return a.mode == TC_RELUGLU ? fmaxf(g, 0.f) * u : silu_mul_fast(g, u);
+}
+__device__ __forceinline__ float gate_bias(const TcArgs& a, int n, int up) { return a.bias && n < a.N ? a.bias[up * a.N + n] : 0.f; }
 
 __device__ __forceinline__ void epilogue_store(const TcArgs& a, int m, int n, float v, float up) {
     size_t o = (size_t)m * a.ldo + n;
@@ -150,7 +159,7 @@ __device__ __forceinline__ void epilogue_store(const TcArgs& a, int m, int n, fl
     else if (a.mode == TC_STORE_F32) ((float*)a.out)[o] = v;
     else if (a.mode == TC_ACCUM_F32) ((float*)a.out)[o] += v;
     else if (a.mode == TC_RELU2) { float r = fmaxf(v, 0.f); ((__nv_bfloat16*)a.out)[o] = __float2bfloat16_rn(r * r); }
-    else ((__nv_bfloat16*)a.out)[o] = __float2bfloat16_rn(gated_mul(a.mode, v, up));
+    else ((__nv_bfloat16*)a.out)[o] = __float2bfloat16_rn(gated_mul(a, v, up, gate_bias(a, n, 0), gate_bias(a, n, 1)));
 }
 
 template <int BN, int NACC, bool COOP>
@@ -303,6 +312,7 @@ __global__ void __launch_bounds__(THREADS, 2) gemm_tc_kernel(const __grid_consta
             // two threads of a feature share each chunk of 16 tokens: the gate thread takes tokens 0..7 (and
             // needs their up values), the up thread tokens 8..15 (and needs their gate values).
             bool up_row = row >= 64;
+            const float bg = gate_bias(a, n, 0), bu = gate_bias(a, n, 1);
 #pragma unroll 1
             for (int c = 0; c < BN; c += 16) {
                 if (c >= m_valid) break;
@@ -327,7 +337,7 @@ __global__ void __launch_bounds__(THREADS, 2) gemm_tc_kernel(const __grid_consta
                     for (int j = 0; j < 8; ++j) {
                         float gate = up_row ? xg[j] : g[j];
                         float upv = up_row ? g[8 + j] : xu[j];
-                        if (c + t0 + j < m_valid) op[(size_t)j * a.ldo] = __float2bfloat16_rn(gated_mul_fast(a.mode, gate, upv));
+                        if (c + t0 + j < m_valid) op[(size_t)j * a.ldo] = __float2bfloat16_rn(gated_mul_fast(a, gate, upv, bg, bu));
                     }
                 }
             }
@@ -545,14 +555,17 @@ __global__ void __launch_bounds__(THREADS, 2) gemm_tc_kernel(const __grid_consta
 // A block takes 128 output features of one tile: the same roles and pipeline as the kernel above, without split-K.
 // Where N is no multiple of 128 the last box of an expert reaches into the next expert's rows (or past the stack's
 // end, which reads zeros): those features are not stored.  Without tables it is one expert's product over the rows as
-// they lie.  Epilogue: store in bfloat16, optionally the square of relu first.
+// they lie.  Epilogue: store in bfloat16, optionally the square of relu first, or (act 2) the clamped gated activation of row
+// pairs: an expert's rows are then gate and up rows by turns (row 2j the gate of feature j, row 2j + 1 its up), neighbouring lanes
+// hold a feature's two values, and N / 2 features are stored.
 // ---------------------------------------------------------------------------------------------
 struct TcGroupArgs {
     __nv_bfloat16* out;          // [rows, ldo]
     const int* tile_expert;      // [tiles] or null
     const int* n_tiles;          // [1] or null
     int* status;
-    int rows, N, K, ldo, kblocks, act;       // act 1: relu(v)^2
+    int rows, N, K, ldo, kblocks, act;       // act 1: relu(v)^2; 2: the clamped gated activation of row pairs
+    float limit, alpha;
 };
 
 template <int BN>
@@ -669,7 +682,19 @@ __global__ void __launch_bounds__(THREADS, 2) gemm_tc_grouped_kernel(const __gri
 #pragma unroll
                     for (int j = 0; j < 16; ++j) g[j] = 0.f;
                 }
-                if (n < a.N) {
+                if (a.act == 2) {
+                    // the lane of the gate row takes tokens 0..7 of the chunk and needs their up values, the lane of the up row
+                    // tokens 8..15 and needs their gate values
+                    const bool up_row = n & 1;
+                    const int t0 = up_row ? 8 : 0;
+                    __nv_bfloat16* op = a.out + (size_t)(m0 + c + t0) * a.ldo + (n >> 1);
+#pragma unroll
+                    for (int j = 0; j < 8; ++j) {
+                        float other = __shfl_xor_sync(0xffffffffu, up_row ? g[j] : g[8 + j], 1);
+                        float gate = up_row ? other : g[j], up = up_row ? g[8 + j] : other;
+                        if (n < a.N && c + t0 + j < m_valid) op[(size_t)j * a.ldo] = __float2bfloat16_rn(ce_clamp_glu_fast(gate, up, a.limit, a.alpha));
+                    }
+                } else if (n < a.N) {
                     __nv_bfloat16* op = a.out + (size_t)(m0 + c) * a.ldo + n;
 #pragma unroll
                     for (int j = 0; j < 16; ++j) {
@@ -1030,6 +1055,7 @@ __global__ void __launch_bounds__(THREADS) gemm_tc_pair_kernel(const __grid_cons
             int buf = lt & 1;
             int n = (tile / tiles_m) * (2 * ROWS_N) + rank * ROWS_N + (GU ? (row & 63) : row);
             bool up_row = GU && row >= 64;
+            const float bg = GU ? gate_bias(a, n, 0) : 0.f, bu = GU ? gate_bias(a, n, 1) : 0.f;
             int m0 = (tile % tiles_m) * BN;
             int m_valid = min(BN, a.M - m0);
             const bool accum = !GU && a.mode == TC_ACCUM_F32 && n < a.N;
@@ -1090,7 +1116,7 @@ __global__ void __launch_bounds__(THREADS) gemm_tc_pair_kernel(const __grid_cons
                         for (int j = 0; j < 16; ++j) {
                             float gate = up_row ? xg[j] : g[j];
                             float upv = up_row ? g[16 + j] : xu[j];
-                            if (c + t0 + j < m_valid) op[(size_t)j * a.ldo] = __float2bfloat16_rn(gated_mul_fast(a.mode, gate, upv));
+                            if (c + t0 + j < m_valid) op[(size_t)j * a.ldo] = __float2bfloat16_rn(gated_mul_fast(a, gate, upv, bg, bu));
                         }
                     }
                     continue;
@@ -1305,13 +1331,13 @@ extern "C" int ce_gemm_tc_supported(int M, int N, int K, int lda) {
 // (for SwiGLU the intermediate width).  counters: at least ceil(N/128) * ceil(M/BN) zeroed ints.
 extern "C" int ce_gemm_tc(const void* A, const void* W, void* C, int M, int N, int K, int lda, int ldc, int mode,
                           float* scratch, long long scratch_floats, int* counters, int n_counters, int* status,
-                          cudaStream_t stream) {
+                          const float* bias, float limit, float alpha, cudaStream_t stream) {
     if (M == 0 || N == 0) return CE_OK;
     if (!A || !W || !C || !status) return ce_fail(CE_ERR_ARG, "ce_gemm_tc: null pointer");
     if (!ce_gemm_tc_supported(M, N, K, lda))
         return ce_fail(CE_ERR_SIZE, "ce_gemm_tc: K=%d and the row stride %d must be multiples of 8", K, lda);
     if (((uintptr_t)A | (uintptr_t)W) & 15) return ce_fail(CE_ERR_SIZE, "ce_gemm_tc: operands must be 16-byte aligned");
-    if (mode < 0 || mode > 5) return ce_fail(CE_ERR_ARG, "ce_gemm_tc: unknown epilogue %d", mode);
+    if (mode < 0 || mode > 6) return ce_fail(CE_ERR_ARG, "ce_gemm_tc: unknown epilogue %d", mode);
     int nacc = TC_GATED(mode) ? 2 : 1;
     int kblocks = (K + BK - 1) / BK;
     bool early_pairs = pairs_from_129(M, N, nacc);
@@ -1324,7 +1350,7 @@ extern "C" int ce_gemm_tc(const void* A, const void* W, void* C, int M, int N, i
         if (prc) return prc;
         if ((prc = get_map(A, M, K, lda, pbn, &px))) return prc;
         static int ptrace = getenv("CE_GEMM_TRACE") ? 1 : 0;
-        TcArgs pa{C, scratch, counters, status, M, N, K, ldc, mode, 1, kblocks, kblocks, ptrace, 0};
+        TcArgs pa{C, scratch, counters, status, M, N, K, ldc, mode, 1, kblocks, kblocks, ptrace, 0, 0, bias, limit, alpha};
         static int use_pairs = getenv("CE_GEMM_NO_PAIRS") ? 0 : 1;
         if (use_pairs && N >= 2 * BM) {     // CTA pairs: 256 weight rows a tile, each CTA loads half of the tokens
             // SwiGLU: 128 gate rows and their 128 up rows a pair tile (boxes of 64 rows), 256 tokens as well
@@ -1377,7 +1403,7 @@ extern "C" int ce_gemm_tc(const void* A, const void* W, void* C, int M, int N, i
     static int coop_off = getenv("CE_GEMM_NO_COOP") ? 1 : 0;
     int coop = !coop_off && splits > 1 && !cluster && M > 8 && (long long)grid.x * grid.y * grid.z <= resident &&
                n_counters >= 2 * (int)(grid.x * grid.y);
-    TcArgs a{C, scratch, counters, status, M, N, K, ldc, mode, splits, (kblocks + splits - 1) / splits, kblocks, trace, cluster, coop};
+    TcArgs a{C, scratch, counters, status, M, N, K, ldc, mode, splits, (kblocks + splits - 1) / splits, kblocks, trace, cluster, coop, bias, limit, alpha};
 #define TC_CASE(BN_)                                                                  \
     case BN_:                                                                         \
         return nacc == 2 ? launch<BN_, 2, false>(mw, mx, a, grid, stream)                  \
@@ -1419,14 +1445,15 @@ extern "C" int ce_gemm_tc_grouped_supported(int tile, int N, int K, int ldi, int
 
 // x [x_rows, ldi] bf16, W [experts, N, K] bf16, out [>= rows, ldo] bf16.  With the layout's tables (tile_expert [max_tiles],
 // n_tiles [1], both on the device) tile j of `tile` rows is expert tile_expert[j]'s and rows = max_tiles * tile; without
-// them it is expert 0's product over `rows` rows.  act: 0 none, 1 the square of relu.
+// them it is expert 0's product over `rows` rows.  act: 0 none, 1 the square of relu, 2 the clamped gated activation of row pairs
+// (N even; N / 2 columns are stored).
 extern "C" int ce_gemm_tc_grouped(const void* x, const void* W, void* out, const int* tile_expert, const int* n_tiles, int max_tiles,
-                                  int tile, int experts, int N, int K, int ldi, int ldo, int x_rows, int rows, int act, int* status,
-                                  cudaStream_t stream) {
+                                  int tile, int experts, int N, int K, int ldi, int ldo, int x_rows, int rows, int act, float limit,
+                                  float alpha, int* status, cudaStream_t stream) {
     if (max_tiles == 0 || rows == 0 || N == 0) return CE_OK;
     if (!x || !W || !out || !status || (tile_expert == nullptr) != (n_tiles == nullptr))
         return ce_fail(CE_ERR_ARG, "ce_gemm_tc_grouped: null pointer");
-    if (!ce_gemm_tc_grouped_supported(tile, N, K, ldi, ldo) || experts <= 0 || act < 0 || act > 1)
+    if (!ce_gemm_tc_grouped_supported(tile, N, K, ldi, ldo) || experts <= 0 || act < 0 || act > 2 || (act == 2 && N % 2))
         return ce_fail(CE_ERR_SIZE, "ce_gemm_tc_grouped: tiles of %d rows, N=%d, K=%d, row stride %d", tile, N, K, ldi);
     if (((uintptr_t)x | (uintptr_t)W) & 15) return ce_fail(CE_ERR_SIZE, "ce_gemm_tc_grouped: operands must be 16-byte aligned");
     if (max_tiles > 65535 || (long long)experts * N > 2147483647LL || (long long)max_tiles * tile > (long long)rows + tile - 1 ||
@@ -1436,7 +1463,7 @@ extern "C" int ce_gemm_tc_grouped(const void* x, const void* W, void* out, const
     int rc = get_map(W, (long long)experts * N, K, K, BM, &mw);
     if (rc) return rc;
     if ((rc = get_map(x, x_rows, K, ldi, tile, &mx))) return rc;
-    TcGroupArgs a{(__nv_bfloat16*)out, tile_expert, n_tiles, status, rows, N, K, ldo, (K + BK - 1) / BK, act};
+    TcGroupArgs a{(__nv_bfloat16*)out, tile_expert, n_tiles, status, rows, N, K, ldo, (K + BK - 1) / BK, act, limit, alpha};
     dim3 grid((N + BM - 1) / BM, max_tiles);
     switch (tile) {
         case 16: return launch_grouped<16>(mw, mx, a, grid, stream);

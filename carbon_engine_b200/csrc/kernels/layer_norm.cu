@@ -159,6 +159,97 @@ __global__ void rmsnorm_add_vec_kernel(const float* __restrict__ y, const float*
     }
 }
 
+// The same, and the NEXT norm of the new x in the same pass:  y may still owe a bias (float32 [H] or null);
+//   x[t] += (y[t] + bias) / sqrt(mean((y[t] + bias)^2) + eps) * w;     h[t] = x[t] / sqrt(mean(x[t]^2) + eps2) * w2
+// h (or null: no next norm) is float32 or bfloat16.  VEC: float4 accesses, a row in registers (widths in multiples of 4 up to
+// 4 * threads * LNV_MAX).
+template <typename T, bool VEC>
+__global__ void rmsnorm_add_norm_kernel(const float* __restrict__ y, const float* __restrict__ bias, const float* __restrict__ w,
+                                        float* __restrict__ x, const float* __restrict__ w2, T* __restrict__ h, int H, float eps,
+                                        float eps2) {
+    ce_pdl_begin();
+    __shared__ float scratch[32];
+    const int t = blockIdx.x, tid = threadIdx.x;
+    if (VEC) {
+        const int H4 = H >> 2;
+        const float4* yr = reinterpret_cast<const float4*>(y + (size_t)t * H);
+        const float4* b4 = reinterpret_cast<const float4*>(bias);
+        const float4* w4 = reinterpret_cast<const float4*>(w);
+        float4* xr = reinterpret_cast<float4*>(x + (size_t)t * H);
+        float4 v[LNV_MAX], xv[LNV_MAX];
+        float q = 0.f;
+#pragma unroll
+        for (int n = 0; n < LNV_MAX; ++n) {
+            int j = tid + n * blockDim.x;
+            v[n] = j < H4 ? yr[j] : make_float4(0.f, 0.f, 0.f, 0.f);
+            xv[n] = j < H4 ? xr[j] : make_float4(0.f, 0.f, 0.f, 0.f);
+            if (bias && j < H4) { float4 b = b4[j]; v[n].x += b.x; v[n].y += b.y; v[n].z += b.z; v[n].w += b.w; }
+            q += (v[n].x * v[n].x + v[n].y * v[n].y) + (v[n].z * v[n].z + v[n].w * v[n].w);
+        }
+        float inv = 1.0f / sqrtf(ce_block_sum(q, scratch) / (float)H + eps);
+        q = 0.f;
+#pragma unroll
+        for (int n = 0; n < LNV_MAX; ++n) {
+            int j = tid + n * blockDim.x;
+            if (j < H4) {
+                float4 ww = w4[j];
+                xv[n].x += v[n].x * inv * ww.x; xv[n].y += v[n].y * inv * ww.y; xv[n].z += v[n].z * inv * ww.z; xv[n].w += v[n].w * inv * ww.w;
+                xr[j] = xv[n];
+            }
+            q += (xv[n].x * xv[n].x + xv[n].y * xv[n].y) + (xv[n].z * xv[n].z + xv[n].w * xv[n].w);
+        }
+        if (!h) return;
+        inv = 1.0f / sqrtf(ce_block_sum(q, scratch) / (float)H + eps2);
+        const float4* w24 = reinterpret_cast<const float4*>(w2);
+#pragma unroll
+        for (int n = 0; n < LNV_MAX; ++n) {
+            int j = tid + n * blockDim.x;
+            if (j >= H4) continue;
+            float4 ww = w24[j];
+            float o0 = xv[n].x * inv * ww.x, o1 = xv[n].y * inv * ww.y, o2 = xv[n].z * inv * ww.z, o3 = xv[n].w * inv * ww.w;
+            if (sizeof(T) == 4) reinterpret_cast<float4*>(h + (size_t)t * H)[j] = make_float4(o0, o1, o2, o3);
+            else {
+                __nv_bfloat162 lo = __floats2bfloat162_rn(o0, o1), hi = __floats2bfloat162_rn(o2, o3);
+                reinterpret_cast<uint2*>(h + (size_t)t * H)[j] = make_uint2(*reinterpret_cast<unsigned*>(&lo), *reinterpret_cast<unsigned*>(&hi));
+            }
+        }
+    } else {
+        const float* yr = y + (size_t)t * H;
+        float* xr = x + (size_t)t * H;
+        float q = 0.f;
+        for (int j = tid; j < H; j += blockDim.x) { float v = yr[j] + (bias ? bias[j] : 0.f); q = fmaf(v, v, q); }
+        float inv = 1.0f / sqrtf(ce_block_sum(q, scratch) / (float)H + eps);
+        q = 0.f;
+        for (int j = tid; j < H; j += blockDim.x) {
+            float v = xr[j] + (yr[j] + (bias ? bias[j] : 0.f)) * inv * w[j];
+            xr[j] = v;
+            q = fmaf(v, v, q);
+        }
+        if (!h) return;
+        inv = 1.0f / sqrtf(ce_block_sum(q, scratch) / (float)H + eps2);
+        for (int j = tid; j < H; j += blockDim.x) CeType<T>::store(h + (size_t)t * H + j, xr[j] * inv * w2[j]);       // (its own writes)
+    }
+}
+
+extern "C" int ce_rmsnorm_add_norm(const float* y, const float* bias, const float* w, float* x, const float* w2, void* h, int h_dtype,
+                                   int T, int H, float eps, float eps2, cudaStream_t stream) {
+    if (T == 0) return CE_OK;
+    if (!y || !w || !x || (h && !w2)) return ce_fail(CE_ERR_ARG, "ce_rmsnorm_add_norm: null pointer");
+    if (H <= 0 || (h_dtype != CE_F32 && h_dtype != CE_BF16)) return ce_fail(CE_ERR_ARG, "ce_rmsnorm_add_norm: width %d, dtype %d", H, h_dtype);
+    bool vec = H % 4 == 0 && H >= 256 && ((((uintptr_t)x | (uintptr_t)w | (uintptr_t)y | (uintptr_t)bias | (uintptr_t)w2 | (uintptr_t)h) & 15) == 0);
+    int H4 = H / 4, vt = H4 >= 2048 ? 1024 : H4 >= 512 ? 512 : H4 >= 256 ? 256 : 128;
+    ce_note("rmsnorm_add_norm_kernel");
+    if (vec && H4 <= vt * LNV_MAX) {
+        if (h_dtype == CE_F32) ce_launch(rmsnorm_add_norm_kernel<float, true>, T, vt, 0, stream, y, bias, w, x, w2, (float*)h, H, eps, eps2);
+        else ce_launch(rmsnorm_add_norm_kernel<__nv_bfloat16, true>, T, vt, 0, stream, y, bias, w, x, w2, (__nv_bfloat16*)h, H, eps, eps2);
+    } else {
+        int th = H >= 4096 ? 512 : H >= 1024 ? 256 : 128;
+        if (h_dtype == CE_F32) ce_launch(rmsnorm_add_norm_kernel<float, false>, T, th, 0, stream, y, bias, w, x, w2, (float*)h, H, eps, eps2);
+        else ce_launch(rmsnorm_add_norm_kernel<__nv_bfloat16, false>, T, th, 0, stream, y, bias, w, x, w2, (__nv_bfloat16*)h, H, eps, eps2);
+    }
+    return ce_check_launch("ce_rmsnorm_add_norm");
+}
+
 // xb (or null): receives the new x rounded to bfloat16, what a sublayer that reads the residual itself takes as its input
 extern "C" int ce_rmsnorm_add(const float* y, const float* w, float* x, void* xb, int T, int H, float eps, cudaStream_t stream) {
     if (T == 0) return CE_OK;

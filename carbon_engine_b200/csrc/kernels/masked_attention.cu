@@ -165,8 +165,15 @@ extern "C" int ce_norm_rope_kvwrite(const float* proj, void* q_out, void* k_pool
 // and the key/value row (r latent columns, then dr columns of the rotated key part, from off_kv).
 //   cq[t]  = rms_norm(query latent) * wq                                    -> [T, qr], activation dtype
 //   page row of the token = [ rms_norm(latent) * wkv | rotate(key part) ]   -> K pool [pages, 1, page, r + dr]
-// The rotation turns element i of the part's first rd with element i + rd/2 by the angle of the token's position.
+// The rotation turns, of the part's first rd elements, element i with element i + rd/2 (pairing 0) or 2i with 2i + 1 (pairing 1)
+// by angle i of the token's position.
 // ---------------------------------------------------------------------------------------------
+// Element i of a part of which the first rd elements turn (i < rd): its partner, and the index of its angle.
+__device__ __forceinline__ void rope_pair(int i, int half, int pairing, int& partner, int& angle, bool& first) {
+    if (pairing) { partner = i ^ 1; angle = i >> 1; first = (i & 1) == 0; }
+    else { first = i < half; partner = first ? i + half : i - half; angle = first ? i : i - half; }
+}
+
 struct LatentPrepArgs {
     const float* proj;
     const float* wq;             // [qr]
@@ -182,6 +189,7 @@ struct LatentPrepArgs {
     int* status;
     int ld, off_q, qr, off_kv, r, dr, rd, page_size, max_pages, num_pages, max_pos, write_kv;
     float eps;
+    int pairing;
 };
 
 template <typename T>
@@ -217,10 +225,14 @@ __global__ void latent_prepare_kernel(LatentPrepArgs a) {
     }
     const float* part = kv + a.r;
     for (int i = threadIdx.x; i < a.dr; i += blockDim.x) {
-        float v;
-        if (rotate && i < half) v = part[i] * a.cos_table[(size_t)p * half + i] - part[i + half] * a.sin_table[(size_t)p * half + i];
-        else if (rotate && i < a.rd) v = part[i] * a.cos_table[(size_t)p * half + i - half] + part[i - half] * a.sin_table[(size_t)p * half + i - half];
-        else v = part[i];
+        float v = part[i];
+        if (rotate && i < a.rd) {
+            int partner, angle;
+            bool first;
+            rope_pair(i, half, a.pairing, partner, angle, first);
+            float c = a.cos_table[(size_t)p * half + angle], s = a.sin_table[(size_t)p * half + angle];
+            v = first ? v * c - part[partner] * s : v * c + part[partner] * s;
+        }
         CeType<T>::store(dst + a.r + i, v);
     }
 }
@@ -229,7 +241,7 @@ extern "C" int ce_latent_prepare(const float* proj, const float* wq, const float
                                  const float* cos_table, const float* sin_table, const int* positions, const int* seq_of_token,
                                  const int* seq_slot, const int* block_table, int* status, int T, int ld, int off_q, int qr,
                                  int off_kv, int r, int dr, int rd, int page_size, int max_pages, int num_pages, int max_pos,
-                                 int write_kv, float eps, cudaStream_t stream) {
+                                 int write_kv, float eps, int pairing, cudaStream_t stream) {
     if (T == 0) return CE_OK;
     if (!proj || !positions || !seq_of_token || !seq_slot || !status || (qr > 0 && (!wq || !cq)))
         return ce_fail(CE_ERR_ARG, "ce_latent_prepare: null pointer");
@@ -237,7 +249,7 @@ extern "C" int ce_latent_prepare(const float* proj, const float* wq, const float
     if (rd < 0 || rd > dr || rd % 2 || (rd > 0 && (!cos_table || !sin_table)))
         return ce_fail(CE_ERR_SIZE, "ce_latent_prepare: %d rotated elements of %d", rd, dr);
     LatentPrepArgs a{proj, wq, wkv, cq, k_pool, cos_table, sin_table, positions, seq_of_token, seq_slot, block_table, status,
-                     ld, off_q, qr, off_kv, r, dr, rd, page_size, max_pages, num_pages, max_pos, write_kv, eps};
+                     ld, off_q, qr, off_kv, r, dr, rd, page_size, max_pages, num_pages, max_pos, write_kv, eps, pairing};
     int threads = (qr > r ? qr : r) >= 1024 ? 256 : 128;
     ce_note("latent_prepare_kernel");
     if (dtype == CE_F32) ce_launch(latent_prepare_kernel<float>, T, threads, 0, stream, a);
@@ -254,7 +266,7 @@ template <typename T>
 __global__ void rope_part_kernel(const T* __restrict__ src, int src_stride, int src_head, int src_off, T* __restrict__ dst,
                                  int dst_stride, int dst_head, int dst_off, const float* __restrict__ cos_table,
                                  const float* __restrict__ sin_table, const int* __restrict__ positions, int* __restrict__ status,
-                                 int H, int dr, int rd, int max_pos) {
+                                 int H, int dr, int rd, int max_pos, int pairing) {
     ce_pdl_begin();
     int t = blockIdx.x, p = positions[t], half = rd / 2;
     bool rotate = half > 0;
@@ -265,27 +277,29 @@ __global__ void rope_part_kernel(const T* __restrict__ src, int src_stride, int 
     for (int e = threadIdx.x; e < H * dr; e += blockDim.x) {
         int h = e / dr, i = e % dr;
         const T* s = src + (size_t)t * src_stride + (size_t)h * src_head + src_off;
-        float v;
-        if (rotate && i < half)
-            v = CeType<T>::load(s + i) * cos_table[(size_t)p * half + i] - CeType<T>::load(s + i + half) * sin_table[(size_t)p * half + i];
-        else if (rotate && i < rd)
-            v = CeType<T>::load(s + i) * cos_table[(size_t)p * half + i - half] + CeType<T>::load(s + i - half) * sin_table[(size_t)p * half + i - half];
-        else v = CeType<T>::load(s + i);
+        float v = CeType<T>::load(s + i);
+        if (rotate && i < rd) {
+            int partner, angle;
+            bool first;
+            rope_pair(i, half, pairing, partner, angle, first);
+            float c = cos_table[(size_t)p * half + angle], sn = sin_table[(size_t)p * half + angle], y = CeType<T>::load(s + partner);
+            v = first ? v * c - y * sn : v * c + y * sn;
+        }
         CeType<T>::store(dst + (size_t)t * dst_stride + (size_t)h * dst_head + dst_off + i, v);
     }
 }
 
 extern "C" int ce_rope_part(const void* src, int src_stride, int src_head, int src_off, void* dst, int dst_stride, int dst_head,
                             int dst_off, int dtype, const float* cos_table, const float* sin_table, const int* positions,
-                            int* status, int T, int H, int dr, int rd, int max_pos, cudaStream_t stream) {
+                            int* status, int T, int H, int dr, int rd, int max_pos, int pairing, cudaStream_t stream) {
     if (T == 0 || H == 0 || dr == 0) return CE_OK;
     if (!src || !dst || !positions || !status) return ce_fail(CE_ERR_ARG, "ce_rope_part: null pointer");
     if (rd < 0 || rd > dr || rd % 2 || (rd > 0 && (!cos_table || !sin_table)))
         return ce_fail(CE_ERR_SIZE, "ce_rope_part: %d rotated elements of %d", rd, dr);
     int threads = H * dr >= 1024 ? 256 : 128;
     ce_note("rope_part_kernel");
-    if (dtype == CE_F32) ce_launch(rope_part_kernel<float>, T, threads, 0, stream, (const float*)src, src_stride, src_head, src_off, (float*)dst, dst_stride, dst_head, dst_off, cos_table, sin_table, positions, status, H, dr, rd, max_pos);
-    else if (dtype == CE_BF16) ce_launch(rope_part_kernel<__nv_bfloat16>, T, threads, 0, stream, (const __nv_bfloat16*)src, src_stride, src_head, src_off, (__nv_bfloat16*)dst, dst_stride, dst_head, dst_off, cos_table, sin_table, positions, status, H, dr, rd, max_pos);
+    if (dtype == CE_F32) ce_launch(rope_part_kernel<float>, T, threads, 0, stream, (const float*)src, src_stride, src_head, src_off, (float*)dst, dst_stride, dst_head, dst_off, cos_table, sin_table, positions, status, H, dr, rd, max_pos, pairing);
+    else if (dtype == CE_BF16) ce_launch(rope_part_kernel<__nv_bfloat16>, T, threads, 0, stream, (const __nv_bfloat16*)src, src_stride, src_head, src_off, (__nv_bfloat16*)dst, dst_stride, dst_head, dst_off, cos_table, sin_table, positions, status, H, dr, rd, max_pos, pairing);
     else return ce_fail(CE_ERR_ARG, "ce_rope_part: unknown dtype %d", dtype);
     return ce_check_launch("ce_rope_part");
 }

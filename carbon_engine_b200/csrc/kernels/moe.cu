@@ -1,16 +1,18 @@
 // Mixture of experts: routing, the layout of a step's (token, expert) pairs by expert, the experts' two products as
 // grouped products over that layout, and the weighted sum back into token order.
 //
-//   route    z [T, ld] float32 router logits -> s = softmax(z[:E]); experts in `groups` equal groups of neighbours, a
-//            group's score the largest s in it, only the best `keep` groups' experts eligible; the `top` eligible experts
-//            with the largest s are chosen (ties: the lower index); weights s / (sum of the chosen s + 1e-20) * scale.
+//   route    z [T, ld] float32 router logits -> s = softmax(z[:E]) or sigmoid(z[:E]); choice scores c = s (+ a correction per
+//            expert); experts in `groups` equal groups of neighbours, a group's score the largest c in it or the sum of its two
+//            largest, only the best `keep` groups' experts eligible; the `top` eligible experts with the largest c are chosen
+//            (ties: the lower index); weights s / (sum of the chosen s + 1e-20) * scale, or s * scale as they are.
 //            Column E of z, where there is one, is the logit of a shared expert's gate: sgate[t] = sigmoid(z[t, E]).
 //   align    the T*top pairs sorted by expert into rows of a padded layout: every expert's rows start at a multiple of
 //            the tile height BM, so a tile of BM rows belongs to ONE expert.  row_token[p] is the token of row p (-1: a
 //            padding row), pair_row[i] the row of pair i, tile_expert[j] the expert of tile j, n_tiles[0] their count.
 //            Nothing of it reaches the host: the products launch a grid for the most tiles a step of that size can have,
 //            and blocks past n_tiles leave at once, so a captured graph replays with any routing.
-//   products out[p] = act(in[row p's token, or p] W[e]^T), e = tile_expert[p / BM]; act = relu^2 or none.  Every output
+//   products out[p] = act(in[row p's token, or p] W[e]^T), e = tile_expert[p / BM]; act = none, relu^2, or the clamped gated
+//            activation of row pairs (rows 2j and 2j + 1 of W[e] are feature j's gate and up).  Every output
 //            element is a sum over k in a fixed order that depends on neither the row's place in its tile nor on the
 //            other rows, so a token's result does not depend on the batch.  float32 FMA for any size and both dtypes;
 //            bfloat16 on the tensor cores (wmma m16n16k16, float32 sums) for sizes in multiples of 16.
@@ -30,6 +32,10 @@ struct MoeRouteArgs {
     float* sgate;       // [T] or null
     int T, ld, E, top, groups, keep;
     float scale;
+    const float* correction;     // [E] or null: added to the scores for the choice, not for the weights
+    int scoring;                 // 0: softmax over the experts, 1: sigmoid
+    int group_score;             // 0: a group's largest choice score, 1: the sum of its two largest
+    int renormalize;             // 1: the weights are divided by the sum of the chosen scores
 };
 
 __device__ __forceinline__ void moe_warp_argmax(float& v, int& i) {
@@ -46,34 +52,44 @@ __global__ void __launch_bounds__(128) moe_route_kernel(MoeRouteArgs a) {
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int t = blockIdx.x * 4 + warp;
     if (t >= a.T) return;
-    float* s = moe_route_smem + (size_t)warp * 2 * a.E;      // scores; a chosen or barred expert's score becomes -1
-    float* gs = s + a.E;                                     // the groups' scores
+    float* s = moe_route_smem + (size_t)warp * 3 * a.E;      // scores
+    float* c = s + a.E;                                      // choice scores; a chosen or barred expert's becomes -inf
+    float* gs = c + a.E;                                     // the groups' scores; a kept group's becomes +inf
     const float* zr = a.z + (size_t)t * a.ld;
-    float mx = -INFINITY;
-    for (int e = lane; e < a.E; e += 32) mx = fmaxf(mx, zr[e]);
-    for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
-    float sum = 0.f;
-    for (int e = lane; e < a.E; e += 32) { float v = expf(zr[e] - mx); s[e] = v; sum += v; }
-    for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
-    const float inv = 1.0f / sum;
-    for (int e = lane; e < a.E; e += 32) s[e] *= inv;
+    if (a.scoring == 0) {
+        float mx = -INFINITY;
+        for (int e = lane; e < a.E; e += 32) mx = fmaxf(mx, zr[e]);
+        for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+        float sum = 0.f;
+        for (int e = lane; e < a.E; e += 32) { float v = expf(zr[e] - mx); s[e] = v; sum += v; }
+        for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+        const float inv = 1.0f / sum;
+        for (int e = lane; e < a.E; e += 32) s[e] *= inv;
+    } else {
+        for (int e = lane; e < a.E; e += 32) s[e] = 1.0f / (1.0f + expf(-zr[e]));
+    }
+    for (int e = lane; e < a.E; e += 32) c[e] = a.correction ? s[e] + a.correction[e] : s[e];
     __syncwarp();
     if (a.groups > 1 && a.keep < a.groups) {
         const int size = a.E / a.groups;
         for (int g = lane; g < a.groups; g += 32) {
-            float best = -1.f;
-            for (int j = 0; j < size; ++j) best = fmaxf(best, s[g * size + j]);
-            gs[g] = best;
+            float best = -INFINITY, second = -INFINITY;
+            for (int j = 0; j < size; ++j) {
+                float v = c[g * size + j];
+                second = fmaxf(second, fminf(v, best));
+                best = fmaxf(best, v);
+            }
+            gs[g] = a.group_score == 1 && size > 1 ? best + second : best;
         }
         __syncwarp();
-        for (int k = 0; k < a.keep; ++k) {                   // the best groups' scores become 2 (a score is at most 1)
-            float v = -1.f; int i = 0x7fffffff;
-            for (int g = lane; g < a.groups; g += 32) if (gs[g] <= 1.f && gs[g] > v) { v = gs[g]; i = g; }
+        for (int k = 0; k < a.keep; ++k) {
+            float v = -INFINITY; int i = 0x7fffffff;
+            for (int g = lane; g < a.groups; g += 32) if (gs[g] < INFINITY && gs[g] > v) { v = gs[g]; i = g; }
             moe_warp_argmax(v, i);
-            if (lane == 0) gs[i] = 2.f;
+            if (lane == 0 && i < a.groups) gs[i] = INFINITY;
             __syncwarp();
         }
-        for (int e = lane; e < a.E; e += 32) if (gs[e / size] <= 1.f) s[e] = -1.f;
+        for (int e = lane; e < a.E; e += 32) if (gs[e / size] < INFINITY) c[e] = -INFINITY;
         __syncwarp();
     }
     float total = 0.f, mine = 0.f;                           // lane k keeps the k-th pick (32 picks at a time)
@@ -81,34 +97,39 @@ __global__ void __launch_bounds__(128) moe_route_kernel(MoeRouteArgs a) {
     for (int k0 = 0; k0 < a.top; k0 += 32) {
         const int n = min(32, a.top - k0);
         for (int k = 0; k < n; ++k) {
-            float v = -1.f; int i = 0x7fffffff;
-            for (int e = lane; e < a.E; e += 32) if (s[e] > v) { v = s[e]; i = e; }
+            float v = -INFINITY; int i = 0x7fffffff;
+            for (int e = lane; e < a.E; e += 32) if (c[e] > v) { v = c[e]; i = e; }
             moe_warp_argmax(v, i);
-            if (lane == k) { mine = v; mine_id = i; }
-            if (lane == 0) s[i] = -1.f;
-            total += v;
+            if (i >= a.E) i = k0 + k;                        // (only scores that are no numbers leave nothing to choose)
+            const float w = s[i];
+            if (lane == k) { mine = w; mine_id = i; }
+            if (lane == 0) c[i] = -INFINITY;
+            total += w;
             __syncwarp();
         }
         if (lane < n) {
             a.ids[(size_t)t * a.top + k0 + lane] = mine_id;
-            a.weights[(size_t)t * a.top + k0 + lane] = mine;        // divided below, once the sum is known
+            a.weights[(size_t)t * a.top + k0 + lane] = mine;        // scaled below, once the sum is known
         }
     }
     __syncwarp();
-    const float norm = a.scale / (total + 1e-20f);
+    const float norm = a.renormalize ? a.scale / (total + 1e-20f) : a.scale;
     for (int k = lane; k < a.top; k += 32) a.weights[(size_t)t * a.top + k] *= norm;
     if (a.sgate && lane == 0) a.sgate[t] = 1.0f / (1.0f + expf(-zr[a.E]));
 }
 
 extern "C" int ce_moe_route(const float* z, int* ids, float* weights, float* sgate, int T, int ld, int E, int top, int groups,
-                            int keep, float scale, cudaStream_t stream) {
+                            int keep, float scale, const float* correction, int scoring, int group_score, int renormalize,
+                            cudaStream_t stream) {
     if (T == 0) return CE_OK;
     if (!z || !ids || !weights) return ce_fail(CE_ERR_ARG, "ce_moe_route: null pointer");
     if (E <= 0 || E > MOE_MAX_EXPERTS || top <= 0 || top > E || groups <= 0 || E % groups || keep <= 0 || keep > groups ||
         (long long)keep * (E / groups) < top || ld < E + (sgate ? 1 : 0))
         return ce_fail(CE_ERR_SIZE, "ce_moe_route: %d experts, top %d, %d groups of which %d are kept", E, top, groups, keep);
-    MoeRouteArgs a{z, ids, weights, sgate, T, ld, E, top, groups, keep, scale};
-    size_t smem = (size_t)4 * 2 * E * sizeof(float);
+    if (scoring < 0 || scoring > 1 || group_score < 0 || group_score > 1)
+        return ce_fail(CE_ERR_ARG, "ce_moe_route: scoring %d, group score %d", scoring, group_score);
+    MoeRouteArgs a{z, ids, weights, sgate, T, ld, E, top, groups, keep, scale, correction, scoring, group_score, renormalize};
+    size_t smem = (size_t)4 * 3 * E * sizeof(float);
     if (smem > 40 * 1024) cudaFuncSetAttribute(moe_route_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     ce_note("moe_route_kernel");
     ce_launch(moe_route_kernel, (T + 3) / 4, 128, smem, stream, a);
@@ -197,7 +218,7 @@ extern "C" int ce_moe_align(const int* ids, int n_pairs, int top, int E, int BM,
 // ---------------------------------------------------------------------------------------------
 // grouped products
 // ---------------------------------------------------------------------------------------------
-enum { MOE_ACT_NONE = 0, MOE_ACT_RELU2 = 1 };
+enum { MOE_ACT_NONE = 0, MOE_ACT_RELU2 = 1, MOE_ACT_CLAMPGLU = 2 };      // 2: of row pairs (gate, up), one output a pair
 
 __device__ __forceinline__ float moe_act(int act, float v) {
     if (act == MOE_ACT_RELU2) { v = fmaxf(v, 0.f); return v * v; }
@@ -212,6 +233,7 @@ struct MoeMatmulArgs {
     const int* tile_expert;
     const int* n_tiles;          // or null: every tile of the grid
     int ldi, ldo, N, K, BM, act, n_rows;     // n_rows: rows of `in` when they are taken as they lie (later rows are padding)
+    float limit, alpha;          // act 2
 };
 
 #define MP_BN 64
@@ -264,6 +286,14 @@ __global__ void __launch_bounds__(256) moe_matmul_plain_kernel(MoeMatmulArgs a) 
 #pragma unroll
     for (int i = 0; i < RPT; ++i) {
         if (src[tm + i] < 0) continue;
+        if (a.act == MOE_ACT_CLAMPGLU) {
+#pragma unroll
+            for (int j = 0; j < 4; j += 2)
+                if (n0 + tn + j < a.N)
+                    CeType<T>::store((T*)a.out + (size_t)(p0 + tm + i) * a.ldo + (n0 + tn + j) / 2,
+                                     ce_clamp_glu(acc[i][j], acc[i][j + 1], a.limit, a.alpha));
+            continue;
+        }
 #pragma unroll
         for (int j = 0; j < 4; ++j)
             if (n0 + tn + j < a.N) CeType<T>::store((T*)a.out + (size_t)(p0 + tm + i) * a.ldo + n0 + tn + j, moe_act(a.act, acc[i][j]));
@@ -327,20 +357,26 @@ __global__ void __launch_bounds__(128) moe_matmul_wmma_kernel(MoeMatmulArgs a) {
     for (int e = tid; e < BM * (MW_BN / 2); e += 128) {
         int r = e / (MW_BN / 2), c = (e % (MW_BN / 2)) * 2;
         if (src[r] < 0 || n0 + c >= a.N) continue;
+        if (a.act == MOE_ACT_CLAMPGLU) {
+            ((__nv_bfloat16*)a.out)[(size_t)(p0 + r) * a.ldo + (n0 + c) / 2] =
+                __float2bfloat16_rn(ce_clamp_glu_fast(Cs[r][c], Cs[r][c + 1], a.limit, a.alpha));
+            continue;
+        }
         __nv_bfloat162 v = __floats2bfloat162_rn(moe_act(a.act, Cs[r][c]), moe_act(a.act, Cs[r][c + 1]));
         *reinterpret_cast<__nv_bfloat162*>((__nv_bfloat16*)a.out + (size_t)(p0 + r) * a.ldo + n0 + c) = v;
     }
 }
 
-// in [*, ldi], W [E, N, K], out [max_tiles * BM, ldo]; BM is 16 or 64 and is the tile height the layout was made with.
+// in [*, ldi], W [E, N, K], out [max_tiles * BM, ldo] (N columns, N / 2 with the activation of row pairs); BM is 16 or 64 and is the tile height the layout was made with.
 // Without the layout's tables (all three null) it is one expert's product over n_rows rows as they lie.
 extern "C" int ce_moe_matmul(const void* in, const void* W, void* out, const int* row_token, const int* tile_expert,
                              const int* n_tiles, int dtype, int max_tiles, int BM, int N, int K, int ldi, int ldo, int act,
-                             int n_rows, cudaStream_t stream) {
+                             float limit, float alpha, int n_rows, cudaStream_t stream) {
     if (max_tiles == 0 || N == 0) return CE_OK;
     if (!in || !W || !out || K <= 0) return ce_fail(CE_ERR_ARG, "ce_moe_matmul: null pointer or K=%d", K);
     if ((BM != 16 && BM != 64) || max_tiles > 65535) return ce_fail(CE_ERR_SIZE, "ce_moe_matmul: tiles of %d rows, %d tiles", BM, max_tiles);
-    MoeMatmulArgs a{in, W, out, row_token, tile_expert, n_tiles, ldi, ldo, N, K, BM, act, n_rows};
+    if (act < 0 || act > 2 || (act == MOE_ACT_CLAMPGLU && N % 2)) return ce_fail(CE_ERR_ARG, "ce_moe_matmul: activation %d of %d rows", act, N);
+    MoeMatmulArgs a{in, W, out, row_token, tile_expert, n_tiles, ldi, ldo, N, K, BM, act, n_rows, limit, alpha};
     if (dtype == CE_BF16 && N % 16 == 0 && K % 16 == 0 && ldi % 8 == 0 && ldo % 2 == 0 &&
         ((((uintptr_t)in) & 15) == 0) && ((((uintptr_t)W) & 31) == 0) && ((((uintptr_t)out) & 3) == 0)) {
         dim3 grid((N + MW_BN - 1) / MW_BN, max_tiles);

@@ -102,6 +102,8 @@ class StepContext:
         self.plans: Dict[str, Any] = {}
         #: what a layer leaves for later layers of the SAME step (values that later layers blend with their own), by name
         self.shared: Dict[str, Any] = {}
+        #: the norm in front of the layer run that follows the running one, where that block names it (``leading_norm``)
+        self.next_norm = None
         self._scratch = {}
         self.n_decode = 0                    # the first n_decode sequences bring exactly one token
         self.max_position = 0

@@ -15,8 +15,10 @@ from .csrc.kernel_lib import KernelError, kernels
 
 F32, BF16 = 0, 1
 GEMM_STORE, GEMM_STORE_F32, GEMM_ACCUM_F32, GEMM_SWIGLU, GEMM_RELUGLU, GEMM_RELU2 = 0, 1, 2, 3, 4, 5      # 5: relu(v)^2, stored like 0
-#: epilogues whose weight holds gate rows and up rows: act(gate) * up with act = SiLU or ReLU
-GEMM_GATED = (GEMM_SWIGLU, GEMM_RELUGLU)
+#: g = min(gate + bias, limit), u = up + bias cut to [-limit, limit]: g sigmoid(alpha g) (u + 1)
+GEMM_CLAMPGLU = 6
+#: epilogues whose weight holds gate rows and up rows: act(gate) * up with act = SiLU or ReLU, or the clamped one
+GEMM_GATED = (GEMM_SWIGLU, GEMM_RELUGLU, GEMM_CLAMPGLU)
 ROPE_PAIRINGS = {"half": 0, "interleaved": 1}
 
 
@@ -178,6 +180,27 @@ def reset_kernel_counts() -> None:
     kernels().ce_kernel_counts_reset()
 
 
+class GluParams:
+    """What the clamped gated epilogue needs: the limit, the sigmoid's factor and an optional bias (float32, gate values then up
+    values)."""
+
+    def __init__(self, limit: float, alpha: float, bias: Optional[torch.Tensor] = None):
+        self.limit, self.alpha, self.bias = float(limit), float(alpha), bias
+
+
+def glu_args(glu: Optional[GluParams], mode: int, n: int):
+    """(bias pointer, limit, alpha) for a product with ``n`` output columns."""
+    if mode != GEMM_CLAMPGLU:
+        return None, 0.0, 0.0
+    if glu is None:
+        raise KernelError("the clamped gated epilogue needs its limit and factor")
+    if glu.bias is not None:
+        _need(glu.bias, "bias", torch.float32)
+        if glu.bias.numel() < 2 * n:
+            raise KernelError(f"the gated epilogue's bias has {glu.bias.numel()} elements, not {2 * n}")
+    return _ptr(glu.bias), glu.limit, glu.alpha
+
+
 def embed(table: torch.Tensor, tokens: torch.Tensor, x: torch.Tensor, status: torch.Tensor, scale: float = 1.0) -> None:
     """x[t, :] = table[tokens[t], :] * scale as float32."""
     _need(table, "table"); _need(tokens, "tokens", torch.int32); _need(x, "x", torch.float32)
@@ -253,6 +276,16 @@ def reluglu(gate_up: torch.Tensor, out: torch.Tensor) -> None:
     _ok(kernels().ce_reluglu(_ptr(gate_up), _ptr(out), dtype_code(out.dtype), T, I, _stream()))
 
 
+def clamp_glu(gate_up: torch.Tensor, out: torch.Tensor, glu: GluParams) -> None:
+    """out[t, i] = the clamped gated activation of gate_up[t, i] and gate_up[t, I + i] (plus the bias)."""
+    _need(gate_up, "gate_up"); _need(out, "out", gate_up.dtype)
+    T, I = out.shape
+    if gate_up.shape != (T, 2 * I):
+        raise KernelError("clamp_glu: gate_up must be [T, 2I]")
+    bias, limit, alpha = glu_args(glu, GEMM_CLAMPGLU, I)
+    _ok(kernels().ce_clamp_glu(_ptr(gate_up), _ptr(out), dtype_code(out.dtype), bias, limit, alpha, T, I, _stream()))
+
+
 def relu2(inp: torch.Tensor, out: torch.Tensor) -> None:
     """out[t, i] = relu(inp[t, i])^2; inp contiguous [T, I], out rows of stride out.stride(0)."""
     _need(inp, "inp")
@@ -285,6 +318,26 @@ def rmsnorm_add(y: torch.Tensor, weight: torch.Tensor, x: torch.Tensor, eps: flo
         if rounded.shape != x.shape:
             raise KernelError("rmsnorm_add: the rounded copy must have the shape of x")
     _ok(kernels().ce_rmsnorm_add(_ptr(y), _ptr(weight), _ptr(x), _ptr(rounded), x.shape[0], x.shape[1], float(eps), _stream()))
+
+
+def rmsnorm_add_norm(y: torch.Tensor, weight: torch.Tensor, x: torch.Tensor, eps: float, bias: Optional[torch.Tensor] = None,
+                     next_weight: Optional[torch.Tensor] = None, next_eps: float = 0.0, out: Optional[torch.Tensor] = None) -> None:
+    """x[t] += rmsnorm(y[t] + bias) * weight; then, with ``out``, out[t] = rmsnorm(x[t]) * next_weight: the norm of a sublayer's
+    output added into the residual, and the norm in front of the next sublayer, in one pass.  All float32 but ``out``."""
+    _need(y, "y", torch.float32); _need(weight, "weight", torch.float32); _need(x, "x", torch.float32)
+    T, W = x.shape
+    if y.shape != x.shape or weight.numel() != W:
+        raise KernelError("rmsnorm_add_norm: sizes differ")
+    if bias is not None:
+        _need(bias, "bias", torch.float32)
+        if bias.numel() != W:
+            raise KernelError("rmsnorm_add_norm: the bias must have the width of x")
+    if out is not None:
+        _need(out, "out"); _need(next_weight, "next_weight", torch.float32)
+        if out.shape != x.shape or next_weight.numel() != W:
+            raise KernelError("rmsnorm_add_norm: the next norm's sizes differ")
+    _ok(kernels().ce_rmsnorm_add_norm(_ptr(y), _ptr(bias), _ptr(weight), _ptr(x), _ptr(next_weight), _ptr(out),
+                                      F32 if out is None else dtype_code(out.dtype), T, W, float(eps), float(next_eps), _stream()))
 
 
 def tanh_cap(x: torch.Tensor, cap: float) -> None:
@@ -325,7 +378,8 @@ def value_mix(rows: torch.Tensor, off: int, n: int, first: torch.Tensor, first_o
 
 
 def latent_prepare(proj, wq, wkv, cq, k_pool, cos, sin, positions, seq_of_token, seq_slot, block_table, status, off_q: int,
-                   qr: int, off_kv: int, r: int, dr: int, rd: int, page_size: int, eps: float, write_kv: bool = True) -> None:
+                   qr: int, off_kv: int, r: int, dr: int, rd: int, page_size: int, eps: float, write_kv: bool = True,
+                   pairing: str = "half") -> None:
     """Latent attention's operands from one float32 product row: cq = rms_norm(query latent) * wq; the token's
     cache row [rms_norm(latent) * wkv | rotated key part] into ``k_pool`` [pages, 1, page, r + dr]."""
     _need(proj, "proj", torch.float32)
@@ -345,17 +399,19 @@ def latent_prepare(proj, wq, wkv, cq, k_pool, cos, sin, positions, seq_of_token,
         _ptr(seq_of_token), _ptr(seq_slot), _ptr(block_table), _ptr(status), proj.shape[0], proj.stride(0), int(off_q), int(qr),
         int(off_kv), int(r), int(dr), int(rd), int(page_size), block_table.shape[1] if block_table is not None else 0,
         k_pool.shape[0] if k_pool is not None else 0, cos.shape[0] if cos is not None else 0, 1 if write_kv else 0, float(eps),
-        _stream()))
+        ROPE_PAIRINGS[pairing], _stream()))
 
 
 def rope_part(src, src_head: int, src_off: int, dst, dst_head: int, dst_off: int, cos, sin, positions, status, heads: int,
-              dr: int, rd: int) -> None:
-    """dst[t, h*dst_head + dst_off + i] = src[t, h*src_head + src_off + i] for i < dr, its first rd elements rotated in half pairs."""
+              dr: int, rd: int, pairing: str = "half") -> None:
+    """dst[t, h*dst_head + dst_off + i] = src[t, h*src_head + src_off + i] for i < dr, its first rd elements rotated (``pairing``:
+    i with i + rd/2, or 2i with 2i + 1)."""
     if src.dtype != dst.dtype or src.stride(-1) != 1 or dst.stride(-1) != 1:
         raise KernelError("rope_part: rows of one dtype are needed")
     _ok(kernels().ce_rope_part(_ptr(src), src.stride(0), int(src_head), int(src_off), _ptr(dst), dst.stride(0), int(dst_head),
                                int(dst_off), dtype_code(src.dtype), _ptr(cos), _ptr(sin), _ptr(positions), _ptr(status),
-                               src.shape[0], int(heads), int(dr), int(rd), cos.shape[0] if cos is not None else 0, _stream()))
+                               src.shape[0], int(heads), int(dr), int(rd), cos.shape[0] if cos is not None else 0, ROPE_PAIRINGS[pairing],
+                               _stream()))
 
 
 def head_matmul(inp, in_head: int, w, out, out_head: int, heads: int, n: int, k: int, gate=None, gate_per_head: bool = False) -> None:
@@ -453,55 +509,80 @@ def norm_rope_kvwrite(proj, q_out, k_pool, v_pool, wq, wk, head_scale, cos, sin,
         cos.shape[0] if cos is not None else 0, 1 if write_kv else 0, float(eps), _stream()))
 
 
-def gated_delta_prep_width(heads: int, key_heads: int, d: int, dv: int) -> int:
-    return kernels().ce_gated_delta_prep_width(heads, key_heads, d, dv)
-
-
-DECAY_PER_CHANNEL, DECAY_PER_HEAD, DECAY_CONSTANT = 0, 1, 2
+DECAY_PER_CHANNEL, DECAY_PER_HEAD, DECAY_CONSTANT, DECAY_EXP_GATES = 0, 1, 2, 3
 GATE_SIGMOID, GATE_SILU = 0, 1
+#: what becomes of q, k and v: short convolution, SiLU, unit q and k; rotated by the position; convolution and SiLU only; as projected
+OPERANDS_UNIT, OPERANDS_ROTATED, OPERANDS_CONV, OPERANDS_PLAIN = 0, 1, 2, 3
+
+
+def gated_delta_prep_width(heads: int, key_heads: int, d: int, dv: int, decay: int = DECAY_PER_CHANNEL) -> int:
+    return kernels().ce_gated_delta_prep_width(heads, key_heads, d, dv, int(decay))
 
 
 def gated_delta(proj, dec, gz, taps, a_log, dt_bias, norm_w, prep, raw, state, kept, out, seq_of_token, seq_slot, q_start,
                 n_seqs: int, off_conv: int, off_b: int, heads: int, key_heads: int, d: int, dv: int, n_taps: int, eps: float,
                 decay: int = DECAY_PER_CHANNEL, gate: int = GATE_SIGMOID, delta: bool = True, out_scale: float = 1.0,
-                rotation=None) -> None:
+                rotation=None, operands: Optional[int] = None, conv_bias=None, write_step: bool = False, skip=None, m_state=None,
+                cap: float = 0.0, normalizer: bool = False, norm_parts: int = 0) -> None:
     """The recurrent mixers with a matrix state per head over each sequence's tokens of the step, from and to ``state``
     [slots, heads, d, dv] (float32).  ``proj`` float32 [T, ld] holds q | k | v from ``off_conv`` and the beta logits at
     ``off_b``; ``gz`` the gate logits [T, heads * dv] (rows of any stride).
 
-    ``delta``: the gated delta rule (True) or the plain decaying sum of outer products, which writes v itself (False).
+    ``delta``: the gated delta rule (True) or the plain decaying sum of outer products, which writes beta v itself (False).
     ``decay``: per head and key channel from logits ``dec`` [T, heads * d] with ``dt_bias`` [heads * d]; per head from
-    logits ``dec`` [T, heads] with ``dt_bias`` [heads]; or constant, ``a_log`` then holding the heads' decays themselves.
-    ``rotation`` None: q, k, v pass the short convolution (``taps`` [C, n_taps], the kept rows ``kept`` [slots, taps - 1, C])
-    and SiLU, and q and k become unit vectors; ``rotation`` = (cos, sin, rotary_dim, positions, status): no convolution, q and
-    k are rotated by the position and k is multiplied by d^-1/2 (with constant decays).  ``gate``: sigmoid or SiLU of the
-    gate logits; ``norm_w`` None: no weight after the root mean square; ``out_scale`` multiplies what is stored.
-    Four launches: prepare, keep, walk, finish."""
+    logits ``dec`` [T, heads] with ``dt_bias`` [heads]; constant, ``a_log`` then holding the heads' decays themselves; or
+    exponential gates: ``dec`` [T, 2 heads] the input gates' logits, then the forget gates', ``dt_bias`` their biases,
+    ``cap`` the bound of both, ``m_state`` [slots, heads] the running maximum (``a_log`` None).
+    ``operands`` (OPERANDS_*): the short convolution (``taps`` [C, n_taps], ``conv_bias`` [C] or None, the kept rows ``kept``
+    [slots, taps - 1, C]) and SiLU with or without unit q and k; ``rotation`` = (cos, sin, rotary_dim, positions, status): no
+    convolution, q and k rotated by the position and k times d^-1/2 (with constant decays); as projected, q times d^-1/2 (with
+    exponential gates).  None: by ``rotation``.
+    ``write_step``: beta is the step size, softplus of the decay's logits with their bias, instead of a sigmoid.
+    ``normalizer``: the state [slots, heads, d * (dv + 1)] also carries the decayed sum of the keys, and a head's output is
+    divided by max(|its read-out|, exp(-m)) + 1e-6.
+    ``gate``: sigmoid or SiLU of the gate logits; ``norm_w`` of size dv, of size heads * dv, or None: no weight after the root
+    mean square; ``norm_parts`` > 0: ``skip`` [heads] times v is added, the gate comes first and the root mean square is
+    taken in that many equal parts of all heads' values; ``out_scale`` multiplies what is stored.
+    Launches: prepare, keep or scan (not in a step of single tokens), walk, finish."""
     _need(state, "state", torch.float32); _need(out, "out")
-    for name, t in (("taps", taps), ("a_log", a_log), ("dt_bias", dt_bias), ("norm_w", norm_w), ("prep", prep), ("raw", raw)):
+    for name, t in (("taps", taps), ("a_log", a_log), ("dt_bias", dt_bias), ("norm_w", norm_w), ("prep", prep), ("raw", raw),
+                    ("conv_bias", conv_bias), ("skip", skip), ("m_state", m_state)):
         if t is not None:
             _need(t, name, torch.float32)
     for name, t in (("proj", proj), ("dec", dec), ("gz", gz)):
         if t is not None and (t.dtype != torch.float32 or t.stride(-1) != 1 or not t.is_cuda):
             raise KernelError(f"gated_delta: {name} must be float32 rows on the GPU")
+    if operands is None:
+        operands = OPERANDS_UNIT if rotation is None else OPERANDS_ROTATED
+    if (operands == OPERANDS_ROTATED) != (rotation is not None):
+        raise KernelError("gated_delta: rotated operands come with a rotation")
     T, C = out.shape[0], 2 * key_heads * d + heads * dv
-    P = gated_delta_prep_width(heads, key_heads, d, dv)
-    n_dec = {DECAY_PER_CHANNEL: heads * d, DECAY_PER_HEAD: heads}.get(decay)
-    if tuple(state.shape[1:]) != (heads, d, dv) or out.shape[1] != heads * dv or tuple(gz.shape) != (T, heads * dv) or \
-            prep.numel() < T * P or raw.numel() < T * heads * dv or a_log.numel() != heads or \
-            (norm_w is not None and norm_w.numel() != dv):
+    P = gated_delta_prep_width(heads, key_heads, d, dv, decay)
+    ones = 1 if normalizer else 0
+    n_dec = {DECAY_PER_CHANNEL: heads * d, DECAY_PER_HEAD: heads, DECAY_EXP_GATES: 2 * heads}.get(decay)
+    if state[0].numel() != heads * d * (dv + ones) or state.shape[1] != heads or out.shape[1] != heads * dv or \
+            tuple(gz.shape) != (T, heads * dv) or prep.numel() < T * P or raw.numel() < T * heads * (dv + ones) or \
+            (decay != DECAY_EXP_GATES and a_log.numel() != heads) or (norm_w is not None and norm_w.numel() not in (dv, heads * dv)):
         raise KernelError("gated_delta: sizes do not fit")
     if n_dec is not None and (dec is None or tuple(dec.shape) != (T, n_dec) or dt_bias is None or dt_bias.numel() != n_dec):
         raise KernelError("gated_delta: the decay's logits or bias do not fit")
+    if decay == DECAY_EXP_GATES and (m_state is None or m_state.shape != (state.shape[0], heads)):
+        raise KernelError("gated_delta: the running maximum does not fit")
+    if norm_parts > 0 and norm_w is not None and norm_w.numel() != heads * dv:
+        raise KernelError("gated_delta: a norm in parts has a weight of all heads' size")
+    if (conv_bias is not None and conv_bias.numel() != C) or (skip is not None and skip.numel() != heads):
+        raise KernelError("gated_delta: the convolution's bias or the skip weights do not fit")
     cos = sin = positions = status = None
     rd = max_pos = 0
-    if rotation is None:
+    if operands in (OPERANDS_UNIT, OPERANDS_CONV):
         if tuple(taps.shape) != (C, n_taps) or (n_taps > 1 and tuple(kept.shape[1:]) != (n_taps - 1, C)):
             raise KernelError("gated_delta: the convolution's sizes do not fit")
-    else:
+    elif n_taps != 1:
+        raise KernelError("gated_delta: these operands come without a convolution")
+    if rotation is not None:
         cos, sin, rd, positions, status = rotation
-        if n_taps != 1 or decay != DECAY_CONSTANT:
-            raise KernelError("gated_delta: rotated operands come without a convolution and with constant decays")
+        if decay != DECAY_CONSTANT:
+            raise KernelError("gated_delta: rotated operands come with constant decays")
         if cos is not None:
             _need(cos, "cos", torch.float32); _need(sin, "sin", torch.float32)
             if cos.shape[1] != rd // 2:
@@ -512,8 +593,9 @@ def gated_delta(proj, dec, gz, taps, a_log, dt_bias, norm_w, prep, raw, state, k
     prof, work = profiling(), None
     if prof is not None:
         work, prof._work = prof._work, (0, 0)            # the caller's figures belong to the walk
+    norm_all = 1 if norm_w is not None and norm_w.numel() == heads * dv and heads > 1 else 0
     for stage in (1, 2, 3, 4):
-        if stage == 2 and n_taps == 1:
+        if stage == 2 and (T == n_seqs or (n_taps == 1 and decay != DECAY_EXP_GATES)):
             continue
         if stage == 3 and work is not None:
             prof.note_work(*work)
@@ -521,9 +603,10 @@ def gated_delta(proj, dec, gz, taps, a_log, dt_bias, norm_w, prep, raw, state, k
                                      _ptr(prep), _ptr(raw), _ptr(state), _ptr(kept), _ptr(out), dtype_code(out.dtype),
                                      _ptr(seq_of_token), _ptr(seq_slot), _ptr(q_start), T, n_seqs, proj.stride(0), int(off_conv),
                                      int(off_b), heads, key_heads, d, dv, n_taps, float(eps),
-                                     dec.stride(0) if dec is not None else 0, gz.stride(0), int(decay), 0 if rotation is None else 1,
+                                     dec.stride(0) if dec is not None else 0, gz.stride(0), int(decay), int(operands),
                                      0 if delta else 1, int(gate), float(out_scale), _ptr(cos), _ptr(sin), _ptr(positions),
-                                     _ptr(status), int(rd), int(max_pos), stage, _stream()))
+                                     _ptr(status), int(rd), int(max_pos), _ptr(conv_bias), _ptr(skip), _ptr(m_state), float(cap),
+                                     1 if write_step else 0, ones, norm_all, int(norm_parts), stage, _stream()))
 
 
 def attention_generic(q, q_stride: int, k_pool, v_pool, out, positions, seq_of_token, seq_slot, block_table,
@@ -539,7 +622,7 @@ def attention_generic(q, q_stride: int, k_pool, v_pool, out, positions, seq_of_t
         k_pool.shape[0], int(window), float(scale), _stream()))
 
 
-def gemm_plain(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, mode: int) -> None:
+def gemm_plain(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, mode: int, glu: Optional[GluParams] = None) -> None:
     """c = a @ w.T with float32 FMA arithmetic; see csrc/kernels/gemm_plain.cu for the epilogues."""
     _need(w, "w", a.dtype); _need(c, "c")
     if a.stride(-1) != 1 or c.stride(-1) != 1:
@@ -552,8 +635,9 @@ def gemm_plain(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, mode: int) -> 
     want = torch.float32 if mode in (GEMM_STORE_F32, GEMM_ACCUM_F32) else a.dtype
     if c.dtype != want:
         raise KernelError(f"gemm_plain: output must be {want}")
+    bias, limit, alpha = glu_args(glu, mode, N)
     _ok(kernels().ce_gemm_plain(_ptr(a), _ptr(w), _ptr(c), dtype_code(a.dtype), M, N, K, a.stride(0), c.stride(0),
-                                mode, _stream()))
+                                mode, bias, limit, alpha, _stream()))
 
 
 def streams_norm(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, eps: float, groups: int = 1,
@@ -723,21 +807,31 @@ def general_delta(proj, zz, w0, a_bias, norm_w, prep, raw, state, out, seq_slot,
                                        proj.stride(0), off_r, off_k, off_v, off_a, off_g, heads, d, float(eps), stage, _stream()))
 
 
-MOE_ACTIVATIONS = {"none": 0, "relu2": 1}
+#: "clamped_glu": an expert's rows are gate and up rows by turns (2j the gate of feature j, 2j + 1 its up); one output a pair
+MOE_ACTIVATIONS = {"none": 0, "relu2": 1, "clamped_glu": 2}
+MOE_SCORES = {"softmax": 0, "sigmoid": 1}
+MOE_GROUP_SCORES = {"max": 0, "top2": 1}
 
 
 def moe_route(z: torch.Tensor, experts: int, top: int, groups: int, keep: int, scale: float, ids: torch.Tensor,
-              weights: torch.Tensor, sgate: Optional[torch.Tensor] = None) -> None:
+              weights: torch.Tensor, sgate: Optional[torch.Tensor] = None, scoring: str = "softmax",
+              correction: Optional[torch.Tensor] = None, group_score: str = "max", renormalize: bool = True) -> None:
     """Router logits z [T, >= experts (+1)] float32 -> the ``top`` experts of every token (``ids`` int32 [T, top], best
-    first) and their weights (float32 [T, top]): softmax over the experts, experts in ``groups`` equal groups of neighbours
-    of which the ``keep`` with the largest member stay eligible, weights = chosen scores / their sum * scale.  With
-    ``sgate`` (float32 [T]) column ``experts`` of z is a gate logit: sgate = sigmoid of it."""
+    first) and their weights (float32 [T, top]): scores s = softmax over the experts or sigmoid, choice scores s +
+    ``correction`` (float32 [experts]), experts in ``groups`` equal groups of neighbours of which the ``keep`` with the
+    largest member (or, "top2", the largest sum of two members) stay eligible, weights = chosen s / their sum * scale, or s *
+    scale without ``renormalize``.  With ``sgate`` (float32 [T]) column ``experts`` of z is a gate logit: sgate = sigmoid of it."""
     _need(z, "z", torch.float32); _need(ids, "ids", torch.int32); _need(weights, "weights", torch.float32)
     T = z.shape[0]
     if ids.shape != (T, top) or weights.shape != (T, top) or (sgate is not None and (sgate.dtype != torch.float32 or sgate.numel() != T)):
         raise KernelError("moe_route: sizes do not fit")
+    if correction is not None:
+        _need(correction, "correction", torch.float32)
+        if correction.numel() != experts:
+            raise KernelError("moe_route: one correction per expert")
     _ok(kernels().ce_moe_route(_ptr(z), _ptr(ids), _ptr(weights), _ptr(sgate), T, z.stride(0), int(experts), int(top), int(groups),
-                               int(keep), float(scale), _stream()))
+                               int(keep), float(scale), _ptr(correction), MOE_SCORES[scoring], MOE_GROUP_SCORES[group_score],
+                               1 if renormalize else 0, _stream()))
 
 
 def moe_max_tiles(n_pairs: int, experts: int, tile: int) -> int:
@@ -759,12 +853,14 @@ def moe_align(ids: torch.Tensor, experts: int, tile: int, row_token: torch.Tenso
 
 
 def moe_matmul(inp: torch.Tensor, w: torch.Tensor, out: torch.Tensor, tile: int, activation: str = "none", row_token=None,
-               tile_expert=None, n_tiles=None) -> None:
+               tile_expert=None, n_tiles=None, limit: float = 0.0, alpha: float = 0.0) -> None:
     """out[p] = act(inp[row_token[p]] @ w[tile_expert[p // tile]].T) for the rows of the layout's tiles (``row_token``
     None: the input rows are the layout's rows already).  Without any table: out = act(inp @ w[0].T), row by row.
-    w [experts, N, K]; operands and output in one dtype."""
+    w [experts, N, K]; operands and output in one dtype.  "clamped_glu" (``limit``, ``alpha``): rows 2j and 2j + 1 of an expert
+    are feature j's gate and up, and ``out`` has N / 2 columns."""
     _need(w, "w", inp.dtype); _need(out, "out", inp.dtype)
-    if inp.stride(-1) != 1 or w.dim() != 3 or inp.shape[1] != w.shape[2] or out.shape[1] != w.shape[1]:
+    per = 2 if activation == "clamped_glu" else 1
+    if inp.stride(-1) != 1 or w.dim() != 3 or inp.shape[1] != w.shape[2] or out.shape[1] * per != w.shape[1]:
         raise KernelError("moe_matmul: shapes do not fit")
     if tile_expert is None:
         rows = inp.shape[0]
@@ -785,7 +881,7 @@ def moe_matmul(inp: torch.Tensor, w: torch.Tensor, out: torch.Tensor, tile: int,
                        2 * n_rows * w.shape[1] * w.shape[2])
     _ok(kernels().ce_moe_matmul(_ptr(inp), _ptr(w), _ptr(out), _ptr(row_token), _ptr(tile_expert), _ptr(n_tiles), dtype_code(inp.dtype),
                                 tiles, int(tile), w.shape[1], w.shape[2], inp.stride(0), out.stride(0), MOE_ACTIVATIONS[activation],
-                                rows, _stream()))
+                                float(limit), float(alpha), rows, _stream()))
 
 
 def moe_gather(inp: torch.Tensor, row_token: torch.Tensor, n_tiles: torch.Tensor, tile: int, out: torch.Tensor) -> None:

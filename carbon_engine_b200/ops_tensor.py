@@ -27,11 +27,11 @@ kernel_lib.declare("ce_attention_prefill_bf16_sink", _i, [_p] * 11 + [_i] * 9 + 
 kernel_lib.declare("ce_gemm_tc_supported", _i, [_i, _i, _i, _i])
 kernel_lib.declare("ce_gemm_tc_scratch", _ll, [_i, _i, _i, _i])
 kernel_lib.declare("ce_gemm_tc_splits", _i, [_i, _i, _i])
-# A, W, C, M, N, K, lda, ldc, mode, scratch, scratch_floats, counters, n_counters, status, stream
-kernel_lib.declare("ce_gemm_tc", _i, [_p, _p, _p, _i, _i, _i, _i, _i, _i, _p, _ll, _p, _i, _p, _p])
+# A, W, C, M, N, K, lda, ldc, mode, scratch, scratch_floats, counters, n_counters, status, bias, limit, alpha, stream
+kernel_lib.declare("ce_gemm_tc", _i, [_p, _p, _p, _i, _i, _i, _i, _i, _i, _p, _ll, _p, _i, _p, _p, _f, _f, _p])
 kernel_lib.declare("ce_gemm_tc_grouped_supported", _i, [_i, _i, _i, _i, _i])
-# x, W, out, tile_expert, n_tiles, max_tiles, tile, experts, N, K, ldi, ldo, x_rows, rows, act, status, stream
-kernel_lib.declare("ce_gemm_tc_grouped", _i, [_p] * 5 + [_i] * 10 + [_p, _p])
+# x, W, out, tile_expert, n_tiles, max_tiles, tile, experts, N, K, ldi, ldo, x_rows, rows, act, limit, alpha, status, stream
+kernel_lib.declare("ce_gemm_tc_grouped", _i, [_p] * 5 + [_i] * 10 + [_f, _f, _p, _p])
 
 
 def decode_split() -> int:
@@ -88,8 +88,9 @@ def gemm_status(device) -> int:
     return 0 if ws is None else int(ws.status.item())
 
 
-def gemm_bf16(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, mode: int) -> bool:
-    """out (op)= a @ w.T on the tcgen05 kernel; False if the shape is refused."""
+def gemm_bf16(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, mode: int, glu=None) -> bool:
+    """out (op)= a @ w.T on the tcgen05 kernel; False if the shape is refused.  ``glu``: what the clamped gated epilogue needs
+    (``ops.GluParams``)."""
     if not USE_TENSOR_GEMM or a.dtype != torch.bfloat16:
         return False
     M, K = a.shape
@@ -99,13 +100,14 @@ def gemm_bf16(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, mode: int) ->
         return False
     if not k.ce_gemm_tc_supported(M, N, K, a.stride(0)) or (a.data_ptr() | w.data_ptr()) & 15:
         return False
+    bias, limit, alpha = ops.glu_args(glu, mode, N)
     need = k.ce_gemm_tc_scratch(M, N, K, mode)
     ws = gemm_workspace(a.device)
     if need > ws.scratch.numel():
         return False
     ops._ok(k.ce_gemm_tc(a.data_ptr(), w.data_ptr(), out.data_ptr(), M, N, K, a.stride(0), out.stride(0), mode,
                          ws.scratch.data_ptr(), ws.scratch.numel(), ws.counters.data_ptr(), ws.counters.numel(),
-                         ws.status.data_ptr(), ops._stream()))
+                         ws.status.data_ptr(), bias, limit, alpha, ops._stream()))
     return True
 
 
@@ -114,9 +116,11 @@ def grouped_bf16_supported(tile: int, n: int, k: int, ldi: int, ldo: int, dtype)
     return USE_TENSOR_GEMM and dtype == torch.bfloat16 and bool(kernels().ce_gemm_tc_grouped_supported(tile, n, k, ldi, ldo))
 
 
-def grouped_bf16(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, tile: int, act: int, tile_expert=None, n_tiles=None) -> bool:
+def grouped_bf16(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, tile: int, act: int, tile_expert=None, n_tiles=None,
+                 limit: float = 0.0, alpha: float = 0.0) -> bool:
     """out[p] = act(x[p] @ w[tile_expert[p // tile]].T) over a layout by expert on the tcgen05 kernel (w [experts, N, K]; x
-    already in the layout's order), or, without the tables, out = act(x @ w[0].T); False if the shape is refused."""
+    already in the layout's order), or, without the tables, out = act(x @ w[0].T); False if the shape is refused.  ``act``, ``limit``,
+    ``alpha`` as in :func:`ops.moe_matmul`."""
     if x.dim() != 2 or x.stride(1) != 1 or out.stride(1) != 1 or not w.is_contiguous() or w.dtype != x.dtype or out.dtype != x.dtype:
         return False
     E, N, K = w.shape
@@ -138,7 +142,7 @@ def grouped_bf16(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, tile: int,
         prof.note_work((rows * (N + K) + live * N * K) * 2, 2 * rows * N * K)
     ws = gemm_workspace(x.device)
     ops._ok(kernels().ce_gemm_tc_grouped(x.data_ptr(), w.data_ptr(), out.data_ptr(), ops._ptr(tile_expert), ops._ptr(n_tiles), tiles,
-                                         tile, E, N, K, x.stride(0), out.stride(0), x.shape[0], rows, act, ws.status.data_ptr(),
+                                         tile, E, N, K, x.stride(0), out.stride(0), x.shape[0], rows, act, float(limit), float(alpha), ws.status.data_ptr(),
                                          ops._stream()))
     return True
 

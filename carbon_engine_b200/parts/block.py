@@ -1,6 +1,6 @@
 """Arrangements of parts in a layer.  Pre-norm: x += mixer(norm1(x)); x += ffn(norm2(x))
-(src/model/mod.rs:645-650).  Output-norm: x += norm1(mixer(x)); x += norm2(ffn(x)).  Parallel: h = norm1(x);
-x += mixer(h) + ffn(h)."""
+(src/model/mod.rs:645-650).  Output-norm: x += norm1(mixer(x)); x += norm2(ffn(x)).  Sandwich-norm:
+x += norm1b(mixer(norm1(x))); x += norm2b(ffn(norm2(x))).  Parallel: h = norm1(x); x += mixer(h) + ffn(h)."""
 from __future__ import annotations
 
 from typing import List, Optional
@@ -9,6 +9,7 @@ import torch
 
 from .. import ops
 from .base import Block, BundleCacheSpec, FeedForward, Mixer, Norm, Part
+from .norm import RMSNorm
 
 
 class PreNormBlock(Block):
@@ -121,6 +122,66 @@ class OutputNormBlock(Block):
         if owed is not None:
             ops.add_bias(y, owed)
         self._add(ctx, self.ffn_norm, y, x)
+
+
+class SandwichNormBlock(Block):
+    """A norm in front of each sublayer and another on its OUTPUT: x += mixer_out(mixer(mixer_norm(x))); x += ffn_out(ffn(ffn_norm(x))).
+    The sublayers STORE their result in a float32 buffer (``can_store``); one kernel adds the normed result (and a bias the
+    sublayer still owes) into the residual and takes the norm that comes next: this block's ``ffn_norm``, or the norm in front of
+    the next layer run (``ctx.next_norm``), whose block finds its input ready.  The norms are RMS norms.  ``ffn`` None: the layer has only the
+    mixer."""
+
+    #: what the last kernel left in ``ctx.shared``: (the norm it took, of which residual, its output)
+    NORMED = "residual.normed"
+
+    def __init__(self, width: int, mixer_norm: RMSNorm, mixer: Mixer, mixer_out: RMSNorm, ffn_norm: Optional[RMSNorm] = None,
+                 ffn: Optional[FeedForward] = None, ffn_out: Optional[RMSNorm] = None):
+        if len({ffn is None, ffn_norm is None, ffn_out is None}) != 1:
+            raise ValueError("a feed-forward and its two norms come together")
+        for part in (mixer, ffn):
+            if part is not None and not getattr(part, "can_store", False):
+                raise ValueError(f"{type(part).__name__} cannot store its output, which a norm on the output needs")
+        for norm in (mixer_norm, mixer_out, ffn_norm, ffn_out):
+            if norm is not None and not isinstance(norm, RMSNorm):
+                raise ValueError(f"{type(norm).__name__}: this block's norms are RMS norms")
+        self.width, self.mixer, self.ffn = int(width), mixer, ffn
+        self.mixer_norm, self.mixer_out, self.ffn_norm, self.ffn_out = mixer_norm, mixer_out, ffn_norm, ffn_out
+
+    @property
+    def leading_norm(self) -> Norm:
+        return self.mixer_norm
+
+    def children(self) -> List[Part]:
+        return [p for p in (self.mixer_norm, self.mixer, self.mixer_out, self.ffn_norm, self.ffn, self.ffn_out) if p is not None]
+
+    def step_bytes(self, tokens: int, element_size: int) -> int:
+        ffn = self.ffn.step_bytes(tokens, element_size) if self.ffn is not None else 0
+        return tokens * self.width * (2 * element_size + 4) + max(self.mixer.step_bytes(tokens, element_size), ffn)
+
+    def _read(self, ctx, norm: RMSNorm, x: torch.Tensor) -> torch.Tensor:
+        left = ctx.shared.pop(self.NORMED, None)
+        if left is not None and left[0] is norm and left[1] == x.data_ptr() and left[2].shape == x.shape:
+            return left[2]
+        h = ctx.buffer(tuple(x.shape))
+        norm.forward(x, h)
+        return h
+
+    def _add(self, ctx, norm: RMSNorm, y: torch.Tensor, owed: Optional[torch.Tensor], x: torch.Tensor, following: Optional[Norm]) -> None:
+        if not isinstance(following, RMSNorm):
+            ops.rmsnorm_add_norm(y, norm.weight, x, norm.eps, owed)
+            return
+        h = ctx.buffer(tuple(x.shape))
+        ops.rmsnorm_add_norm(y, norm.weight, x, norm.eps, owed, following.weight, following.eps, h)
+        ctx.shared[self.NORMED] = (following, x.data_ptr(), h)
+
+    def forward(self, ctx, x: torch.Tensor, cache) -> None:
+        y = ctx.buffer(tuple(x.shape), torch.float32)
+        owed = self.mixer.forward(ctx, self._read(ctx, self.mixer_norm, x), y, cache, accumulate=False)
+        self._add(ctx, self.mixer_out, y, owed, x, self.ffn_norm if self.ffn is not None else ctx.next_norm)
+        if self.ffn is None:
+            return
+        owed = self.ffn.forward(ctx, self._read(ctx, self.ffn_norm, x), y, accumulate=False)
+        self._add(ctx, self.ffn_out, y, owed, x, ctx.next_norm)
 
 
 class StreamBlock(Block):

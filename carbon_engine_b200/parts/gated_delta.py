@@ -14,7 +14,7 @@ multiplied by a weight of size vdim that the heads share and by sigmoid(W_g2 (W_
 
 Kept per request: the state [heads, dim, vdim] and the convolution's last ``taps - 1`` inputs, both float32 in both
 precisions.  One product gives q | k | v | beta | a1 | g1 in float32; the two narrow second products are ordinary
-``Linear``s; then four kernels (csrc/kernels/gated_delta.cu): prepare, keep, walk, finish.
+``Linear``s; then the kernels of csrc/kernels/gated_delta.cu: prepare, keep, walk, finish.
 
 With one decay per head, g_t = exp(-exp(A_h) softplus(W_a h + bias_h)) multiplies every row of the head's state alike, and
 the gate is an activation (SiLU or sigmoid) of a projection of full rank: one product gives q | k | v | beta | a | g.
@@ -162,7 +162,7 @@ class HeadGatedDelta(Mixer):
 
     def step_bytes(self, tokens: int, element_size: int) -> int:
         H, d, dv = self.heads, self.dim, self.vdim
-        prep = self.channels + H * d + H + 3
+        prep = self.channels + 2 * H + 3
         return tokens * ((self.inp.padded_out + prep + H * dv) * 4 + H * dv * element_size)
 
     def forward(self, ctx, h: torch.Tensor, x: torch.Tensor, cache, accumulate: bool = True) -> None:
@@ -172,7 +172,7 @@ class HeadGatedDelta(Mixer):
         self.inp.forward(h, proj, STORE_F32)
         off_b = self.channels
         dec, gz = proj[:, off_b + H:off_b + 2 * H], proj[:, off_b + 2 * H:off_b + 2 * H + H * dv]
-        prep = ctx.buffer((T, ops.gated_delta_prep_width(H, G, d, dv)), torch.float32)
+        prep = ctx.buffer((T, ops.gated_delta_prep_width(H, G, d, dv, ops.DECAY_PER_HEAD)), torch.float32)
         raw = ctx.buffer((T, H * dv), torch.float32)
         out = ctx.buffer((T, H * dv))
         prof = ops.profiling()

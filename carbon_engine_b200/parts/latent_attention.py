@@ -11,7 +11,8 @@ exponential joins the softmax's denominator without a key or a value (``sink``);
 instead of one per output element (``gate="head"``); a layer without a down-projection of its own that reads the rows
 another layer cached (``own_kv=False``: the model's schedule gives it that layer's cache, read-only).
 
-The rotation turns the first ``rotary_dim`` elements of the rotated parts in half pairs.  The keys and values of a
+The rotation turns the first ``rotary_dim`` elements of the rotated parts in the pairs its position encoding names (i with
+i + rotary_dim/2, or 2i with 2i + 1).  The keys and values of a
 head are never formed: with W_uk moved to the query side, <q_plain, W_uk c> = <W_uk^T q_plain, c>, so every head
 attends over the cached rows themselves with a query of size kv_rank + rot_dim, the weighted sum of the rows' latent
 parts comes out (size kv_rank), and W_uv is applied to that sum.  The two per-head products are one kernel each.
@@ -122,6 +123,7 @@ class LatentAttention(Mixer):
         cos = pos.cos if pos is not None else None
         sin = pos.sin if pos is not None else None
         rd = pos.rotary_dim if cos is not None else 0
+        pairing = pos.pairing if pos is not None else "half"
         if cos is not None and ctx.max_position >= cos.shape[0]:
             raise ValueError(f"position {ctx.max_position} is beyond the rotary table ({cos.shape[0]}): raise max_seq_len")
         if cache.writes and not self.own_kv:
@@ -135,12 +137,12 @@ class LatentAttention(Mixer):
         cq = ctx.buffer((T, qr)) if qr > 0 else None
         if qr > 0 or writes:
             ops.latent_prepare(proj, self.wq, self.wkv, cq, cache.k_pool, cos, sin, ctx.positions, ctx.seq_of_token, ctx.seq_slot,
-                               table, ctx.status, 0, qr, qr, r, dr, rd, cache.page_size, self.eps, write_kv=writes)
+                               table, ctx.status, 0, qr, qr, r, dr, rd, cache.page_size, self.eps, write_kv=writes, pairing=pairing)
         q = ctx.buffer((T, H * (d + dr)))
         self.uq.forward(cq if qr > 0 else h, q, STORE)
         qa = ctx.buffer((T, H * row))
         ops.head_matmul(q, d + dr, self.uk_t, qa, row, H, r, d)
-        ops.rope_part(q, d + dr, d, qa, row, r, cos, sin, ctx.positions, ctx.status, H, dr, rd)
+        ops.rope_part(q, d + dr, d, qa, row, r, cos, sin, ctx.positions, ctx.status, H, dr, rd, pairing)
         lat = ctx.buffer((T, H * r))
         attend(ctx, ctx.plans.get(self.plan_key), qa, row, cache, row, row, cache.k_pool, None, lat, table, H, 1, row, r,
                self.window, 0, self.scale, 0.0, self.sinks)

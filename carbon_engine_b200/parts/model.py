@@ -94,6 +94,9 @@ class DecoderModel(Part):
             ops.streams_broadcast(x, xs)
             x = xs
         for i, call in enumerate(self.schedule):
+            # the norm in front of the next call, which the last kernel of this one may take along
+            following = self.schedule[i + 1].block if i + 1 < len(self.schedule) else None
+            ctx.next_norm = getattr(self.blocks[following], "leading_norm", None) if following is not None else None
             self.blocks[call.block].forward(ctx, x, caches.view(call))
             if tap is not None:
                 tap(i, x)

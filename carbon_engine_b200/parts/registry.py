@@ -14,12 +14,14 @@ from .combine import SummedMixers
 from .gated_delta import ChannelGatedDelta, HeadGatedDelta
 from .latent_attention import LatentAttention
 from .masked_attention import GatedWindowAttention
+from .matrix_memory import MatrixMemory
 from .mlp import DenseMLP, GatedMLP
 from .moe import RoutedExperts
 from .norm import GroupedRMSNorm, LayerNorm, RMSNorm
 from .retention import Retention
 from .rope import NoPositionEncoding, RotaryEmbedding
 from .sink_attention import SinkAttention
+from .state_space import StateSpace
 
 _KINDS: Dict[str, Dict[str, Callable]] = {"mixer": {}, "feed_forward": {}, "norm": {}, "position": {}}
 
@@ -60,6 +62,8 @@ register_mixer("head_gated_delta", HeadGatedDelta)
 register_mixer("retention", Retention)
 register_mixer("sink_attention", SinkAttention)
 register_mixer("summed_mixers", SummedMixers)
+register_mixer("state_space", StateSpace)
+register_mixer("matrix_memory", MatrixMemory)
 register_feed_forward("gated_mlp", GatedMLP)
 register_feed_forward("dense_mlp", DenseMLP)
 register_feed_forward("routed_experts", RoutedExperts)

@@ -59,7 +59,7 @@ class Retention(Mixer):
 
     def step_bytes(self, tokens: int, element_size: int) -> int:
         H, d, dv = self.heads, self.dim, self.vdim
-        prep = 2 * H * d + H * dv + H * d + H + 3
+        prep = 2 * H * d + H * dv + 2 * H + 3
         return tokens * ((self.inp.padded_out + prep + H * dv) * 4 + H * dv * element_size)
 
     def forward(self, ctx, h: torch.Tensor, x: torch.Tensor, cache, accumulate: bool = True) -> None:
@@ -74,7 +74,7 @@ class Retention(Mixer):
         if cos is not None and ctx.max_position >= cos.shape[0]:
             raise ValueError(f"position {ctx.max_position} is beyond the rotary table ({cos.shape[0]}): raise max_seq_len")
         rotation = (cos, pos.sin if pos is not None else None, pos.rotary_dim if cos is not None else 0, ctx.positions, ctx.status)
-        prep = ctx.buffer((T, ops.gated_delta_prep_width(H, H, d, dv)), torch.float32)
+        prep = ctx.buffer((T, ops.gated_delta_prep_width(H, H, d, dv, ops.DECAY_CONSTANT)), torch.float32)
         raw = ctx.buffer((T, H * dv), torch.float32)
         out = ctx.buffer((T, H * dv))
         prof = ops.profiling()
