@@ -235,15 +235,38 @@ def pugozen_config(width, heads, kv_heads, ff, layers, vocab):
                                     "embedding": {"scale": float(width) ** 0.5}, "max_position_embeddings": 8192})
 
 
+def rapovik_config(width, heads, kv_heads, ff, layers, vocab):
+    """A Rapovik model of the usual proportions at the Qwen3 model's layer sizes: layers go state space (state heads of 128 x 128
+    filling the width, 1 group, 4 taps), matrix memory (state heads of 128 x 128), latent attention (heads of 128 + 32, values of
+    128, a cached row of 256 + 32 per token, a window of 1,024), state space again.  The feed-forward alternates between the dense
+    gated one and a mixture of 32 gated experts in 4 groups (2 kept), 4 per token, each an eighth of the dense width, beside a shared expert of
+    half the dense width: a token's products are as wide as the dense layer's.  No layer is looped."""
+    from carbon_engine_b200.config.rapovik import RapovikConfig
+    n = width // 128
+    ssm = {"type": "mamba2", "mixer": {"heads": n, "vdim": 128, "state": 128, "groups": 1, "conv": 4, "norm_groups": 1}}
+    memory = {"type": "mlstm", "mixer": {"heads": n, "dim": 128, "vdim": 128, "gate_cap": 15.0}}
+    latent = {"type": "latent_attention",
+              "mixer": {"heads": heads, "dim": 128, "rot_dim": 32, "vdim": 128, "kv_rank": 256, "scale": 160 ** -0.5,
+                        "rot": {"dims": 32, "base": 1e6}, "mask": {"size": 1024}}}
+    dense = {"kind": "dense", "ff": ff, "limit": 7.0}
+    moe = {"kind": "moe", "expert": {"ff": ff // 8, "limit": 7.0}, "shared": {"ff": ff // 2, "limit": 7.0},
+           "router": {"experts": 32, "top": 4, "groups": {"count": 4, "keep": 2}}}
+    kinds = (ssm, memory, latent, ssm)
+    return RapovikConfig.from_dict({"architecture": "Rapovik", "vocab": vocab, "width": width,
+                                    "layers": [dict(kinds[i % 4], mlp=dense if i % 2 == 0 else moe) for i in range(layers)],
+                                    "norm": {"eps": 1e-6}, "max_position_embeddings": 8192})
+
+
 def compare_designs(args, BenchHarness, pk) -> int:
-    """Prefill and decode throughput of the engine's other designs (--designs: munizen, lunerax, vamadra, pugozen) beside the Qwen3 dense
+    """Prefill and decode throughput of the engine's other designs (--designs: munizen, lunerax, vamadra, pugozen, rapovik) beside the Qwen3 dense
     design at equal layer sizes (random weights, a few layers), with the kernels of each and their distance from the roofline."""
     import torch
-    makers = {"munizen": munizen_config, "lunerax": lunerax_config, "vamadra": vamadra_config, "pugozen": pugozen_config}
+    makers = {"munizen": munizen_config, "lunerax": lunerax_config, "vamadra": vamadra_config, "pugozen": pugozen_config,
+              "rapovik": rapovik_config}
     designs = [x for x in args.designs.split(",") if x != "qwen3"]
     for x in designs:
         if x not in makers:
-            raise SystemExit(f"--designs {x}: munizen, lunerax, vamadra, pugozen and qwen3 are built")
+            raise SystemExit(f"--designs {x}: munizen, lunerax, vamadra, pugozen, rapovik and qwen3 are built")
     layers = args.layers if args.layers != SIZES_8B["num_hidden_layers"] else 4
     vocab, out = 32768, {}
     for name in args.sizes.split(","):
@@ -302,7 +325,7 @@ def main() -> int:
     ap.add_argument("--sizes", default="1b,8b", help="with --workload compare-designs: which of the layer sizes "
                     "1b, 4b, 8b (width / heads / feed-forward of models of about that size), with commas between them")
     ap.add_argument("--designs", default="munizen,qwen3", help="with --workload compare-designs: the designs set beside one another "
-                    "(munizen, lunerax, vamadra, pugozen; qwen3 is always the last)")
+                    "(munizen, lunerax, vamadra, pugozen, rapovik; qwen3 is always the last)")
     ap.add_argument("--workload", default="decode", choices=["decode", "mixed-14b", "batch16-32b", "compare-designs"],
                     help="decode: the headline line (default).  mixed-14b: 32 requests with prompts of 128 to 3,072 tokens at "
                          "Qwen3-14B sizes, prompts cut under a 2,048-token step budget beside the decoding requests, 128 new "
