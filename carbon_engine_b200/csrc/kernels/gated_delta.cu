@@ -194,54 +194,136 @@ __global__ void gated_delta_prepare_kernel(GatedDeltaArgs a) {
     }
 }
 
-// The running maximum of the exponential gates, token after token: a block per (sequence, 32 heads).  The chain is one addition
-// and one maximum a token; one warp walks it, a head a lane, over a chunk of tokens in shared memory, and all warps fetch the
-// chunk's gates before and take the exponentials after.
-#define GD_SCAN_TOKENS 64
+// The same for operands 2 (nothing couples the channels): a thread takes one channel of GD_CONV_TOKENS tokens, so that a token's input
+// is read once and not K times, and the channel's taps once for all of them.
+#define GD_CONV_TOKENS 8
+template <int K>
+__global__ void __launch_bounds__(256) gated_delta_conv_kernel(GatedDeltaArgs a, int T, int tile) {
+    ce_pdl_begin();
+    const int C = 2 * a.G * a.d + a.H * a.dv, H = a.H;
+    const int t0 = blockIdx.x * tile, nt = min(tile, T - t0), c = blockIdx.y * 256 + threadIdx.x;
+    const int b0 = a.seq_of_token[t0], rel0 = t0 - a.q_start[b0];
+    if (c < C) {
+        float w[K];
+#pragma unroll
+        for (int j = 0; j < K; ++j) w[j] = a.taps[(size_t)c * K + j];
+        const float bias = a.conv_bias ? a.conv_bias[c] : 0.f;
+        const float* in = a.proj + a.off_conv + c;
+        auto out = [&](int t, float y) { a.prep[(size_t)t * a.P + c] = y / (1.0f + expf(-y)); };
+        if (nt == GD_CONV_TOKENS && a.seq_of_token[t0 + nt - 1] == b0) {
+            const float* kept = a.kept + (size_t)a.seq_slot[b0] * (K - 1) * C + c;
+            float x[GD_CONV_TOKENS + K - 1];          // the tile's inputs, after the K - 1 before it
+#pragma unroll
+            for (int i = 0; i < K - 1; ++i)
+                x[i] = K - 1 - i <= rel0 ? in[(size_t)(t0 - (K - 1) + i) * a.ld] : kept[(size_t)(rel0 + i) * C];
+#pragma unroll
+            for (int i = 0; i < GD_CONV_TOKENS; ++i) x[K - 1 + i] = in[(size_t)(t0 + i) * a.ld];
+#pragma unroll
+            for (int i = 0; i < GD_CONV_TOKENS; ++i) {
+                float y = bias;
+#pragma unroll
+                for (int j = 0; j < K; ++j) y = fmaf(w[j], x[i + j], y);
+                out(t0 + i, y);
+            }
+        } else {
+            for (int t = t0; t < t0 + nt; ++t) {
+                const int b = a.seq_of_token[t], rel = t - a.q_start[b];
+                float* kept = a.kept + (size_t)a.seq_slot[b] * (K - 1) * C + c;
+                float y = bias, x[K];
+#pragma unroll
+                for (int j = 0; j < K; ++j) {
+                    const int back = K - 1 - j;
+                    x[j] = back <= rel ? in[(size_t)(t - back) * a.ld] : kept[(size_t)(K - 1 + rel - back) * C];
+                }
+#pragma unroll
+                for (int j = 0; j < K; ++j) y = fmaf(w[j], x[j], y);
+                if (a.single) {                       // the kept rows move up by one
+#pragma unroll
+                    for (int j = 1; j < K; ++j) kept[(size_t)(j - 1) * C] = x[j];
+                }
+                out(t, y);
+            }
+        }
+    }
+    if (blockIdx.y == gridDim.y - 1) {
+        for (int e = threadIdx.x; e < nt * H; e += 256) {
+            const int t = t0 + e / H, h = e % H;
+            float* gates = a.prep + (size_t)t * a.P + C;
+            float step = a.decay_mode == 1 ? gd_softplus(a.dec[(size_t)t * a.ld_dec + h] + a.dt_bias[h]) : 0.f;
+            gates[h] = a.decay_mode == 1 ? expf(-expf(a.a_log[h]) * step) : a.a_log[h];
+            gates[H + h] = a.write_mode == 1 ? step : gd_sigmoid(a.proj[(size_t)t * a.ld + a.off_b + h]);
+        }
+    }
+}
+
+// The running maximum of the exponential gates, token after token: a block per (sequence, 8 heads).  The chain is one addition
+// and one maximum a token; a lane per head walks it over a chunk of tokens in shared memory, 16 tokens' gates in registers at a
+// time, while all threads have the next chunk's gates on their way; all of them take the exponentials after.
+#define GD_SCAN_TOKENS 256
+#define GD_SCAN_HEADS 8
+#define GD_SCAN_RUN 16
 __global__ void __launch_bounds__(256) gated_delta_scan_kernel(GatedDeltaArgs a) {
     ce_pdl_begin();
-    __shared__ float fs[GD_SCAN_TOKENS][32], is[GD_SCAN_TOKENS][32], ms[GD_SCAN_TOKENS + 1][32];
-    int b = blockIdx.x, h0 = blockIdx.y * 32, tid = threadIdx.x, H = a.H;
+    __shared__ float fs[GD_SCAN_TOKENS][GD_SCAN_HEADS], is[GD_SCAN_TOKENS][GD_SCAN_HEADS], ms[GD_SCAN_TOKENS + 1][GD_SCAN_HEADS];
+    int b = blockIdx.x, h0 = blockIdx.y * GD_SCAN_HEADS, tid = threadIdx.x, H = a.H;
     int t_begin = a.q_start[b], n = a.q_start[b + 1] - t_begin;
     if (n <= 0) return;
     size_t off = (size_t)2 * a.G * a.d + (size_t)H * a.dv;
     float* m_state = a.m_state + (size_t)a.seq_slot[b] * H;
-    if (tid < 32) ms[0][tid] = h0 + tid < H ? m_state[h0 + tid] : 0.f;
+    const bool walks = tid < GD_SCAN_HEADS;
+    if (walks) ms[0][tid] = h0 + tid < H ? m_state[h0 + tid] : 0.f;
+    constexpr int STRIDE = 256 / GD_SCAN_HEADS, PER = GD_SCAN_TOKENS / STRIDE;
+    const int hh = tid % GD_SCAN_HEADS, tok0 = tid / GD_SCAN_HEADS;            // head hh of tokens tok0, tok0 + STRIDE, ...
+    const bool in = h0 + hh < H;
+    float* col = a.prep + (size_t)t_begin * a.P + off + h0 + hh;
+    float fr[PER], ir[PER];
+    auto fetch = [&](int c0) {
+#pragma unroll
+        for (int k = 0; k < PER; ++k) {
+            int tok = c0 + tok0 + STRIDE * k;
+            bool there = in && tok < n;
+            fr[k] = there ? col[(size_t)tok * a.P] : 0.f;
+            ir[k] = there ? col[(size_t)tok * a.P + H] : 0.f;
+        }
+    };
+    fetch(0);
     for (int c0 = 0; c0 < n; c0 += GD_SCAN_TOKENS) {
         int nt = min(GD_SCAN_TOKENS, n - c0);
-        for (int e = tid; e < nt * 32; e += 256) {
-            int tok = e >> 5, h = e & 31;
-            const float* g = a.prep + (size_t)(t_begin + c0 + tok) * a.P + off + h0 + h;
-            bool in = h0 + h < H;
-            fs[tok][h] = in ? g[0] : 0.f;
-            is[tok][h] = in ? g[H] : 0.f;
-        }
+#pragma unroll
+        for (int k = 0; k < PER; ++k) { fs[tok0 + STRIDE * k][hh] = fr[k]; is[tok0 + STRIDE * k][hh] = ir[k]; }
         __syncthreads();
-        if (tid < 32) {
+        fetch(c0 + GD_SCAN_TOKENS);
+        if (walks) {
             float m = ms[0][tid];
-#pragma unroll 8
-            for (int tok = 0; tok < nt; ++tok) {
-                m = fmaxf(__fadd_rn(fs[tok][tid], m), is[tok][tid]);
-                ms[tok + 1][tid] = m;
+            for (int k0 = 0; k0 < nt; k0 += GD_SCAN_RUN) {       // (tokens past nt walk on zeros and are not used)
+                float f[GD_SCAN_RUN], i[GD_SCAN_RUN];
+#pragma unroll
+                for (int k = 0; k < GD_SCAN_RUN; ++k) { f[k] = fs[k0 + k][tid]; i[k] = is[k0 + k][tid]; }
+#pragma unroll
+                for (int k = 0; k < GD_SCAN_RUN; ++k) {
+                    m = fmaxf(__fadd_rn(f[k], m), i[k]);
+                    ms[k0 + k + 1][tid] = m;
+                }
             }
         }
         __syncthreads();
-        for (int e = tid; e < nt * 32; e += 256) {
-            int tok = e >> 5, h = e & 31;
-            if (h0 + h >= H) continue;
-            float* g = a.prep + (size_t)(t_begin + c0 + tok) * a.P + off + h0 + h;
-            float m = ms[tok + 1][h], fm = __fadd_rn(fs[tok][h], ms[tok][h]);
+#pragma unroll
+        for (int k = 0; k < PER; ++k) {
+            int tok = tok0 + STRIDE * k;
+            if (!in || tok >= nt) continue;
+            float* g = col + (size_t)(c0 + tok) * a.P;
+            float m = ms[tok + 1][hh], fm = __fadd_rn(fs[tok][hh], ms[tok][hh]);
             g[0] = expf(__fsub_rn(fm, m));
-            g[H] = expf(__fsub_rn(is[tok][h], m));
+            g[H] = expf(__fsub_rn(is[tok][hh], m));
             g[2 * H] = m;
         }
         __syncthreads();
-        if (tid < 32) {
+        if (walks) {
             float m = ms[nt][tid];
             ms[0][tid] = m;
             if (c0 + nt >= n && h0 + tid < H) m_state[h0 + tid] = m;
         }
-        __syncthreads();
+        // (the next chunk's first barrier comes before ms[0] is read by anyone but its writer)
     }
 }
 
@@ -602,20 +684,20 @@ __global__ void gated_delta_finish_kernel(GatedDeltaArgs a) {
     const float* o = a.raw + (size_t)t * a.H * (dv + a.ones);
     const float* gz = a.gz + (size_t)t * a.ld_gz;
     for (int h = warp; h < a.H; h += nwarp) {
-        float den = 1.f;
+        float part = 1.f;                        // what the extra channel divides the head's output by, as its inverse
         if (a.ones) {
             float m = a.prep[(size_t)t * a.P + 2 * a.G * a.d + n + 2 * a.H + h];
-            den = fmaxf(fabsf(o[n + h]), expf(-m)) + 1e-6f;
+            part = 1.0f / (fmaxf(fabsf(o[n + h]), expf(-m)) + 1e-6f);
         }
         float ss = 0.f;
-        for (int c = lane; c < dv; c += 32) { float v = o[h * dv + c] / den; ss = fmaf(v, v, ss); }
+        for (int c = lane; c < dv; c += 32) { float v = o[h * dv + c] * part; ss = fmaf(v, v, ss); }
         for (int k = 16; k > 0; k >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, k);
         float inv = 1.0f / sqrtf(ss / (float)dv + a.eps);
         for (int c = lane; c < dv; c += 32) {
             int col = h * dv + c;
             float z = gz[col], g = gd_sigmoid(z);
             if (a.gate_act == 1) g *= z;
-            float y = o[col] / den * inv;
+            float y = o[col] * part * inv;
             if (a.norm_w) y *= a.norm_w[a.norm_all ? col : c];
             CeType<T>::store((T*)a.out + (size_t)t * n + col, y * g * a.out_scale);
         }
@@ -624,16 +706,48 @@ __global__ void gated_delta_finish_kernel(GatedDeltaArgs a) {
 
 // The other order (parts > 0): a block per (token, part) of all heads' values: y = (o + skip_h v) gate(z), divided by the part's
 // own root mean square, times the weight.
-template <typename T>
+template <typename T, bool VEC>
 __global__ void gated_delta_part_finish_kernel(GatedDeltaArgs a) {
     ce_pdl_begin();
-    extern __shared__ float gd_part_smem[];          // the part's values
+    extern __shared__ __align__(16) float gd_part_smem[];          // the part's values
     __shared__ float scratch[32];
     int t = blockIdx.x, n = a.H * a.dv, size = n / a.parts, c0 = blockIdx.y * size;
     const float* o = a.raw + (size_t)t * n;
     const float* v = a.prep + (size_t)t * a.P + 2 * a.G * a.d;
     const float* gz = a.gz + (size_t)t * a.ld_gz;
     float ss = 0.f;
+    if (VEC) {                                       // four values at a time (rows on 16-byte boundaries, four of one head)
+        for (int i = threadIdx.x * 4; i < size; i += blockDim.x * 4) {
+            int c = c0 + i;
+            float4 z4 = *reinterpret_cast<const float4*>(gz + c), o4 = *reinterpret_cast<const float4*>(o + c);
+            float4 v4 = *reinterpret_cast<const float4*>(v + c), y4;
+            float sk = a.skip ? a.skip[c / a.dv] : 0.f;
+            auto one = [&](float z, float oo, float vv) {
+                float g = gd_sigmoid(z);
+                if (a.gate_act == 1) g *= z;
+                float y = (a.skip ? fmaf(sk, vv, oo) : oo) * g;
+                ss = fmaf(y, y, ss);
+                return y;
+            };
+            y4.x = one(z4.x, o4.x, v4.x); y4.y = one(z4.y, o4.y, v4.y); y4.z = one(z4.z, o4.z, v4.z); y4.w = one(z4.w, o4.w, v4.w);
+            *reinterpret_cast<float4*>(gd_part_smem + i) = y4;
+        }
+        float inv = 1.0f / sqrtf(ce_block_sum(ss, scratch) / (float)size + a.eps);
+        for (int i = threadIdx.x * 4; i < size; i += blockDim.x * 4) {          // (every thread reads what it wrote)
+            int c = c0 + i;
+            float4 y4 = *reinterpret_cast<const float4*>(gd_part_smem + i);
+            float4 w4 = a.norm_w ? *reinterpret_cast<const float4*>(a.norm_w + c) : make_float4(1.f, 1.f, 1.f, 1.f);
+            float r0 = y4.x * inv * w4.x * a.out_scale, r1 = y4.y * inv * w4.y * a.out_scale;
+            float r2 = y4.z * inv * w4.z * a.out_scale, r3 = y4.w * inv * w4.w * a.out_scale;
+            T* dst = (T*)a.out + (size_t)t * n + c;
+            if (sizeof(T) == 4) *reinterpret_cast<float4*>(dst) = make_float4(r0, r1, r2, r3);
+            else {
+                __nv_bfloat162 lo = __floats2bfloat162_rn(r0, r1), hi = __floats2bfloat162_rn(r2, r3);
+                *reinterpret_cast<uint2*>(dst) = make_uint2(*reinterpret_cast<unsigned*>(&lo), *reinterpret_cast<unsigned*>(&hi));
+            }
+        }
+        return;
+    }
     for (int i = threadIdx.x; i < size; i += blockDim.x) {
         int c = c0 + i;
         float z = gz[c], g = gd_sigmoid(z);
@@ -737,7 +851,18 @@ extern "C" int ce_gated_delta(const float* proj, const float* dec, const float* 
                      write_mode, ones, norm_all, parts, T == B ? 1 : 0};
     int heads = 2 * G + H;
     int threads = heads >= 8 ? 256 : 32 * heads;
-    if (stage == 1) {
+    if (stage == 1 && operands == 2 && K <= 5 && decay_mode != 0) {
+        const int C = 2 * G * d + H * dv, tile = T >= 4 * GD_CONV_TOKENS ? GD_CONV_TOKENS : 1;
+        dim3 grid((T + tile - 1) / tile, (C + 255) / 256);
+        ce_note("gated_delta_conv_kernel");
+        switch (K) {
+            case 1: ce_launch(gated_delta_conv_kernel<1>, grid, 256, 0, stream, a, T, tile); break;
+            case 2: ce_launch(gated_delta_conv_kernel<2>, grid, 256, 0, stream, a, T, tile); break;
+            case 3: ce_launch(gated_delta_conv_kernel<3>, grid, 256, 0, stream, a, T, tile); break;
+            case 4: ce_launch(gated_delta_conv_kernel<4>, grid, 256, 0, stream, a, T, tile); break;
+            default: ce_launch(gated_delta_conv_kernel<5>, grid, 256, 0, stream, a, T, tile); break;
+        }
+    } else if (stage == 1) {
         ce_note("gated_delta_prepare_kernel");
         int per_block = threads / 32, want = (heads + per_block - 1) / per_block, room = 4 * 148 / T;
         int split = want < room ? want : room;
@@ -746,7 +871,7 @@ extern "C" int ce_gated_delta(const float* proj, const float* dec, const float* 
         if (T == B) return CE_OK;               // prepare has done it
         if (decay_mode == 3) {
             ce_note("gated_delta_scan_kernel");
-            ce_launch(gated_delta_scan_kernel, dim3(B, (H + 31) / 32), 256, 0, stream, a);
+            ce_launch(gated_delta_scan_kernel, dim3(B, (H + GD_SCAN_HEADS - 1) / GD_SCAN_HEADS), 256, 0, stream, a);
             return ce_check_launch("ce_gated_delta");
         }
         if (K == 1) return CE_OK;
@@ -755,14 +880,17 @@ extern "C" int ce_gated_delta(const float* proj, const float* dec, const float* 
         ce_launch(gated_delta_keep_kernel, (int)(want < 148 * 8 ? want : 148 * 8), 256, 0, stream, a, B);
     } else if (stage == 4 && parts > 0) {
         ce_note("gated_delta_part_finish_kernel");
-        int size = H * dv / parts, th = size >= 2048 ? 256 : size >= 512 ? 128 : 64;
+        int size = H * dv / parts, P_v = 2 * G * d;
+        bool v4 = size % 4 == 0 && dv % 4 == 0 && P_v % 4 == 0 && ld_gz % 4 == 0 &&
+                  (((uintptr_t)gz | (uintptr_t)raw | (uintptr_t)prep | (uintptr_t)norm_w | (uintptr_t)out) & 15) == 0;
+        int items = v4 ? size / 4 : size, th = items >= 1024 ? 1024 : items >= 256 ? 256 : items >= 128 ? 128 : 64;
         size_t smem = (size_t)size * sizeof(float);
         auto go = [&](auto kernel) {
             if (smem > 40 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
             ce_launch(kernel, dim3(T, parts), th, smem, stream, a);
         };
-        if (out_dtype == CE_F32) go(gated_delta_part_finish_kernel<float>);
-        else go(gated_delta_part_finish_kernel<__nv_bfloat16>);
+        if (out_dtype == CE_F32) { if (v4) go(gated_delta_part_finish_kernel<float, true>); else go(gated_delta_part_finish_kernel<float, false>); }
+        else { if (v4) go(gated_delta_part_finish_kernel<__nv_bfloat16, true>); else go(gated_delta_part_finish_kernel<__nv_bfloat16, false>); }
     } else if (stage == 4) {
         ce_note("gated_delta_finish_kernel");
         int th = H >= 8 ? 256 : 32 * H;

@@ -139,25 +139,41 @@ extern "C" int ce_moe_route(const float* z, int* ids, float* weights, float* sga
 // ---------------------------------------------------------------------------------------------
 // the pairs laid out by expert: one block
 // ---------------------------------------------------------------------------------------------
+// An expert's rows follow the order of the pairs.  Every warp owns a run of consecutive pairs: it counts them by expert, the
+// warps' counts of an expert become the warps' first places by a running sum, and every warp deals its pairs out from there.
 __global__ void __launch_bounds__(1024) moe_align_kernel(const int* __restrict__ ids, int n, int top, int E, int BM, int max_rows,
                                                          int* __restrict__ row_token, int* __restrict__ pair_row,
                                                          int* __restrict__ tile_expert, int* __restrict__ n_tiles) {
     ce_pdl_begin();
     extern __shared__ int moe_align_smem[];
-    int* count = moe_align_smem;          // [E], then the next free row of every expert
-    int* first = count + E;               // [E + 1]: an expert's first row
-    for (int e = threadIdx.x; e < E; e += blockDim.x) count[e] = 0;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n_warps = blockDim.x >> 5;
+    int* place = moe_align_smem;          // [n_warps][E]: a warp's count of an expert, then its next free row
+    int* first = place + (size_t)n_warps * E;     // [E + 1]: an expert's first row
+    for (int e = threadIdx.x; e < n_warps * E; e += blockDim.x) place[e] = 0;
     __syncthreads();
-    for (int i = threadIdx.x; i < n; i += blockDim.x) {
+    const int per = ((n + n_warps - 1) / n_warps + 31) / 32 * 32;          // pairs a warp owns
+    const int lo = min(n, warp * per), hi = min(n, lo + per);
+    int* mine = place + (size_t)warp * E;
+    for (int i = lo + lane; i < hi; i += 32) {
         int e = ids[i];
-        if (e >= 0 && e < E) atomicAdd(&count[e], 1);
+        if (e >= 0 && e < E) atomicAdd(&mine[e], 1);
+    }
+    __syncthreads();
+    for (int e = threadIdx.x; e < E; e += blockDim.x) {           // the warps' counts to offsets within the expert
+        int sum = 0;
+        for (int w = 0; w < n_warps; ++w) {
+            int c = place[(size_t)w * E + e];
+            place[(size_t)w * E + e] = sum;
+            sum += c;
+        }
+        first[e] = sum;
     }
     __syncthreads();
     if (threadIdx.x < 32) {               // a warp's running sum over the experts, 32 at a time
         int base = 0;
         for (int e0 = 0; e0 < E; e0 += 32) {
             int e = e0 + threadIdx.x;
-            int c = e < E ? (count[e] + BM - 1) / BM * BM : 0, incl = c;
+            int c = e < E ? (first[e] + BM - 1) / BM * BM : 0, incl = c;
             for (int o = 1; o < 32; o <<= 1) {
                 int v = __shfl_up_sync(0xffffffffu, incl, o);
                 if ((int)threadIdx.x >= o) incl += v;
@@ -170,30 +186,24 @@ __global__ void __launch_bounds__(1024) moe_align_kernel(const int* __restrict__
     __syncthreads();
     const int rows = first[E];
     for (int p = threadIdx.x; p < rows && p < max_rows; p += blockDim.x) row_token[p] = -1;
-    for (int e = threadIdx.x; e < E; e += blockDim.x) {
+    for (int e = threadIdx.x; e < E; e += blockDim.x)
         for (int p = first[e]; p < first[e + 1]; p += BM) tile_expert[p / BM] = e;
-        count[e] = first[e];
-    }
     __syncthreads();
-    // an expert's rows in the order of the pairs: a thread's pairs are consecutive, and the threads take their turns by
-    // counting how many earlier pairs name the same expert (ranks through shared-memory counters, chunk by chunk)
-    for (int i0 = 0; i0 < n; i0 += blockDim.x) {
-        int i = i0 + threadIdx.x;
-        int e = i < n ? ids[i] : -1;
-        // rank among the chunk's pairs of the same expert: warp by warp, in order
-        for (int w = 0; w < (int)(blockDim.x >> 5); ++w) {
-            if ((int)(threadIdx.x >> 5) == w && e >= 0 && e < E) {
-                unsigned same = __match_any_sync(__activemask(), e);
-                int rank = __popc(same & ((1u << (threadIdx.x & 31)) - 1));
-                int base = count[e];
-                __syncwarp(__activemask());
-                int p = base + rank;
-                pair_row[i] = p;
-                row_token[p] = i / top;
-                if (rank == __popc(same) - 1) count[e] = base + rank + 1;
-            }
-            __syncthreads();
+    for (int i0 = lo; i0 < hi; i0 += 32) {
+        const int i = i0 + lane, e = i < hi ? ids[i] : -1;
+        const bool live = e >= 0 && e < E;
+        const unsigned same = __match_any_sync(0xffffffffu, live ? e : -1);
+        const int rank = __popc(same & ((1u << lane) - 1));
+        int base = 0;
+        if (live) base = mine[e];
+        __syncwarp();
+        if (live) {
+            int p = first[e] + base + rank;
+            pair_row[i] = p;
+            row_token[p] = i / top;
+            if (rank == __popc(same) - 1) mine[e] = base + rank + 1;
         }
+        __syncwarp();
     }
 }
 
@@ -208,9 +218,12 @@ extern "C" int ce_moe_align(const int* ids, int n_pairs, int top, int E, int BM,
     if (!ids || !row_token || !pair_row || !tile_expert || !n_tiles) return ce_fail(CE_ERR_ARG, "ce_moe_align: null pointer");
     if (E <= 0 || E > MOE_MAX_EXPERTS || BM <= 0 || top <= 0 || max_rows < ce_moe_max_tiles(n_pairs, E, BM) * BM)
         return ce_fail(CE_ERR_SIZE, "ce_moe_align: %d experts, tiles of %d, room for %d rows", E, BM, max_rows);
-    size_t smem = (size_t)(2 * E + 1) * sizeof(int);
-    ce_note("moe_align_kernel");
     int threads = n_pairs >= 1024 ? 1024 : (n_pairs + 31) / 32 * 32;
+    while (threads > 32 && (size_t)(threads / 32 + 1) * E * sizeof(int) > 160 * 1024) threads /= 2;      // (many experts: fewer warps)
+    threads = threads / 32 * 32;
+    size_t smem = ((size_t)(threads / 32 + 1) * E + 1) * sizeof(int);
+    if (smem > 40 * 1024) cudaFuncSetAttribute(moe_align_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    ce_note("moe_align_kernel");
     ce_launch(moe_align_kernel, 1, threads, smem, stream, ids, n_pairs, top, E, BM, max_rows, row_token, pair_row, tile_expert, n_tiles);
     return ce_check_launch("ce_moe_align");
 }
