@@ -142,27 +142,31 @@ struct TcArgs {
 __device__ __forceinline__ float silu_mul(float g, float u) { return g / (1.0f + __expf(-g)) * u; }
 // the same with the approximate reciprocal (the result is rounded to bfloat16 right after)
 __device__ __forceinline__ float silu_mul_fast(float g, float u) { return __fdividef(g, 1.0f + __expf(-g)) * u; }
-// the gated epilogue's activation by mode; bg, bu: the feature's biases (mode 6)
+// the gated epilogue's activation; CLAMP: the clamped one (mode 6) with the feature's biases bg, bu, compiled apart so that the
+// others' epilogues carry nothing of it
+template <bool CLAMP>
 __device__ __forceinline__ float gated_mul(const TcArgs& a, float g, float u, float bg, float bu) {
-    if (a.mode == TC_CLAMPGLU) return ce_clamp_glu_fast(g + bg, u + bu, a.limit, a.alpha);
+    if (CLAMP) return ce_clamp_glu_fast(g + bg, u + bu, a.limit, a.alpha);
     return a.mode == TC_RELUGLU ? fmaxf(g, 0.f) * u : silu_mul(g, u);
 }
+template <bool CLAMP>
 __device__ __forceinline__ float gated_mul_fast(const TcArgs& a, float g, float u, float bg, float bu) {
-    if (a.mode == TC_CLAMPGLU) return ce_clamp_glu_fast(g + bg, u + bu, a.limit, a.alpha);
+    if (CLAMP) return ce_clamp_glu_fast(g + bg, u + bu, a.limit, a.alpha);
     return a.mode == TC_RELUGLU ? fmaxf(g, 0.f) * u : silu_mul_fast(g, u);
 }
 __device__ __forceinline__ float gate_bias(const TcArgs& a, int n, int up) { return a.bias && n < a.N ? a.bias[up * a.N + n] : 0.f; }
 
+template <bool CLAMP = false>
 __device__ __forceinline__ void epilogue_store(const TcArgs& a, int m, int n, float v, float up) {
     size_t o = (size_t)m * a.ldo + n;
     if (a.mode == TC_STORE) ((__nv_bfloat16*)a.out)[o] = __float2bfloat16_rn(v);
     else if (a.mode == TC_STORE_F32) ((float*)a.out)[o] = v;
     else if (a.mode == TC_ACCUM_F32) ((float*)a.out)[o] += v;
     else if (a.mode == TC_RELU2) { float r = fmaxf(v, 0.f); ((__nv_bfloat16*)a.out)[o] = __float2bfloat16_rn(r * r); }
-    else ((__nv_bfloat16*)a.out)[o] = __float2bfloat16_rn(gated_mul(a, v, up, gate_bias(a, n, 0), gate_bias(a, n, 1)));
+    else ((__nv_bfloat16*)a.out)[o] = __float2bfloat16_rn(gated_mul<CLAMP>(a, v, up, CLAMP ? gate_bias(a, n, 0) : 0.f, CLAMP ? gate_bias(a, n, 1) : 0.f));
 }
 
-template <int BN, int NACC, bool COOP>
+template <int BN, int NACC, bool COOP, bool CLAMP = false>
 __global__ void __launch_bounds__(THREADS, 2) gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w,
                                                          const __grid_constant__ CUtensorMap map_x, TcArgs a, int stages) {
     extern __shared__ __align__(1024) unsigned char smem_raw[];
@@ -312,7 +316,7 @@ __global__ void __launch_bounds__(THREADS, 2) gemm_tc_kernel(const __grid_consta
             // two threads of a feature share each chunk of 16 tokens: the gate thread takes tokens 0..7 (and
             // needs their up values), the up thread tokens 8..15 (and needs their gate values).
             bool up_row = row >= 64;
-            const float bg = gate_bias(a, n, 0), bu = gate_bias(a, n, 1);
+            const float bg = CLAMP ? gate_bias(a, n, 0) : 0.f, bu = CLAMP ? gate_bias(a, n, 1) : 0.f;
 #pragma unroll 1
             for (int c = 0; c < BN; c += 16) {
                 if (c >= m_valid) break;
@@ -337,7 +341,7 @@ __global__ void __launch_bounds__(THREADS, 2) gemm_tc_kernel(const __grid_consta
                     for (int j = 0; j < 8; ++j) {
                         float gate = up_row ? xg[j] : g[j];
                         float upv = up_row ? g[8 + j] : xu[j];
-                        if (c + t0 + j < m_valid) op[(size_t)j * a.ldo] = __float2bfloat16_rn(gated_mul_fast(a, gate, upv, bg, bu));
+                        if (c + t0 + j < m_valid) op[(size_t)j * a.ldo] = __float2bfloat16_rn(gated_mul_fast<CLAMP>(a, gate, upv, bg, bu));
                     }
                 }
             }
@@ -737,7 +741,7 @@ __device__ __forceinline__ void tmem_ld32(uint32_t taddr, float (&v)[32]) {
     for (int i = 0; i < 32; ++i) v[i] = __uint_as_float(r[i]);
 }
 
-template <int BN, int NACC>
+template <int BN, int NACC, bool CLAMP = false>
 __global__ void __launch_bounds__(THREADS) gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_w,
                                                                     const __grid_constant__ CUtensorMap map_x, TcArgs a,
                                                                     int stages, int tiles_n, int tiles_m) {
@@ -857,7 +861,7 @@ __global__ void __launch_bounds__(THREADS) gemm_tc_persistent_kernel(const __gri
                     } else {
 #pragma unroll
                         for (int j = 0; j < 32; ++j)
-                            if (c + j < m_valid) epilogue_store(a, m0 + c + j, n, g[j], NACC == 2 ? u[j] : 0.f);
+                            if (c + j < m_valid) epilogue_store<CLAMP>(a, m0 + c + j, n, g[j], NACC == 2 ? u[j] : 0.f);
                     }
                 }
             }
@@ -927,7 +931,7 @@ __device__ __forceinline__ void umma2_commit_both(uint64_t* bar) {
 // features, brought by two TMA boxes into ONE tile, so the product is the same single-accumulator product
 // as any other and a pair tile covers 128 features; in the epilogue the warps that hold the up rows (lanes
 // 64..127 of tensor memory) hand their values to the warps that hold the gate rows through shared memory.
-template <int BN, bool GU, int KSUB>
+template <int BN, bool GU, int KSUB, bool CLAMP = false>
 __global__ void __launch_bounds__(THREADS) gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_w,
                                                               const __grid_constant__ CUtensorMap map_x, TcArgs a,
                                                               int stages, int tiles_n, int tiles_m) {
@@ -1055,7 +1059,7 @@ __global__ void __launch_bounds__(THREADS) gemm_tc_pair_kernel(const __grid_cons
             int buf = lt & 1;
             int n = (tile / tiles_m) * (2 * ROWS_N) + rank * ROWS_N + (GU ? (row & 63) : row);
             bool up_row = GU && row >= 64;
-            const float bg = GU ? gate_bias(a, n, 0) : 0.f, bu = GU ? gate_bias(a, n, 1) : 0.f;
+            const float bg = CLAMP ? gate_bias(a, n, 0) : 0.f, bu = CLAMP ? gate_bias(a, n, 1) : 0.f;
             int m0 = (tile % tiles_m) * BN;
             int m_valid = min(BN, a.M - m0);
             const bool accum = !GU && a.mode == TC_ACCUM_F32 && n < a.N;
@@ -1116,7 +1120,7 @@ __global__ void __launch_bounds__(THREADS) gemm_tc_pair_kernel(const __grid_cons
                         for (int j = 0; j < 16; ++j) {
                             float gate = up_row ? xg[j] : g[j];
                             float upv = up_row ? g[16 + j] : xu[j];
-                            if (c + t0 + j < m_valid) op[(size_t)j * a.ldo] = __float2bfloat16_rn(gated_mul_fast(a, gate, upv, bg, bu));
+                            if (c + t0 + j < m_valid) op[(size_t)j * a.ldo] = __float2bfloat16_rn(gated_mul_fast<CLAMP>(a, gate, upv, bg, bu));
                         }
                     }
                     continue;
@@ -1147,7 +1151,7 @@ int get_map(const void* ptr, long long rows, long long cols, long long ld, int b
     return ce_tensor_map_bf16(ptr, rows, cols, ld, box_rows, out, "ce_gemm_tc");
 }
 
-template <int BN, int NACC, bool COOP>
+template <int BN, int NACC, bool COOP, bool CLAMP = false>
 int launch(const CUtensorMap& mw, const CUtensorMap& mx, const TcArgs& a, dim3 grid, cudaStream_t stream) {
     constexpr size_t stage = BM * BK * 2 + BN * BK * 2;
     // small tiles: at most half an SM's shared memory, so that the blocks of the next kernel (launched
@@ -1162,7 +1166,7 @@ int launch(const CUtensorMap& mw, const CUtensorMap& mx, const TcArgs& a, dim3 g
     size_t smem = stages * stage + 1024;
     static bool attr_set = false;
     if (!attr_set) {
-        cudaError_t e = cudaFuncSetAttribute(gemm_tc_kernel<BN, NACC, COOP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaError_t e = cudaFuncSetAttribute(gemm_tc_kernel<BN, NACC, COOP, CLAMP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return ce_fail(CE_ERR_CUDA, "ce_gemm_tc: %s", cudaGetErrorString(e));
         attr_set = true;
     }
@@ -1182,15 +1186,15 @@ int launch(const CUtensorMap& mw, const CUtensorMap& mx, const TcArgs& a, dim3 g
         cfg.attrs = attr;
         cfg.numAttrs = ce_pdl_enabled() ? 2 : 1;
         ce_note("gemm_tc_kernel (split-K in a cluster)");
-        cudaError_t e = cudaLaunchKernelEx(&cfg, gemm_tc_kernel<BN, NACC, COOP>, mw, mx, a, stages);
+        cudaError_t e = cudaLaunchKernelEx(&cfg, gemm_tc_kernel<BN, NACC, COOP, CLAMP>, mw, mx, a, stages);
         if (e != cudaSuccess) return ce_fail(CE_ERR_CUDA, "ce_gemm_tc (cluster of %d): %s", (int)grid.z, cudaGetErrorString(e));
         return ce_check_launch("ce_gemm_tc");
     }
-    { ce_note(COOP ? "gemm_tc_kernel (split-K, splits add together)" : a.splits > 1 ? "gemm_tc_kernel (split-K)" : "gemm_tc_kernel"); ce_launch(gemm_tc_kernel<BN, NACC, COOP>, grid, THREADS, smem, stream, mw, mx, a, stages); }
+    { ce_note(COOP ? "gemm_tc_kernel (split-K, splits add together)" : a.splits > 1 ? "gemm_tc_kernel (split-K)" : "gemm_tc_kernel"); ce_launch(gemm_tc_kernel<BN, NACC, COOP, CLAMP>, grid, THREADS, smem, stream, mw, mx, a, stages); }
     return ce_check_launch("ce_gemm_tc");
 }
 
-template <int BN, int NACC>
+template <int BN, int NACC, bool CLAMP = false>
 int launch_persistent(const CUtensorMap& mw, const CUtensorMap& mx, const TcArgs& a, int tiles_n, int tiles_m, cudaStream_t stream) {
     constexpr size_t stage = NACC * BM * BK * 2 + BN * BK * 2;
     int stages = (int)((200 * 1024) / stage);
@@ -1198,17 +1202,17 @@ int launch_persistent(const CUtensorMap& mw, const CUtensorMap& mx, const TcArgs
     size_t smem = stages * stage + 1024;
     static bool attr_set = false;
     if (!attr_set) {
-        cudaError_t e = cudaFuncSetAttribute(gemm_tc_persistent_kernel<BN, NACC>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024 - 2048);
+        cudaError_t e = cudaFuncSetAttribute(gemm_tc_persistent_kernel<BN, NACC, CLAMP>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024 - 2048);
         if (e != cudaSuccess) return ce_fail(CE_ERR_CUDA, "ce_gemm_tc: %s", cudaGetErrorString(e));
         attr_set = true;
     }
     long long total = (long long)tiles_n * tiles_m;
     int grid = (int)(total < ce_sm_count() ? total : ce_sm_count());
-    { ce_note("gemm_tc_persistent_kernel"); ce_launch(gemm_tc_persistent_kernel<BN, NACC>, grid, THREADS, smem, stream, mw, mx, a, stages, tiles_n, tiles_m); }
+    { ce_note("gemm_tc_persistent_kernel"); ce_launch(gemm_tc_persistent_kernel<BN, NACC, CLAMP>, grid, THREADS, smem, stream, mw, mx, a, stages, tiles_n, tiles_m); }
     return ce_check_launch("ce_gemm_tc (persistent)");
 }
 
-template <int BN, bool GU, int KSUB>
+template <int BN, bool GU, int KSUB, bool CLAMP = false>
 int launch_pair(const CUtensorMap& mw, const CUtensorMap& mx, const TcArgs& a, int tiles_n, int tiles_m, cudaStream_t stream) {
     constexpr size_t stage = KSUB * (BM * BK * 2 + (BN / 2) * BK * 2);
     int stages = (int)((200 * 1024) / stage);
@@ -1216,7 +1220,7 @@ int launch_pair(const CUtensorMap& mw, const CUtensorMap& mx, const TcArgs& a, i
     size_t smem = stages * stage + 1024;
     static bool attr_set = false;
     if (!attr_set) {
-        cudaError_t e = cudaFuncSetAttribute(gemm_tc_pair_kernel<BN, GU, KSUB>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaError_t e = cudaFuncSetAttribute(gemm_tc_pair_kernel<BN, GU, KSUB, CLAMP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return ce_fail(CE_ERR_CUDA, "ce_gemm_tc: %s", cudaGetErrorString(e));
         attr_set = true;
     }
@@ -1236,7 +1240,7 @@ int launch_pair(const CUtensorMap& mw, const CUtensorMap& mx, const TcArgs& a, i
         cfg.attrs = attr;
         cfg.numAttrs = 1;
         int n = 0;
-        cudaError_t e = cudaOccupancyMaxActiveClusters(&n, gemm_tc_pair_kernel<BN, GU, KSUB>, &cfg);
+        cudaError_t e = cudaOccupancyMaxActiveClusters(&n, gemm_tc_pair_kernel<BN, GU, KSUB, CLAMP>, &cfg);
         if (e != cudaSuccess || n < 1) return ce_fail(CE_ERR_CUDA, "ce_gemm_tc (pairs): no resident cluster: %s", cudaGetErrorString(e));
         max_pairs = n;
         if (getenv("CE_GEMM_TRACE")) fprintf(stderr, "[carbon_engine_b200] gemm pairs<%d,%d>: %d resident\n", BN, (int)GU, n);
@@ -1249,7 +1253,7 @@ int launch_pair(const CUtensorMap& mw, const CUtensorMap& mx, const TcArgs& a, i
     cfg.attrs = attr;
     cfg.numAttrs = ce_pdl_enabled() ? 2 : 1;
     ce_note("gemm_tc_pair_kernel");
-    cudaError_t e = cudaLaunchKernelEx(&cfg, gemm_tc_pair_kernel<BN, GU, KSUB>, mw, mx, a, stages, tiles_n, tiles_m);
+    cudaError_t e = cudaLaunchKernelEx(&cfg, gemm_tc_pair_kernel<BN, GU, KSUB, CLAMP>, mw, mx, a, stages, tiles_n, tiles_m);
     if (e != cudaSuccess) return ce_fail(CE_ERR_CUDA, "ce_gemm_tc (pairs): %s", cudaGetErrorString(e));
     return ce_check_launch("ce_gemm_tc (pairs)");
 }
@@ -1366,12 +1370,16 @@ extern "C" int ce_gemm_tc(const void* A, const void* W, void* C, int M, int N, i
             long long ptiles_m = (M + ptok - 1) / ptok;
             if (nacc == 2) {
                 if ((prc = get_map(W, (long long)N * 2, K, K, BM / 2, &pw2))) return prc;
+                if (mode == TC_CLAMPGLU)
+                    return ptok == 128 ? launch_pair<128, true, 2, true>(pw2, px2, pa, (int)rows_t, (int)ptiles_m, stream)
+                                       : launch_pair<256, true, 2, true>(pw2, px2, pa, (int)rows_t, (int)ptiles_m, stream);
                 return ptok == 128 ? launch_pair<128, true, 2>(pw2, px2, pa, (int)rows_t, (int)ptiles_m, stream)
                                    : launch_pair<256, true, 2>(pw2, px2, pa, (int)rows_t, (int)ptiles_m, stream);
             }
             return ptok == 128 ? launch_pair<128, false, 2>(pw, px2, pa, (int)rows_t, (int)ptiles_m, stream)
                                : launch_pair<256, false, 2>(pw, px2, pa, (int)rows_t, (int)ptiles_m, stream);
         }
+        if (mode == TC_CLAMPGLU) return launch_persistent<128, 2, true>(pw, px, pa, (int)tiles_n, (int)tiles_m, stream);
         return nacc == 2 ? launch_persistent<128, 2>(pw, px, pa, (int)tiles_n, (int)tiles_m, stream)
                          : launch_persistent<256, 1>(pw, px, pa, (int)tiles_n, (int)tiles_m, stream);
     }
@@ -1406,7 +1414,8 @@ extern "C" int ce_gemm_tc(const void* A, const void* W, void* C, int M, int N, i
     TcArgs a{C, scratch, counters, status, M, N, K, ldc, mode, splits, (kblocks + splits - 1) / splits, kblocks, trace, cluster, coop, bias, limit, alpha};
 #define TC_CASE(BN_)                                                                  \
     case BN_:                                                                         \
-        return nacc == 2 ? launch<BN_, 2, false>(mw, mx, a, grid, stream)                  \
+        return mode == TC_CLAMPGLU ? launch<BN_, 2, false, true>(mw, mx, a, grid, stream)      \
+               : nacc == 2 ? launch<BN_, 2, false>(mw, mx, a, grid, stream)                  \
                          : a.coop ? launch<BN_, 1, true>(mw, mx, a, grid, stream) : launch<BN_, 1, false>(mw, mx, a, grid, stream);
     switch (bn) {
         TC_CASE(16)
