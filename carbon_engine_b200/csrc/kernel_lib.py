@@ -23,6 +23,8 @@ _SIGNATURES = {
     "ce_set_pdl": (None, [_i]),
     # table, dtype, tokens, x, T, H, V, status, scale, stream
     "ce_embed": (_i, [_p, _i, _p, _p, _i, _i, _i, _p, _f, _p]),
+    # table, dtype, tokens, w, x, xb, T, H, V, status, scale, eps, stream
+    "ce_embed_norm": (_i, [_p, _i] + [_p] * 4 + [_i] * 3 + [_p, _f, _f, _p]),
     # x, w, out, out_dtype, rows, R, H, eps, stream
     "ce_rmsnorm": (_i, [_p, _p, _p, _i, _p, _i, _i, _f, _p]),
     # qkv, k_pool, v_pool, dtype, qw, kw, cos, sin, positions, seq_of_token, seq_slot, block_table, status,
@@ -42,6 +44,8 @@ _SIGNATURES = {
     "ce_rmsnorm_add": (_i, [_p, _p, _p, _p, _i, _i, _f, _p]),
     # y, bias, w, x, w2, h, h_dtype, T, H, eps, eps2, stream
     "ce_rmsnorm_add_norm": (_i, [_p] * 6 + [_i] * 3 + [_f, _f, _p]),
+    # y0, y1, wm0, wm1, members, bias, w, x, xb, T, H, alpha, c, eps, eps_m, stream
+    "ce_residual_norm": (_i, [_p] * 4 + [_i] + [_p] * 4 + [_i] * 2 + [_f] * 4 + [_p]),
     # x, n, cap, stream
     "ce_tanh_cap": (_i, [_p, _ll, _f, _p]),
     # src, out, out_dtype, T, ld, off, L, stream
@@ -60,17 +64,18 @@ _SIGNATURES = {
     "ce_head_matmul": (_i, [_p, _i, _i, _p, _p, _i, _i, _p, _i, _i, _i, _i, _i, _i, _i, _p]),
     # q, k_pool, v_pool, gate, out, dtype, positions, seq_of_token, seq_slot, block_table, status, T, nh, nkv, d, dv,
     # q_stride, q_head, ldk, ldv, gate_stride, page_size, max_pages, num_pages, window, keep_first, scale, softcap, sinks,
-    # out_scale, stream
-    "ce_masked_attention": (_i, [_p] * 5 + [_i] + [_p] * 5 + [_i] * 15 + [_f, _f, _p, _f, _p]),
-    # proj, q_out, k_pool, v_pool, dtype, wq, wk, head_scale, cos, sin, positions, seq_of_token, seq_slot, block_table, status,
-    # T, ld, off_q, off_k, off_v, nh, nkv, d, dv, rd, page_size, max_pages, num_pages, max_pos, write_kv, eps, stream
-    "ce_norm_rope_kvwrite": (_i, [_p] * 4 + [_i] + [_p] * 10 + [_i] * 15 + [_f, _p]),
+    # out_scale, slopes, stream
+    "ce_masked_attention": (_i, [_p] * 5 + [_i] + [_p] * 5 + [_i] * 15 + [_f, _f, _p, _f, _p, _p]),
+    # proj, q_out, k_pool, v_pool, dtype, wq, wk, head_scale, pos_scale, cos, sin, positions, seq_of_token, seq_slot, block_table,
+    # status, T, ld, off_q, off_k, off_v, nh, nkv, d, dv, rd, page_size, max_pages, num_pages, max_pos, write_kv, eps, norm_mode,
+    # pairing, max_pos_scale, stream
+    "ce_norm_rope_kvwrite": (_i, [_p] * 4 + [_i] + [_p] * 11 + [_i] * 15 + [_f] + [_i] * 3 + [_p]),
     # d, dv, q_stride, q_head, ldk, ldv, alias
     "ce_masked_attention_mma_supported": (_i, [_i] * 7),
     # q, k_pool, v_pool, gate, out, positions, seq_slot, q_start, block_table, tiles, status, n_tiles, n_tokens, nh, nkv, d, dv,
     # q_stride, q_head, ldk, ldv, gate_stride, page_size, max_pages, num_pages, window, keep_first, scale, softcap, sinks,
-    # out_scale, stream
-    "ce_masked_attention_mma": (_i, [_p] * 11 + [_i] * 16 + [_f, _f, _p, _f, _p]),
+    # out_scale, slopes, stream
+    "ce_masked_attention_mma": (_i, [_p] * 11 + [_i] * 16 + [_f, _f, _p, _f, _p, _p]),
     # H, G, d, dv, decay_mode
     "ce_gated_delta_prep_width": (_i, [_i] * 5),
     # proj, dec, gz, taps, a_log, dt_bias, norm_w, prep, raw, state, kept, out, out_dtype, seq_of_token, seq_slot, q_start,
@@ -110,8 +115,8 @@ _SIGNATURES = {
     # q, k_pool, v_pool, gate, out, positions, seq_slot, q_start, block_table, tiles, status, n_tiles, nh, nkv, d, dv,
     # q_stride, gate_stride, page_size, max_pages, num_pages, window, chunk, scale, lambda, eps, out_scale, stream
     "ce_diff_attention_mma": (_i, [_p] * 11 + [_i] * 12 + [_f] * 4 + [_p]),
-    # z, ids, weights, sgate, T, ld, E, top, groups, keep, scale, correction, scoring, group_score, renormalize, stream
-    "ce_moe_route": (_i, [_p] * 4 + [_i] * 6 + [_f, _p, _i, _i, _i, _p]),
+    # z, ids, weights, sgate, T, ld, E, top, groups, keep, scale, correction, scoring, group_score, renormalize, bias, stream
+    "ce_moe_route": (_i, [_p] * 4 + [_i] * 6 + [_f, _p, _i, _i, _i, _p, _p]),
     "ce_moe_max_tiles": (_i, [_i, _i, _i]),
     # ids, n_pairs, top, E, BM, max_rows, row_token, pair_row, tile_expert, n_tiles, stream
     "ce_moe_align": (_i, [_p] + [_i] * 5 + [_p] * 5),

@@ -72,7 +72,9 @@ struct MmaAttnArgs {
     float scale_log2;           // scale * log2(e)
     const float* sinks;         // [nh] or null: exp(sinks[h]) joins head h's denominator, with no key and no value
     float out_scale;            // the stored rows are multiplied by this
+    const float* slopes;        // [nh] or null: slopes[h] * (position - key) is taken off head h's scaled scores
 };
+// The kernels that form scores are compiled apart (BIAS) for a penalty on distance, so that the plain scores carry nothing of it.
 
 // Stage keys [k0, k0 + AM_TILE) of one KV head into shared memory rows of d + AM_PAD elements.
 // Keys outside [lo, hi] are filled with zeros, so that a masked probability of 0 never meets a NaN.
@@ -137,10 +139,12 @@ __device__ __forceinline__ void ldmatrix_x4(uint32_t (&r)[4], const bf16* p) {
 }
 
 // MASK false: every staged key of the tile is visible to every row of the warp (no compares).
-template <int DMAX, int NK8, bool MASK>
+// BIAS: slope2[r] (base-2 domain) times the distance to the row's position (hi[r]) comes off the scaled score.
+template <int DMAX, int NK8, bool MASK, bool BIAS>
 __device__ __forceinline__ void warp_tile(const uint32_t (&qf)[DMAX / 16][4], float (&o)[DMAX / 8][4], float (&m)[2],
                                           float (&l)[2], const bf16* Ks, const bf16* Vs, int ld, int d, int key_base,
-                                          const int (&lo)[2], const int (&hi)[2], float scale_log2) {
+                                          const int (&lo)[2], const int (&hi)[2], float score_scale, const float (&slope2)[2]) {
+    const float scale_log2 = BIAS ? 1.0f : score_scale;      // what is left to scale once the penalty is in the scores
     int lane = threadIdx.x & 31, quad = lane & 3;
     int mi = lane >> 3, rr = lane & 7;
     float s[NK8][4];
@@ -177,6 +181,13 @@ __device__ __forceinline__ void warp_tile(const uint32_t (&qf)[DMAX / 16][4], fl
             }
         }
     }
+    if (BIAS) {
+#pragma unroll
+        for (int j = 0; j < NK8; ++j)
+#pragma unroll
+            for (int e = 0; e < 4; ++e)
+                s[j][e] = fmaf(s[j][e], score_scale, slope2[e >> 1] * (float)(key_base + j * 8 + 2 * quad + (e & 1) - hi[e >> 1]));
+    }
     // raw maxima; the scale (positive) is applied inside the exponent: p = 2^(s * scale - m)
     float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
@@ -206,7 +217,7 @@ __device__ __forceinline__ void warp_tile(const uint32_t (&qf)[DMAX / 16][4], fl
     for (int j = 0; j < NK8; ++j) {
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-            float p = ce_exp2_fast(fmaf(s[j][e], scale_log2, -muse[e >> 1]));
+            float p = ce_exp2_fast(BIAS ? s[j][e] - muse[e >> 1] : fmaf(s[j][e], scale_log2, -muse[e >> 1]));
             s[j][e] = p;
             l[e >> 1] += p;
         }
@@ -235,7 +246,7 @@ __device__ __forceinline__ void warp_tile(const uint32_t (&qf)[DMAX / 16][4], fl
 // ---------------------------------------------------------------------------------------------
 // Decode: grid (n_seqs * max_splits, nkv, head groups of 16)
 // ---------------------------------------------------------------------------------------------
-template <int DMAX, int ST>
+template <int DMAX, int ST, bool BIAS>
 __global__ void __launch_bounds__(AM_THREADS) attention_decode_kernel(MmaAttnArgs a) {
     ce_pdl_begin();
     extern __shared__ __align__(16) unsigned char smem_raw[];
@@ -275,6 +286,12 @@ __global__ void __launch_bounds__(AM_THREADS) attention_decode_kernel(MmaAttnArg
     for (int i = 0; i < DMAX / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
     float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
     int los[2] = {lo, lo}, his[2] = {pos, pos};
+    float slope2[2] = {0.f, 0.f};
+    if (BIAS) {
+        const float* sl = a.slopes + kvh * G + hg * 16;
+        slope2[0] = grp < heads_here ? sl[grp] * 1.4426950408889634f : 0.f;
+        slope2[1] = grp + 8 < heads_here ? sl[grp + 8] * 1.4426950408889634f : 0.f;
+    }
 
     int n_tiles = (k_end - k_begin + AM_TILE - 1) / AM_TILE;
 #pragma unroll
@@ -296,8 +313,8 @@ __global__ void __launch_bounds__(AM_THREADS) attention_decode_kernel(MmaAttnArg
         if (k0 <= pos) {
             const bf16* kt = Ks + (cur * AM_TILE + warp * 16) * ld;
             const bf16* vt = Vs + (cur * AM_TILE + warp * 16) * ld;
-            if (k0 >= lo && k0 + 15 <= pos) warp_tile<DMAX, 2, false>(qf, o, m, l, kt, vt, ld, d, k0, los, his, a.scale_log2);
-            else warp_tile<DMAX, 2, true>(qf, o, m, l, kt, vt, ld, d, k0, los, his, a.scale_log2);
+            if (k0 >= lo && k0 + 15 <= pos) warp_tile<DMAX, 2, false, BIAS>(qf, o, m, l, kt, vt, ld, d, k0, los, his, a.scale_log2, slope2);
+            else warp_tile<DMAX, 2, true, BIAS>(qf, o, m, l, kt, vt, ld, d, k0, los, his, a.scale_log2, slope2);
         }
     }
     cp_async_wait<0>();
@@ -441,10 +458,12 @@ __device__ __forceinline__ void ldmatrix_x4_trans_addr(uint32_t (&r)[4], uint32_
 // lane/4 and lane/4 + 8 for heads 2*(lane%4) and 2*(lane%4) + 1; its running maxima, sums and output
 // columns are for those two heads.
 // ks, vs: shared addresses of the stage's K and V; each is d/64 panels of [64 keys][128 bytes], swizzled.
-template <int DMAX, bool MASK>
+// BIAS: slope2[r] (base-2 domain) of the thread's two heads times the distance to ``hi`` comes off the scaled score.
+template <int DMAX, bool MASK, bool BIAS>
 __device__ __forceinline__ void warp_tile_swz(const uint32_t (&qf)[DMAX / 16][2], float (&o)[DMAX / 16][4], float (&m)[2],
                                               float (&l)[2], uint32_t ks, uint32_t vs, int slab, int d, int key_base,
-                                              int lo, int hi, float scale_log2) {
+                                              int lo, int hi, float score_scale, const float (&slope2)[2]) {
+    const float scale_log2 = BIAS ? 1.0f : score_scale;      // what is left to scale once the penalty is in the scores
     int lane = threadIdx.x & 31, quad = lane & 3, grp = lane >> 2;
     int mi = lane >> 3, rr = lane & 7;
     float s[4] = {0.f, 0.f, 0.f, 0.f}, s2[4] = {0.f, 0.f, 0.f, 0.f}, s3[4] = {0.f, 0.f, 0.f, 0.f}, s4[4] = {0.f, 0.f, 0.f, 0.f};
@@ -465,6 +484,11 @@ __device__ __forceinline__ void warp_tile_swz(const uint32_t (&qf)[DMAX / 16][2]
     }
 #pragma unroll
     for (int e = 0; e < 4; ++e) s[e] = (s[e] + s2[e]) + (s3[e] + s4[e]);
+    if (BIAS) {
+        const float d_a = (float)(key_base + grp - hi), d_b = (float)(key_base + grp + 8 - hi);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) s[e] = fmaf(s[e], score_scale, slope2[e & 1] * (e < 2 ? d_a : d_b));
+    }
     if (MASK) {
         int k_a = key_base + grp, k_b = k_a + 8;
         if (!(k_a >= lo && k_a <= hi)) s[0] = s[1] = -INFINITY;
@@ -487,7 +511,7 @@ __device__ __forceinline__ void warp_tile_swz(const uint32_t (&qf)[DMAX / 16][2]
     float p[4];
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
-        p[e] = ce_exp2_fast(fmaf(s[e], scale_log2, -muse[e & 1]));
+        p[e] = ce_exp2_fast(BIAS ? s[e] - muse[e & 1] : fmaf(s[e], scale_log2, -muse[e & 1]));
         l[e & 1] += p[e];                       // this thread's keys only: the 8 partial sums are added at the end
     }
     // most tiles move no head's maximum: then every alpha is exactly 1 and the output needs no rescaling
@@ -520,7 +544,7 @@ __device__ __forceinline__ void warp_tile_swz(const uint32_t (&qf)[DMAX / 16][2]
     }
 }
 
-template <int DMAX, int ST>
+template <int DMAX, int ST, bool BIAS>
 __global__ void __launch_bounds__(AMT_THREADS) attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k,
                                                                           const __grid_constant__ CUtensorMap map_v,
                                                                           MmaAttnArgs a, int box_rows) {
@@ -634,6 +658,12 @@ __global__ void __launch_bounds__(AMT_THREADS) attention_decode_tma_kernel(const
 #pragma unroll
     for (int i = 0; i < DMAX / 16; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
     float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+    float slope2[2] = {0.f, 0.f};
+    if (BIAS) {
+        const float* sl = a.slopes + kvh * G + hg * 8;
+        slope2[0] = 2 * quad < heads_here ? sl[2 * quad] * 1.4426950408889634f : 0.f;
+        slope2[1] = 2 * quad + 1 < heads_here ? sl[2 * quad + 1] * 1.4426950408889634f : 0.f;
+    }
 
     {
         int s = 0;
@@ -646,7 +676,7 @@ __global__ void __launch_bounds__(AMT_THREADS) attention_decode_tma_kernel(const
             if (k0 <= pos && k0 + 15 >= lo) {
                 uint32_t ks = base + (uint32_t)s * stage_bytes, vs = ks + kv_bytes;
                 if (k0 >= lo && k0 + 15 <= pos) {
-                    warp_tile_swz<DMAX, false>(qf, o, m, l, ks, vs, warp * 16, d, k0, lo, pos, a.scale_log2);
+                    warp_tile_swz<DMAX, false, BIAS>(qf, o, m, l, ks, vs, warp * 16, d, k0, lo, pos, a.scale_log2, slope2);
                 } else {
                     // zero the V rows of this warp's keys that are not visible (16 bytes a lane and step)
                     for (int c = lane; c < 16 * panels * 8; c += 32) {
@@ -657,7 +687,7 @@ __global__ void __launch_bounds__(AMT_THREADS) attention_decode_tma_kernel(const
                                                       (size_t)(warp * 16 + r) * 128 + (size_t)(rest & 7) * 16) = make_uint4(0, 0, 0, 0);
                     }
                     __syncwarp();
-                    warp_tile_swz<DMAX, true>(qf, o, m, l, ks, vs, warp * 16, d, k0, lo, pos, a.scale_log2);
+                    warp_tile_swz<DMAX, true, BIAS>(qf, o, m, l, ks, vs, warp * 16, d, k0, lo, pos, a.scale_log2, slope2);
                     asm volatile("fence.proxy.async.shared::cta;" ::: "memory");   // before a later copy overwrites these rows
                 }
             }
@@ -793,7 +823,7 @@ __global__ void attention_merge_kernel(MmaAttnArgs a) {
 // ---------------------------------------------------------------------------------------------
 // Prefill: grid (n_tiles, nh)
 // ---------------------------------------------------------------------------------------------
-template <int DMAX>
+template <int DMAX, bool BIAS>
 __global__ void __launch_bounds__(AM_THREADS, DMAX <= 128 ? 3 : 1) attention_prefill_kernel(MmaAttnArgs a) {
     ce_pdl_begin();
     extern __shared__ __align__(16) unsigned char smem_raw[];
@@ -832,6 +862,8 @@ __global__ void __launch_bounds__(AM_THREADS, DMAX <= 128 ? 3 : 1) attention_pre
     float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
     int his[2] = {v0 ? p_first + r0 : -1, v1 ? p_first + r1 : -1};
     int los[2] = {a.window > 0 ? max(0, his[0] - a.window + 1) : 0, a.window > 0 ? max(0, his[1] - a.window + 1) : 0};
+    const float slope_h = BIAS ? a.slopes[h] * 1.4426950408889634f : 0.f;
+    const float slope2[2] = {slope_h, slope_h};
     int warp_hi = p_first + min(warp * 16 + 15, nq - 1);     // last key any row of this warp sees
     int warp_lo = a.window > 0 ? max(0, p_first + warp * 16 - a.window + 1) : 0;
     bool warp_rows_full = warp * 16 + 15 < nq;                // all 16 rows of the warp are real queries
@@ -862,9 +894,9 @@ __global__ void __launch_bounds__(AM_THREADS, DMAX <= 128 ? 3 : 1) attention_pre
             const bf16* vt = Vs + cur * AM_TILE * ld;
             // all 64 keys visible to all 16 rows of the warp: at or below its first row, at or above its last row's window
             if (warp_rows_full && k0 + AM_TILE - 1 <= warp_first_hi && k0 >= warp_last_lo)
-                warp_tile<DMAX, 8, false>(qf, o, m, l, kt, vt, ld, d, k0, los, his, a.scale_log2);
+                warp_tile<DMAX, 8, false, BIAS>(qf, o, m, l, kt, vt, ld, d, k0, los, his, a.scale_log2, slope2);
             else
-                warp_tile<DMAX, 8, true>(qf, o, m, l, kt, vt, ld, d, k0, los, his, a.scale_log2);
+                warp_tile<DMAX, 8, true, BIAS>(qf, o, m, l, kt, vt, ld, d, k0, los, his, a.scale_log2, slope2);
         }
     }
     cp_async_wait<0>();
@@ -922,13 +954,14 @@ extern "C" int ce_attention_decode_tma_supported(int d, int page_size) {
     return d >= 64 && d <= 256 && d % 64 == 0 && page_size >= 8 && (page_size & (page_size - 1)) == 0;
 }
 
-// ``sinks`` (float32 [nh] or null) and ``out_scale``: see ce_softmax_inverse.
+// ``sinks`` (float32 [nh] or null) and ``out_scale``: see ce_softmax_inverse.  ``slopes`` (float32 [nh] or null): a penalty per head
+// and token of distance.
 extern "C" int ce_attention_decode_bf16_sink(const void* q, const void* k_pool, const void* v_pool, void* out, float* scratch,
                                              int* counters, int n_counters, const int* positions, const int* seq_slot, const int* q_start,
                                              const int* ctx_len, const int* block_table, int* status, int n_seqs, int nh,
                                              int nkv, int d, int q_stride, int page_size, int max_pages, int num_pages,
                                              int window, float scale, int max_splits, const float* sinks, float out_scale,
-                                             cudaStream_t stream);
+                                             const float* slopes, cudaStream_t stream);
 
 extern "C" int ce_attention_decode_bf16(const void* q, const void* k_pool, const void* v_pool, void* out, float* scratch,
                                         int* counters, int n_counters, const int* positions, const int* seq_slot, const int* q_start,
@@ -937,7 +970,7 @@ extern "C" int ce_attention_decode_bf16(const void* q, const void* k_pool, const
                                         int window, float scale, int max_splits, cudaStream_t stream) {
     return ce_attention_decode_bf16_sink(q, k_pool, v_pool, out, scratch, counters, n_counters, positions, seq_slot, q_start, ctx_len,
                                          block_table, status, n_seqs, nh, nkv, d, q_stride, page_size, max_pages, num_pages, window,
-                                         scale, max_splits, nullptr, 1.0f, stream);
+                                         scale, max_splits, nullptr, 1.0f, nullptr, stream);
 }
 
 extern "C" int ce_attention_decode_bf16_sink(const void* q, const void* k_pool, const void* v_pool, void* out, float* scratch,
@@ -945,7 +978,7 @@ extern "C" int ce_attention_decode_bf16_sink(const void* q, const void* k_pool, 
                                              const int* ctx_len, const int* block_table, int* status, int n_seqs, int nh,
                                              int nkv, int d, int q_stride, int page_size, int max_pages, int num_pages,
                                              int window, float scale, int max_splits, const float* sinks, float out_scale,
-                                             cudaStream_t stream) {
+                                             const float* slopes, cudaStream_t stream) {
     if (n_seqs == 0) return CE_OK;
     if (!q || !k_pool || !v_pool || !out || !scratch || !counters || !positions || !seq_slot || !q_start || !ctx_len || !block_table || !status)
         return ce_fail(CE_ERR_ARG, "ce_attention_decode_bf16: null pointer");
@@ -960,7 +993,7 @@ extern "C" int ce_attention_decode_bf16_sink(const void* q, const void* k_pool, 
     a.status = status; a.nh = nh; a.nkv = nkv; a.d = d; a.q_stride = q_stride; a.page_size = page_size;
     a.max_pages = max_pages; a.num_pages = num_pages; a.window = window;
     a.scale_log2 = scale * 1.4426950408889634f;
-    a.sinks = sinks; a.out_scale = out_scale;
+    a.sinks = sinks; a.out_scale = out_scale; a.slopes = slopes;
     int G = nh / nkv;
     static int use_tma = getenv("CE_ATTN_NO_TMA") ? 0 : 1;
     static int fused = getenv("CE_ATTN_FUSED_MERGE") ? 1 : 0;
@@ -1044,15 +1077,15 @@ extern "C" int ce_attention_decode_bf16_sink(const void* q, const void* k_pool, 
         cfg.numAttrs = n_attr;
         cudaError_t le = cudaSuccess;
         ce_note(a.cluster_merge ? "attention_decode_tma_kernel (merge in the cluster)" : "attention_decode_tma_kernel");
-#define AMT_CASE(DM)                                                                                                   \
-        if (deep3) {                                                                                                   \
-            if ((rc = set_smem(attention_decode_tma_kernel<DM, 3>, tsmem, "ce_attention_decode_bf16"))) return rc;     \
-            le = cudaLaunchKernelEx(&cfg, attention_decode_tma_kernel<DM, 3>, mk, mv, a, box_rows);                    \
-        } else {                                                                                                       \
-            if ((rc = set_smem(attention_decode_tma_kernel<DM, 2>, tsmem, "ce_attention_decode_bf16"))) return rc;     \
-            le = cudaLaunchKernelEx(&cfg, attention_decode_tma_kernel<DM, 2>, mk, mv, a, box_rows);                    \
+#define AMT_LAUNCH(DM, ST, BIAS)                                                                                       \
+        {                                                                                                              \
+            if ((rc = set_smem(attention_decode_tma_kernel<DM, ST, BIAS>, tsmem, "ce_attention_decode_bf16"))) return rc; \
+            le = cudaLaunchKernelEx(&cfg, attention_decode_tma_kernel<DM, ST, BIAS>, mk, mv, a, box_rows);              \
         }
-        if (d == 64) { AMT_CASE(64) } else if (d == 128) { AMT_CASE(128) } else { AMT_CASE(256) }
+        // three stages for heads of up to 128 (deep3), two above
+#define AMT_CASE(DM, ST) if (slopes) AMT_LAUNCH(DM, ST, true) else AMT_LAUNCH(DM, ST, false)
+        if (d == 64) { AMT_CASE(64, 3) } else if (d == 128) { AMT_CASE(128, 3) } else { AMT_CASE(256, 2) }
+#undef AMT_LAUNCH
 #undef AMT_CASE
         if (le != cudaSuccess) return ce_fail(CE_ERR_CUDA, "ce_attention_decode_bf16: %s", cudaGetErrorString(le));
         if ((rc = ce_check_launch("ce_attention_decode_bf16"))) return rc;
@@ -1070,15 +1103,17 @@ extern "C" int ce_attention_decode_bf16_sink(const void* q, const void* k_pool, 
         smem = stage_bytes(d, 2);
         if (comb > smem) smem = comb;
     }
-#define AM_DECODE_CASE(DM)                                                                                        \
-    if (deep) {                                                                                                   \
-        if ((rc = set_smem(attention_decode_kernel<DM, 3>, smem, "ce_attention_decode_bf16"))) return rc;         \
-        { ce_note("attention_decode_kernel"); ce_launch(attention_decode_kernel<DM, 3>, grid, AM_THREADS, smem, stream, a); }                             \
-    } else {                                                                                                      \
-        if ((rc = set_smem(attention_decode_kernel<DM, 2>, smem, "ce_attention_decode_bf16"))) return rc;         \
-        { ce_note("attention_decode_kernel"); ce_launch(attention_decode_kernel<DM, 2>, grid, AM_THREADS, smem, stream, a); }                             \
+#define AM_DECODE_LAUNCH(DM, ST, BIAS)                                                                            \
+    {                                                                                                             \
+        if ((rc = set_smem(attention_decode_kernel<DM, ST, BIAS>, smem, "ce_attention_decode_bf16"))) return rc;  \
+        ce_note("attention_decode_kernel");                                                                       \
+        ce_launch(attention_decode_kernel<DM, ST, BIAS>, grid, AM_THREADS, smem, stream, a);                      \
     }
+#define AM_DECODE_CASE(DM)                                                                                        \
+    if (slopes) { if (deep) AM_DECODE_LAUNCH(DM, 3, true) else AM_DECODE_LAUNCH(DM, 2, true) }                    \
+    else { if (deep) AM_DECODE_LAUNCH(DM, 3, false) else AM_DECODE_LAUNCH(DM, 2, false) }
     if (d <= 64) { AM_DECODE_CASE(64) } else if (d <= 128) { AM_DECODE_CASE(128) } else { AM_DECODE_CASE(256) }
+#undef AM_DECODE_LAUNCH
 #undef AM_DECODE_CASE
     if ((rc = ce_check_launch("ce_attention_decode_bf16"))) return rc;
     g_decode_launches = a.fused_merge ? 1 : 2;
@@ -1094,7 +1129,7 @@ extern "C" int ce_attention_prefill_bf16_sink(const void* q, const void* k_pool,
                                               const int* ctx_len, const int* block_table, const int* tiles, int* status,
                                               int n_tiles, int nh, int nkv, int d, int q_stride, int page_size,
                                               int max_pages, int num_pages, int window, float scale, const float* sinks,
-                                              float out_scale, cudaStream_t stream);
+                                              float out_scale, const float* slopes, cudaStream_t stream);
 
 extern "C" int ce_attention_prefill_bf16(const void* q, const void* k_pool, const void* v_pool, void* out,
                                          const int* positions, const int* seq_slot, const int* q_start,
@@ -1103,7 +1138,7 @@ extern "C" int ce_attention_prefill_bf16(const void* q, const void* k_pool, cons
                                          int max_pages, int num_pages, int window, float scale, cudaStream_t stream) {
     return ce_attention_prefill_bf16_sink(q, k_pool, v_pool, out, positions, seq_slot, q_start, ctx_len, block_table, tiles, status,
                                           n_tiles, nh, nkv, d, q_stride, page_size, max_pages, num_pages, window, scale, nullptr, 1.0f,
-                                          stream);
+                                          nullptr, stream);
 }
 
 extern "C" int ce_attention_prefill_bf16_sink(const void* q, const void* k_pool, const void* v_pool, void* out,
@@ -1111,7 +1146,7 @@ extern "C" int ce_attention_prefill_bf16_sink(const void* q, const void* k_pool,
                                               const int* ctx_len, const int* block_table, const int* tiles, int* status,
                                               int n_tiles, int nh, int nkv, int d, int q_stride, int page_size,
                                               int max_pages, int num_pages, int window, float scale, const float* sinks,
-                                              float out_scale, cudaStream_t stream) {
+                                              float out_scale, const float* slopes, cudaStream_t stream) {
     if (n_tiles == 0) return CE_OK;
     if (!q || !k_pool || !v_pool || !out || !positions || !seq_slot || !q_start || !ctx_len || !block_table || !tiles || !status)
         return ce_fail(CE_ERR_ARG, "ce_attention_prefill_bf16: null pointer");
@@ -1124,18 +1159,18 @@ extern "C" int ce_attention_prefill_bf16_sink(const void* q, const void* k_pool,
     a.tiles = tiles; a.status = status; a.nh = nh; a.nkv = nkv; a.d = d; a.q_stride = q_stride; a.page_size = page_size;
     a.max_pages = max_pages; a.num_pages = num_pages; a.window = window;
     a.scale_log2 = scale * 1.4426950408889634f;
-    a.sinks = sinks; a.out_scale = out_scale;
+    a.sinks = sinks; a.out_scale = out_scale; a.slopes = slopes;
     dim3 grid(n_tiles, nh);
     size_t smem = stage_bytes(d, AM_PF_STAGES);
-    if (d <= 64) {
-        if ((rc = set_smem(attention_prefill_kernel<64>, smem, "ce_attention_prefill_bf16"))) return rc;
-        { ce_note("attention_prefill_kernel"); ce_launch(attention_prefill_kernel<64>, grid, AM_THREADS, smem, stream, a); }
-    } else if (d <= 128) {
-        if ((rc = set_smem(attention_prefill_kernel<128>, smem, "ce_attention_prefill_bf16"))) return rc;
-        { ce_note("attention_prefill_kernel"); ce_launch(attention_prefill_kernel<128>, grid, AM_THREADS, smem, stream, a); }
-    } else {
-        if ((rc = set_smem(attention_prefill_kernel<256>, smem, "ce_attention_prefill_bf16"))) return rc;
-        { ce_note("attention_prefill_kernel"); ce_launch(attention_prefill_kernel<256>, grid, AM_THREADS, smem, stream, a); }
+#define AM_PREFILL_LAUNCH(DM, BIAS)                                                                               \
+    {                                                                                                             \
+        if ((rc = set_smem(attention_prefill_kernel<DM, BIAS>, smem, "ce_attention_prefill_bf16"))) return rc;    \
+        ce_note("attention_prefill_kernel");                                                                      \
+        ce_launch(attention_prefill_kernel<DM, BIAS>, grid, AM_THREADS, smem, stream, a);                         \
     }
+#define AM_PREFILL_CASE(DM) if (slopes) AM_PREFILL_LAUNCH(DM, true) else AM_PREFILL_LAUNCH(DM, false)
+    if (d <= 64) { AM_PREFILL_CASE(64) } else if (d <= 128) { AM_PREFILL_CASE(128) } else { AM_PREFILL_CASE(256) }
+#undef AM_PREFILL_CASE
+#undef AM_PREFILL_LAUNCH
     return ce_check_launch("ce_attention_prefill_bf16");
 }

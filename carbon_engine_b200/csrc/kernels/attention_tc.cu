@@ -148,9 +148,11 @@ struct TcAttnArgs {
     float scale_log2;
     const float* sinks;         // [nh] or null: exp(sinks[h]) joins head h's denominator, with no key and no value
     float out_scale;            // the stored rows are multiplied by this
+    const float* slopes;        // [nh] or null: slopes[h] * (position - key) is taken off head h's scaled scores
 };
 
-template <int D>
+// BIAS: a penalty that grows with a key's distance (``slopes``), compiled apart so that the plain scores carry nothing of it
+template <int D, bool BIAS>
 __global__ void __launch_bounds__(THREADS) attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
                                                                       const __grid_constant__ CUtensorMap map_k,
                                                                       const __grid_constant__ CUtensorMap map_v, TcAttnArgs a) {
@@ -321,6 +323,8 @@ __global__ void __launch_bounds__(THREADS) attention_prefill_tc_kernel(const __g
         int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;
         uint32_t lane_base = (uint32_t)(quad * 32) << 16;
         float m_run = -INFINITY, l_run = 0.f;
+        const float slope2 = BIAS ? a.slopes[h] * 1.4426950408889634f : 0.f;
+        const float row_scale = BIAS ? 1.0f : a.scale_log2;     // what is left to scale once the penalty is in the scores
         bool ok = true;
         int where = 66;                                        // 66..68: which wait of the softmax warps gave up
         for (int j = 0; j < n_kv; ++j) {
@@ -333,6 +337,11 @@ __global__ void __launch_bounds__(THREADS) attention_prefill_tc_kernel(const __g
             asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
             __syncwarp();
             if (lane == 0) mbar_arrive(&s_free);  // (one arrival per warp) S may be overwritten by the next product
+            if (BIAS) {
+                const float b0 = slope2 * (float)(k0 - pos);
+#pragma unroll
+                for (int i = 0; i < BN; ++i) sv[i] = fmaf(sv[i], a.scale_log2, fmaf(slope2, (float)i, b0));
+            }
             bool full = row_valid && k0 >= lo && k0 + BN - 1 <= pos;
             if (!full) {                          // only tiles on the diagonal, at the window's edge or past the rows
 #pragma unroll
@@ -351,7 +360,7 @@ __global__ void __launch_bounds__(THREADS) attention_prefill_tc_kernel(const __g
             // The running maximum is only a scale: it is raised (and the sums rescaled) when a tile's maximum
             // exceeds it by more than 2^8; below that the probabilities stay within bfloat16's range and the
             // output accumulator is left alone.
-            float m_tile = mx * a.scale_log2;
+            float m_tile = mx * row_scale;
             bool raise = m_tile > m_run + 8.0f || (m_run == -INFINITY && m_tile != -INFINITY);
             float m_new = raise ? m_tile : m_run;
             float m_use = m_new == -INFINITY ? 0.f : m_new;
@@ -360,8 +369,8 @@ __global__ void __launch_bounds__(THREADS) attention_prefill_tc_kernel(const __g
             uint32_t packed[BN / 2];
 #pragma unroll
             for (int i = 0; i < BN; i += 2) {
-                float p0 = ce_exp2_fast(fmaf(sv[i], a.scale_log2, -m_use));
-                float p1 = ce_exp2_fast(fmaf(sv[i + 1], a.scale_log2, -m_use));
+                float p0 = ce_exp2_fast(BIAS ? sv[i] - m_use : fmaf(sv[i], a.scale_log2, -m_use));
+                float p1 = ce_exp2_fast(BIAS ? sv[i + 1] - m_use : fmaf(sv[i + 1], a.scale_log2, -m_use));
                 sum += p0; sum1 += p1;
                 packed[i / 2] = pack2(p0, p1);
             }
@@ -450,16 +459,16 @@ int get_map(const void* ptr, long long rows, long long cols, long long ld, int b
     return ce_tensor_map_bf16(ptr, rows, cols, ld, box_rows, out, "ce_attention_prefill_tc");
 }
 
-template <int D>
+template <int D, bool BIAS>
 int launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const TcAttnArgs& a, dim3 grid, cudaStream_t stream) {
     size_t smem = (size_t)BM * D * 2 + STAGES * 2 * BN * D * 2 + BM * BN * 2 + 192;    // tiles + barriers
     static bool attr_set = false;
     if (!attr_set) {
-        cudaError_t e = cudaFuncSetAttribute(attention_prefill_tc_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaError_t e = cudaFuncSetAttribute(attention_prefill_tc_kernel<D, BIAS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return ce_fail(CE_ERR_CUDA, "ce_attention_prefill_tc: %s", cudaGetErrorString(e));
         attr_set = true;
     }
-    { ce_note("attention_prefill_tc_kernel"); ce_launch(attention_prefill_tc_kernel<D>, grid, THREADS, smem, stream, mq, mk, mv, a); }
+    { ce_note("attention_prefill_tc_kernel"); ce_launch(attention_prefill_tc_kernel<D, BIAS>, grid, THREADS, smem, stream, mq, mk, mv, a); }
     return ce_check_launch("ce_attention_prefill_tc");
 }
 
@@ -475,7 +484,8 @@ extern "C" int ce_attention_prefill_tc_sink(const void* q, const void* k_pool, c
                                             const int* q_start, const int* ctx_len, const int* block_table, const int* tiles,
                                             int* status, int n_tiles, int total_tokens, int nh, int nkv, int d, int q_stride,
                                             int page_size, int max_pages, int num_pages, int window, float scale,
-                                            const float* sinks, float out_scale, cudaStream_t stream);
+                                            const float* sinks, float out_scale, const float* slopes,
+                                            cudaStream_t stream);
 
 extern "C" int ce_attention_prefill_tc(const void* q, const void* k_pool, const void* v_pool, void* out, const int* seq_slot,
                                        const int* q_start, const int* ctx_len, const int* block_table, const int* tiles,
@@ -484,15 +494,17 @@ extern "C" int ce_attention_prefill_tc(const void* q, const void* k_pool, const 
                                        cudaStream_t stream) {
     return ce_attention_prefill_tc_sink(q, k_pool, v_pool, out, seq_slot, q_start, ctx_len, block_table, tiles, status, n_tiles,
                                         total_tokens, nh, nkv, d, q_stride, page_size, max_pages, num_pages, window, scale, nullptr,
-                                        1.0f, stream);
+                                        1.0f, nullptr, stream);
 }
 
-// ``sinks`` (float32 [nh] or null) and ``out_scale``: see ce_softmax_inverse.
+// ``sinks`` (float32 [nh] or null) and ``out_scale``: see ce_softmax_inverse.  ``slopes`` (float32 [nh] or null): a penalty per head
+// and token of distance.
 extern "C" int ce_attention_prefill_tc_sink(const void* q, const void* k_pool, const void* v_pool, void* out, const int* seq_slot,
                                             const int* q_start, const int* ctx_len, const int* block_table, const int* tiles,
                                             int* status, int n_tiles, int total_tokens, int nh, int nkv, int d, int q_stride,
                                             int page_size, int max_pages, int num_pages, int window, float scale,
-                                            const float* sinks, float out_scale, cudaStream_t stream) {
+                                            const float* sinks, float out_scale, const float* slopes,
+                                            cudaStream_t stream) {
     if (n_tiles == 0) return CE_OK;
     if (!q || !k_pool || !v_pool || !out || !seq_slot || !q_start || !ctx_len || !block_table || !tiles || !status)
         return ce_fail(CE_ERR_ARG, "ce_attention_prefill_tc: null pointer");
@@ -511,8 +523,9 @@ extern "C" int ce_attention_prefill_tc_sink(const void* q, const void* k_pool, c
     int shift = 0;
     while ((1 << shift) < page_size) ++shift;
     TcAttnArgs a{(__nv_bfloat16*)out, seq_slot, q_start, ctx_len, block_table, tiles, status, nh, nkv, page_size, shift,
-                 max_pages, num_pages, window, scale * 1.4426950408889634f, sinks, out_scale};
+                 max_pages, num_pages, window, scale * 1.4426950408889634f, sinks, out_scale, slopes};
     if (n_tiles > 65535) return ce_fail(CE_ERR_SIZE, "ce_attention_prefill_tc: %d tiles of 128 tokens in one step", n_tiles);
     dim3 grid(nh, n_tiles);
-    return d == 64 ? launch<64>(mq, mk, mv, a, grid, stream) : launch<128>(mq, mk, mv, a, grid, stream);
+    if (slopes) return d == 64 ? launch<64, true>(mq, mk, mv, a, grid, stream) : launch<128, true>(mq, mk, mv, a, grid, stream);
+    return d == 64 ? launch<64, false>(mq, mk, mv, a, grid, stream) : launch<128, false>(mq, mk, mv, a, grid, stream);
 }

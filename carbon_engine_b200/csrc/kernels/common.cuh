@@ -86,6 +86,10 @@ __device__ __forceinline__ float ce_clamp_glu_fast(float g, float u, float limit
     return __fdividef(g, 1.0f + __expf(-alpha * g)) * (u + 1.0f);
 }
 
+// silu(gate) * up, exact and for results that are rounded to bfloat16 right after
+__device__ __forceinline__ float ce_silu_glu(float g, float u) { return g / (1.0f + expf(-g)) * u; }
+__device__ __forceinline__ float ce_silu_glu_fast(float g, float u) { return __fdividef(g, 1.0f + __expf(-g)) * u; }
+
 template <typename T> struct CeType;
 template <> struct CeType<float> {
     static __device__ __forceinline__ float load(const float* p) { return *p; }

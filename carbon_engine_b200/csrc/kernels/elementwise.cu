@@ -40,6 +40,42 @@ extern "C" int ce_embed(const void* table, int dtype, const int* tokens, float* 
 }
 
 // ---------------------------------------------------------------------------------------------
+// Embedding gather with a norm: x[t, :] = v / sqrt(mean(v^2) + eps) * w,  v = table[tok[t], :] * scale.  xb (or null) receives
+// the row rounded to bfloat16 too, for a sublayer that reads the residual itself.
+// ---------------------------------------------------------------------------------------------
+template <typename T>
+__global__ void embed_norm_kernel(const T* __restrict__ table, const int* __restrict__ tokens, const float* __restrict__ w,
+                                  float* __restrict__ x, __nv_bfloat16* __restrict__ xb, int H, int V, int* status, float scale, float eps) {
+    ce_pdl_begin();
+    __shared__ float scratch[32];
+    int t = blockIdx.x, tok = tokens[t];
+    const bool there = tok >= 0 && tok < V;
+    if (!there && threadIdx.x == 0) atomicExch(status, 1);
+    const T* row = table + (size_t)(there ? tok : 0) * H;
+    float ss = 0.f;
+    for (int j = threadIdx.x; j < H; j += blockDim.x) { float v = CeType<T>::load(row + j) * scale; ss = fmaf(v, v, ss); }
+    float inv = 1.0f / sqrtf(ce_block_sum(ss, scratch) / (float)H + eps);
+    for (int j = threadIdx.x; j < H; j += blockDim.x) {
+        float v = there ? CeType<T>::load(row + j) * scale * inv * w[j] : 0.f;
+        x[(size_t)t * H + j] = v;
+        if (xb) xb[(size_t)t * H + j] = __float2bfloat16_rn(v);
+    }
+}
+
+extern "C" int ce_embed_norm(const void* table, int dtype, const int* tokens, const float* w, float* x, void* xb, int T, int H, int V,
+                             int* status, float scale, float eps, cudaStream_t stream) {
+    if (T == 0) return CE_OK;
+    if (!table || !tokens || !w || !x || !status) return ce_fail(CE_ERR_ARG, "ce_embed_norm: null pointer");
+    if (H <= 0 || V <= 0) return ce_fail(CE_ERR_SIZE, "ce_embed_norm: width %d, vocabulary %d", H, V);
+    int threads = H >= 1024 ? 1024 : 256;
+    ce_note("embed_norm_kernel");
+    if (dtype == CE_F32) ce_launch(embed_norm_kernel<float>, T, threads, 0, stream, (const float*)table, tokens, w, x, (__nv_bfloat16*)xb, H, V, status, scale, eps);
+    else if (dtype == CE_BF16) ce_launch(embed_norm_kernel<__nv_bfloat16>, T, threads, 0, stream, (const __nv_bfloat16*)table, tokens, w, x, (__nv_bfloat16*)xb, H, V, status, scale, eps);
+    else return ce_fail(CE_ERR_ARG, "ce_embed_norm: unknown dtype %d", dtype);
+    return ce_check_launch("ce_embed_norm");
+}
+
+// ---------------------------------------------------------------------------------------------
 // RMSNorm over the last dimension: out[r, :] = x[row(r), :] * (1/sqrt(mean(x^2) + eps)) * w
 // One block of 256 threads per row, so the order of the sum depends on the width only.
 // ---------------------------------------------------------------------------------------------

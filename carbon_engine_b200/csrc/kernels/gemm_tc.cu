@@ -559,8 +559,8 @@ __global__ void __launch_bounds__(THREADS, 2) gemm_tc_kernel(const __grid_consta
 // A block takes 128 output features of one tile: the same roles and pipeline as the kernel above, without split-K.
 // Where N is no multiple of 128 the last box of an expert reaches into the next expert's rows (or past the stack's
 // end, which reads zeros): those features are not stored.  Without tables it is one expert's product over the rows as
-// they lie.  Epilogue: store in bfloat16, optionally the square of relu first, or (act 2) the clamped gated activation of row
-// pairs: an expert's rows are then gate and up rows by turns (row 2j the gate of feature j, row 2j + 1 its up), neighbouring lanes
+// they lie.  Epilogue: store in bfloat16, optionally the square of relu first, or (act 2, 3) a gated activation of row
+// pairs, the clamped one or silu(gate) up: an expert's rows are then gate and up rows by turns (row 2j the gate of feature j, row 2j + 1 its up), neighbouring lanes
 // hold a feature's two values, and N / 2 features are stored.
 // ---------------------------------------------------------------------------------------------
 struct TcGroupArgs {
@@ -568,7 +568,7 @@ struct TcGroupArgs {
     const int* tile_expert;      // [tiles] or null
     const int* n_tiles;          // [1] or null
     int* status;
-    int rows, N, K, ldo, kblocks, act;       // act 1: relu(v)^2; 2: the clamped gated activation of row pairs
+    int rows, N, K, ldo, kblocks, act;       // act 1: relu(v)^2; 2: the clamped gated activation of row pairs; 3: silu(gate) up of row pairs
     float limit, alpha;
 };
 
@@ -686,7 +686,7 @@ __global__ void __launch_bounds__(THREADS, 2) gemm_tc_grouped_kernel(const __gri
 #pragma unroll
                     for (int j = 0; j < 16; ++j) g[j] = 0.f;
                 }
-                if (a.act == 2) {
+                if (a.act >= 2) {
                     // the lane of the gate row takes tokens 0..7 of the chunk and needs their up values, the lane of the up row
                     // tokens 8..15 and needs their gate values
                     const bool up_row = n & 1;
@@ -696,7 +696,8 @@ __global__ void __launch_bounds__(THREADS, 2) gemm_tc_grouped_kernel(const __gri
                     for (int j = 0; j < 8; ++j) {
                         float other = __shfl_xor_sync(0xffffffffu, up_row ? g[j] : g[8 + j], 1);
                         float gate = up_row ? other : g[j], up = up_row ? g[8 + j] : other;
-                        if (n < a.N && c + t0 + j < m_valid) op[(size_t)j * a.ldo] = __float2bfloat16_rn(ce_clamp_glu_fast(gate, up, a.limit, a.alpha));
+                        float v = a.act == 3 ? ce_silu_glu_fast(gate, up) : ce_clamp_glu_fast(gate, up, a.limit, a.alpha);
+                        if (n < a.N && c + t0 + j < m_valid) op[(size_t)j * a.ldo] = __float2bfloat16_rn(v);
                     }
                 } else if (n < a.N) {
                     __nv_bfloat16* op = a.out + (size_t)(m0 + c) * a.ldo + n;
@@ -1454,15 +1455,15 @@ extern "C" int ce_gemm_tc_grouped_supported(int tile, int N, int K, int ldi, int
 
 // x [x_rows, ldi] bf16, W [experts, N, K] bf16, out [>= rows, ldo] bf16.  With the layout's tables (tile_expert [max_tiles],
 // n_tiles [1], both on the device) tile j of `tile` rows is expert tile_expert[j]'s and rows = max_tiles * tile; without
-// them it is expert 0's product over `rows` rows.  act: 0 none, 1 the square of relu, 2 the clamped gated activation of row pairs
-// (N even; N / 2 columns are stored).
+// them it is expert 0's product over `rows` rows.  act: 0 none, 1 the square of relu, 2 the clamped gated activation of row pairs,
+// 3 silu(gate) up of row pairs (N even; N / 2 columns are stored).
 extern "C" int ce_gemm_tc_grouped(const void* x, const void* W, void* out, const int* tile_expert, const int* n_tiles, int max_tiles,
                                   int tile, int experts, int N, int K, int ldi, int ldo, int x_rows, int rows, int act, float limit,
                                   float alpha, int* status, cudaStream_t stream) {
     if (max_tiles == 0 || rows == 0 || N == 0) return CE_OK;
     if (!x || !W || !out || !status || (tile_expert == nullptr) != (n_tiles == nullptr))
         return ce_fail(CE_ERR_ARG, "ce_gemm_tc_grouped: null pointer");
-    if (!ce_gemm_tc_grouped_supported(tile, N, K, ldi, ldo) || experts <= 0 || act < 0 || act > 2 || (act == 2 && N % 2))
+    if (!ce_gemm_tc_grouped_supported(tile, N, K, ldi, ldo) || experts <= 0 || act < 0 || act > 3 || (act >= 2 && N % 2))
         return ce_fail(CE_ERR_SIZE, "ce_gemm_tc_grouped: tiles of %d rows, N=%d, K=%d, row stride %d", tile, N, K, ldi);
     if (((uintptr_t)x | (uintptr_t)W) & 15) return ce_fail(CE_ERR_SIZE, "ce_gemm_tc_grouped: operands must be 16-byte aligned");
     if (max_tiles > 65535 || (long long)experts * N > 2147483647LL || (long long)max_tiles * tile > (long long)rows + tile - 1 ||

@@ -1,5 +1,5 @@
-// Layer norm with weight and bias, an RMS norm that adds into the residual stream, the tanh cap of a row of
-// numbers, a copy of a run of float32 columns into the activation dtype, and the gate of a per-token side input.
+// Layer norm with weight and bias, RMS norms that add into the residual stream, the RMS norm of a weighted residual plus a
+// sublayer's output, the tanh cap of a row of numbers, a copy of a run of float32 columns into the activation dtype, and the gate of a per-token side input.
 //
 // All arithmetic is float32; a result is rounded once, at the store.  Sums over a row are taken by one block in
 // an order that depends on the row's width only.
@@ -248,6 +248,153 @@ extern "C" int ce_rmsnorm_add_norm(const float* y, const float* bias, const floa
         else ce_launch(rmsnorm_add_norm_kernel<__nv_bfloat16, false>, T, th, 0, stream, y, bias, w, x, w2, (__nv_bfloat16*)h, H, eps, eps2);
     }
     return ce_check_launch("ce_rmsnorm_add_norm");
+}
+
+// ---------------------------------------------------------------------------------------------
+// The norm after the sum:  z = alpha x[t] + s,  x[t] = z / sqrt(mean(z^2) + eps) * w,  s the sublayer's output,
+//   NM 0  y0[t] (+ bias), as it is
+//   NM 1, 2  c * sum_m y_m[t] / sqrt(mean(y_m[t]^2) + eps_m) * w_m: the outputs of mixers side by side, each normed over the width
+// store_only: s itself is stored in x (or, with alpha 1, added to it) and no norm is taken of the sum.
+// xb (or null) receives the new x rounded to bfloat16.  VEC: float4 accesses, a row in registers.
+// ---------------------------------------------------------------------------------------------
+struct ResidualNormArgs {
+    const float* y[2];
+    const float* wm[2];          // the members' norm weights
+    const float* bias;           // or null (NM 0)
+    const float* w;              // null: store_only
+    float* x;
+    __nv_bfloat16* xb;
+    int H;
+    float alpha, c, eps, eps_m;
+};
+
+template <int NM, bool VEC>
+__global__ void residual_norm_kernel(ResidualNormArgs a) {
+    ce_pdl_begin();
+    __shared__ float scratch[32];
+    const int t = blockIdx.x, tid = threadIdx.x, H = a.H;
+    constexpr int NY = NM == 0 ? 1 : NM;
+    float inv_m[NY];
+    if (VEC) {
+        const int H4 = H >> 2;
+        float4* xr = reinterpret_cast<float4*>(a.x + (size_t)t * H);
+        float4 z[LNV_MAX], v[NY][LNV_MAX];
+#pragma unroll
+        for (int m = 0; m < NY; ++m)
+#pragma unroll
+            for (int n = 0; n < LNV_MAX; ++n) {
+                int j = tid + n * blockDim.x;
+                v[m][n] = j < H4 ? reinterpret_cast<const float4*>(a.y[m] + (size_t)t * H)[j] : make_float4(0.f, 0.f, 0.f, 0.f);
+            }
+#pragma unroll
+        for (int n = 0; n < LNV_MAX; ++n) {
+            int j = tid + n * blockDim.x;
+            z[n] = j < H4 && a.alpha != 0.f ? xr[j] : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+        if (NM > 0) {
+#pragma unroll
+            for (int m = 0; m < NY; ++m) {
+                float q = 0.f;
+#pragma unroll
+                for (int n = 0; n < LNV_MAX; ++n) q += (v[m][n].x * v[m][n].x + v[m][n].y * v[m][n].y) + (v[m][n].z * v[m][n].z + v[m][n].w * v[m][n].w);
+                inv_m[m] = 1.0f / sqrtf(ce_block_sum(q, scratch) / (float)H + a.eps_m);
+            }
+        }
+        float q = 0.f;
+#pragma unroll
+        for (int n = 0; n < LNV_MAX; ++n) {
+            int j = tid + n * blockDim.x;
+            if (j >= H4) continue;
+            float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (NM == 0) {
+                s = v[0][n];
+                if (a.bias) { float4 b = reinterpret_cast<const float4*>(a.bias)[j]; s.x += b.x; s.y += b.y; s.z += b.z; s.w += b.w; }
+            } else {
+#pragma unroll
+                for (int m = 0; m < NY; ++m) {
+                    float4 ww = reinterpret_cast<const float4*>(a.wm[m])[j];
+                    s.x += v[m][n].x * inv_m[m] * ww.x; s.y += v[m][n].y * inv_m[m] * ww.y;
+                    s.z += v[m][n].z * inv_m[m] * ww.z; s.w += v[m][n].w * inv_m[m] * ww.w;
+                }
+                s.x *= a.c; s.y *= a.c; s.z *= a.c; s.w *= a.c;
+            }
+            z[n].x = fmaf(a.alpha, z[n].x, s.x); z[n].y = fmaf(a.alpha, z[n].y, s.y);
+            z[n].z = fmaf(a.alpha, z[n].z, s.z); z[n].w = fmaf(a.alpha, z[n].w, s.w);
+            q += (z[n].x * z[n].x + z[n].y * z[n].y) + (z[n].z * z[n].z + z[n].w * z[n].w);
+        }
+        float inv = 1.0f;
+        if (a.w) inv = 1.0f / sqrtf(ce_block_sum(q, scratch) / (float)H + a.eps);
+#pragma unroll
+        for (int n = 0; n < LNV_MAX; ++n) {
+            int j = tid + n * blockDim.x;
+            if (j >= H4) continue;
+            if (a.w) {
+                float4 ww = reinterpret_cast<const float4*>(a.w)[j];
+                z[n].x *= inv * ww.x; z[n].y *= inv * ww.y; z[n].z *= inv * ww.z; z[n].w *= inv * ww.w;
+            }
+            xr[j] = z[n];
+            if (a.xb) {
+                __nv_bfloat162 lo = __floats2bfloat162_rn(z[n].x, z[n].y), hi = __floats2bfloat162_rn(z[n].z, z[n].w);
+                reinterpret_cast<uint2*>(a.xb + (size_t)t * H)[j] = make_uint2(*reinterpret_cast<unsigned*>(&lo), *reinterpret_cast<unsigned*>(&hi));
+            }
+        }
+    } else {
+        float* xr = a.x + (size_t)t * H;
+        if (NM > 0) {
+#pragma unroll
+            for (int m = 0; m < NY; ++m) {
+                float q = 0.f;
+                for (int j = tid; j < H; j += blockDim.x) { float e = a.y[m][(size_t)t * H + j]; q = fmaf(e, e, q); }
+                inv_m[m] = 1.0f / sqrtf(ce_block_sum(q, scratch) / (float)H + a.eps_m);
+            }
+        }
+        float q = 0.f;
+        for (int j = tid; j < H; j += blockDim.x) {
+            float s = 0.f;
+            if (NM == 0) s = a.y[0][(size_t)t * H + j] + (a.bias ? a.bias[j] : 0.f);
+            else {
+#pragma unroll
+                for (int m = 0; m < NY; ++m) s += a.y[m][(size_t)t * H + j] * inv_m[m] * a.wm[m][j];
+                s *= a.c;
+            }
+            float z = a.alpha != 0.f ? fmaf(a.alpha, xr[j], s) : s;
+            xr[j] = z;
+            q = fmaf(z, z, q);
+        }
+        float inv = 1.0f;
+        if (a.w) inv = 1.0f / sqrtf(ce_block_sum(q, scratch) / (float)H + a.eps);
+        for (int j = tid; j < H; j += blockDim.x) {              // (its own writes)
+            float z = a.w ? xr[j] * (inv * a.w[j]) : xr[j];
+            xr[j] = z;
+            if (a.xb) a.xb[(size_t)t * H + j] = __float2bfloat16_rn(z);
+        }
+    }
+}
+
+template <int NM>
+static void residual_norm_launch(const ResidualNormArgs& a, int T, bool vec, cudaStream_t stream) {
+    int H4 = a.H / 4, vt = H4 >= 2048 ? 1024 : H4 >= 512 ? 512 : H4 >= 256 ? 256 : 128;
+    if (vec && H4 <= vt * LNV_MAX) ce_launch(residual_norm_kernel<NM, true>, T, vt, 0, stream, a);
+    else ce_launch(residual_norm_kernel<NM, false>, T, a.H >= 4096 ? 512 : a.H >= 1024 ? 256 : 128, 0, stream, a);
+}
+
+// members 0: y0 is the sublayer's output as it is (wm0, wm1, y1 null); 1 or 2: y0 (and y1) are normed with wm0 (wm1) and eps_m,
+// their sum multiplied by c.  w null: the sum is stored without a norm (alpha 0: over what x held).
+extern "C" int ce_residual_norm(const float* y0, const float* y1, const float* wm0, const float* wm1, int members, const float* bias,
+                                const float* w, float* x, void* xb, int T, int H, float alpha, float c, float eps, float eps_m,
+                                cudaStream_t stream) {
+    if (T == 0) return CE_OK;
+    if (!y0 || !x || members < 0 || members > 2 || (members > 0 && !wm0) || (members > 1 && (!wm1 || !y1)) || (members > 0 && bias))
+        return ce_fail(CE_ERR_ARG, "ce_residual_norm: null pointer, or %d members", members);
+    if (H <= 0) return ce_fail(CE_ERR_SIZE, "ce_residual_norm: width %d", H);
+    ResidualNormArgs a{{y0, y1}, {wm0, wm1}, bias, w, x, (__nv_bfloat16*)xb, H, alpha, c, eps, eps_m};
+    bool vec = H % 4 == 0 && H >= 256 && ((((uintptr_t)y0 | (uintptr_t)y1 | (uintptr_t)wm0 | (uintptr_t)wm1 | (uintptr_t)bias |
+                                            (uintptr_t)w | (uintptr_t)x | (uintptr_t)xb) & 15) == 0);
+    ce_note("residual_norm_kernel");
+    if (members == 0) residual_norm_launch<0>(a, T, vec, stream);
+    else if (members == 1) residual_norm_launch<1>(a, T, vec, stream);
+    else residual_norm_launch<2>(a, T, vec, stream);
+    return ce_check_launch("ce_residual_norm");
 }
 
 // xb (or null): receives the new x rounded to bfloat16, what a sublayer that reads the residual itself takes as its input

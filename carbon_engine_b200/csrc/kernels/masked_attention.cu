@@ -1,6 +1,6 @@
 // Softmax attention over the paged cache with the options that several designs combine differently, each a
-// parameter: key and value heads of different sizes, a tanh cap on the scores, a sliding window that may keep a
-// sequence's first tokens visible, a sigmoid gate per output element, and a value pool that is a view of the key
+// parameter: key and value heads of different sizes, a tanh cap on the scores, a penalty per head that grows with a key's
+// distance, a sliding window that may keep a sequence's first tokens visible, a sigmoid gate per output element, and a value pool that is a view of the key
 // pool (latent attention keeps ONE row per token, of which the values are the leading part).  Float32 arithmetic,
 // any number of new tokens per sequence; it is the float32 path and the plain twin of the tensor-core kernel.
 //
@@ -42,14 +42,23 @@ extern "C" int ce_value_mix(void* rows, int dtype, int stride, int off, int n, c
     return ce_check_launch("ce_value_mix");
 }
 
+// Element i of a part of which the first rd elements turn (i < rd): its partner, and the index of its angle.
+__device__ __forceinline__ void rope_pair(int i, int half, int pairing, int& partner, int& angle, bool& first) {
+    if (pairing) { partner = i ^ 1; angle = i >> 1; first = (i & 1) == 0; }
+    else { first = i < half; partner = first ? i + half : i - half; angle = first ? i : i - half; }
+}
+
 // ---------------------------------------------------------------------------------------------
 // Operands of attention with a norm per head: proj [T, ld] float32 holds, per token, nh query heads of d from off_q, nkv key
-// heads of d from off_k and nkv value heads of dv from off_v.  Each query and key head is divided by its root mean square and
-// multiplied by a weight of size d (wq, wk; null: no norm), then rotated over its first rd elements (element i with
-// i + rd/2) by the token's position; query head h is also multiplied by head_scale[h] (a temperature per head folded into
-// the query; null: none).  Queries go to q_out [T, nh * d], keys and values to the token's place in the pools.  The values
-// may be the keys as projected (off_v = off_k, dv = d): they are read before the norm and the rotation.
-// A warp per head in turn.
+// heads of d from off_k and nkv value heads of dv from off_v.  Of each query and key head the first rd elements are rotated by
+// the token's position (pairing 0: element i with i + rd/2; 1: element 2i with 2i + 1), and the head is normed:
+//   norm_mode 0  no norm
+//   norm_mode 1  divided by its root mean square and multiplied by a weight of size d (wq, wk), then rotated
+//   norm_mode 2  rotated, then divided by its root mean square (and, where given, multiplied by the weight)
+// Query head h is also multiplied by head_scale[h] and by pos_scale[position] (a temperature per head and one per position,
+// folded into the query; null: none).  Queries go to q_out [T, nh * d], keys and values to the token's place in the pools.  The
+// values may be the keys as projected (off_v = off_k, dv = d): they are read before the norm and the rotation.
+// A warp per head in turn, a head's elements in registers (NV a lane).
 // ---------------------------------------------------------------------------------------------
 struct NormRopeArgs {
     const float* proj;
@@ -59,6 +68,7 @@ struct NormRopeArgs {
     const float* wq;
     const float* wk;
     const float* head_scale;
+    const float* pos_scale;      // [max_pos_scale] or null
     const float* cos_table;      // [max_pos, rd/2] or null
     const float* sin_table;
     const int* positions;
@@ -68,9 +78,10 @@ struct NormRopeArgs {
     int* status;
     int ld, off_q, off_k, off_v, nh, nkv, d, dv, rd, page_size, max_pages, num_pages, max_pos, write_kv;
     float eps;
+    int norm_mode, pairing, max_pos_scale;
 };
 
-template <typename T>
+template <typename T, int NV>
 __global__ void norm_rope_kvwrite_kernel(NormRopeArgs a) {
     ce_pdl_begin();
     int t = blockIdx.x, lane = threadIdx.x & 31, nwarp = (blockDim.x >> 5) * gridDim.y;
@@ -79,9 +90,9 @@ __global__ void norm_rope_kvwrite_kernel(NormRopeArgs a) {
     int p = a.positions[t];
     const float* row = a.proj + (size_t)t * a.ld;
     bool rotate = a.cos_table != nullptr && half > 0;
-    if (rotate && (p < 0 || p >= a.max_pos)) {
+    if ((rotate && (p < 0 || p >= a.max_pos)) || (a.pos_scale && (p < 0 || p >= a.max_pos_scale))) {
         if (threadIdx.x == 0) atomicExch(a.status, 3);
-        rotate = false;
+        return;
     }
     int page = -1, off = 0;
     if (a.write_kv) {
@@ -95,33 +106,59 @@ __global__ void norm_rope_kvwrite_kernel(NormRopeArgs a) {
     }
     const float* cs = rotate ? a.cos_table + (size_t)p * half : nullptr;
     const float* sn = rotate ? a.sin_table + (size_t)p * half : nullptr;
+    const float ps = a.pos_scale ? a.pos_scale[p] : 1.0f;
     for (int hh = warp; hh < a.nh + a.nkv; hh += nwarp) {
         bool is_q = hh < a.nh;
         const float* src = row + (is_q ? a.off_q + hh * d : a.off_k + (hh - a.nh) * d);
-        const float* w = is_q ? a.wq : a.wk;
+        const float* w = a.norm_mode ? (is_q ? a.wq : a.wk) : nullptr;
         T* dst;
         if (is_q) dst = (T*)a.q_out + ((size_t)t * a.nh + hh) * d;
         else {
             if (page < 0) continue;
             dst = (T*)a.k_pool + (((size_t)page * a.nkv + (hh - a.nh)) * a.page_size + off) * d;
         }
+        float v[NV];
+#pragma unroll
+        for (int n = 0; n < NV; ++n) { int j = lane + 32 * n; v[n] = j < d ? src[j] : 0.f; }
         float inv = 1.0f;
-        if (w) {
+        if (a.norm_mode == 1) {
             float ss = 0.f;
-            for (int j = lane; j < d; j += 32) ss = fmaf(src[j], src[j], ss);
+#pragma unroll
+            for (int n = 0; n < NV; ++n) ss = fmaf(v[n], v[n], ss);
             for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
             inv = 1.0f / sqrtf(ss / (float)d + a.eps);
+#pragma unroll
+            for (int n = 0; n < NV; ++n) { int j = lane + 32 * n; if (j < d) v[n] = v[n] * inv * w[j]; }
         }
-        float hs = is_q && a.head_scale ? a.head_scale[hh] : 1.0f;
-        for (int j = lane; j < d; j += 32) {
-            float x = w ? src[j] * inv * w[j] : src[j];
-            if (rotate && j < a.rd) {
-                int partner = j < half ? j + half : j - half;
-                float y = w ? src[partner] * inv * w[partner] : src[partner];
-                x = j < half ? x * cs[j] - y * sn[j] : x * cs[j - half] + y * sn[j - half];
+        if (rotate) {
+#pragma unroll
+            for (int n = 0; n < NV; ++n) {
+                int j = lane + 32 * n;
+                if (32 * n >= a.rd) break;                    // (the same for every lane)
+                float y = 0.f;
+                if (a.pairing) y = __shfl_xor_sync(0xffffffffu, v[n], 1);
+                if (j < a.rd) {
+                    int partner, angle;
+                    bool first;
+                    rope_pair(j, half, a.pairing, partner, angle, first);
+                    if (!a.pairing) y = a.norm_mode == 1 ? src[partner] * inv * w[partner] : src[partner];
+                    float c = cs[angle], s = sn[angle];
+                    v[n] = first ? v[n] * c - y * s : v[n] * c + y * s;
+                }
             }
-            CeType<T>::store(dst + j, x * hs);
         }
+        if (a.norm_mode == 2) {
+            float ss = 0.f;
+#pragma unroll
+            for (int n = 0; n < NV; ++n) ss = fmaf(v[n], v[n], ss);
+            for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+            inv = 1.0f / sqrtf(ss / (float)d + a.eps);
+#pragma unroll
+            for (int n = 0; n < NV; ++n) { int j = lane + 32 * n; if (j < d) v[n] = w ? v[n] * inv * w[j] : v[n] * inv; }
+        }
+        float hs = is_q ? (a.head_scale ? a.head_scale[hh] * ps : ps) : 1.0f;
+#pragma unroll
+        for (int n = 0; n < NV; ++n) { int j = lane + 32 * n; if (j < d) CeType<T>::store(dst + j, v[n] * hs); }
     }
     if (page >= 0) {
         for (int e = blockIdx.y * blockDim.x + threadIdx.x; e < a.nkv * a.dv; e += blockDim.x * gridDim.y) {
@@ -131,21 +168,31 @@ __global__ void norm_rope_kvwrite_kernel(NormRopeArgs a) {
     }
 }
 
+template <typename T>
+static void norm_rope_launch(const NormRopeArgs& a, dim3 grid, int threads, cudaStream_t stream) {
+    if (a.d <= 64) ce_launch(norm_rope_kvwrite_kernel<T, 2>, grid, threads, 0, stream, a);
+    else if (a.d <= 128) ce_launch(norm_rope_kvwrite_kernel<T, 4>, grid, threads, 0, stream, a);
+    else if (a.d <= 256) ce_launch(norm_rope_kvwrite_kernel<T, 8>, grid, threads, 0, stream, a);
+    else ce_launch(norm_rope_kvwrite_kernel<T, 64>, grid, threads, 0, stream, a);
+}
+
 extern "C" int ce_norm_rope_kvwrite(const float* proj, void* q_out, void* k_pool, void* v_pool, int dtype, const float* wq,
-                                    const float* wk, const float* head_scale, const float* cos_table, const float* sin_table,
-                                    const int* positions, const int* seq_of_token, const int* seq_slot, const int* block_table,
-                                    int* status, int T, int ld, int off_q, int off_k, int off_v, int nh, int nkv, int d, int dv, int rd,
-                                    int page_size, int max_pages, int num_pages, int max_pos, int write_kv, float eps,
-                                    cudaStream_t stream) {
+                                    const float* wk, const float* head_scale, const float* pos_scale, const float* cos_table,
+                                    const float* sin_table, const int* positions, const int* seq_of_token, const int* seq_slot,
+                                    const int* block_table, int* status, int T, int ld, int off_q, int off_k, int off_v, int nh, int nkv,
+                                    int d, int dv, int rd, int page_size, int max_pages, int num_pages, int max_pos, int write_kv,
+                                    float eps, int norm_mode, int pairing, int max_pos_scale, cudaStream_t stream) {
     if (T == 0) return CE_OK;
     if (!proj || !q_out || !positions || !seq_of_token || !seq_slot || !status) return ce_fail(CE_ERR_ARG, "ce_norm_rope_kvwrite: null pointer");
     if (write_kv && (!k_pool || !v_pool || !block_table)) return ce_fail(CE_ERR_ARG, "ce_norm_rope_kvwrite: no cache to write to");
     if (rd < 0 || rd > d || rd % 2) return ce_fail(CE_ERR_SIZE, "ce_norm_rope_kvwrite: %d rotated elements of %d", rd, d);
     if (rd > 0 && (!cos_table || !sin_table)) return ce_fail(CE_ERR_ARG, "ce_norm_rope_kvwrite: no rotation tables");
-    if (nh <= 0 || nkv <= 0 || d <= 0 || dv <= 0) return ce_fail(CE_ERR_SIZE, "ce_norm_rope_kvwrite: sizes");
-    NormRopeArgs a{proj, q_out, k_pool, v_pool, wq, wk, head_scale, rd > 0 ? cos_table : nullptr, sin_table, positions, seq_of_token,
-                   seq_slot, block_table, status, ld, off_q, off_k, off_v, nh, nkv, d, dv, rd, page_size, max_pages, num_pages, max_pos,
-                   write_kv, eps};
+    if (nh <= 0 || nkv <= 0 || d <= 0 || d > 2048 || dv <= 0) return ce_fail(CE_ERR_SIZE, "ce_norm_rope_kvwrite: sizes");
+    if (norm_mode < 0 || norm_mode > 2 || (norm_mode == 1 && (!wq || !wk)) || (pairing != 0 && pairing != 1))
+        return ce_fail(CE_ERR_ARG, "ce_norm_rope_kvwrite: norm mode %d, pairing %d", norm_mode, pairing);
+    NormRopeArgs a{proj, q_out, k_pool, v_pool, wq, wk, head_scale, pos_scale, rd > 0 ? cos_table : nullptr, sin_table, positions,
+                   seq_of_token, seq_slot, block_table, status, ld, off_q, off_k, off_v, nh, nkv, d, dv, rd, page_size, max_pages,
+                   num_pages, max_pos, write_kv, eps, norm_mode, pairing, max_pos_scale};
     // a token's heads are dealt to the warps of gridDim.y blocks in turn: one block a token in a long step, a block per
     // handful of heads in a step of few tokens
     int heads = nh + nkv;
@@ -154,8 +201,8 @@ extern "C" int ce_norm_rope_kvwrite(const float* proj, void* q_out, void* k_pool
     int split = want < room ? want : room;
     dim3 grid(T, split < 1 ? 1 : split);
     ce_note("norm_rope_kvwrite_kernel");
-    if (dtype == CE_F32) ce_launch(norm_rope_kvwrite_kernel<float>, grid, threads, 0, stream, a);
-    else if (dtype == CE_BF16) ce_launch(norm_rope_kvwrite_kernel<__nv_bfloat16>, grid, threads, 0, stream, a);
+    if (dtype == CE_F32) norm_rope_launch<float>(a, grid, threads, stream);
+    else if (dtype == CE_BF16) norm_rope_launch<__nv_bfloat16>(a, grid, threads, stream);
     else return ce_fail(CE_ERR_ARG, "ce_norm_rope_kvwrite: unknown dtype %d", dtype);
     return ce_check_launch("ce_norm_rope_kvwrite");
 }
@@ -168,12 +215,6 @@ extern "C" int ce_norm_rope_kvwrite(const float* proj, void* q_out, void* k_pool
 // The rotation turns, of the part's first rd elements, element i with element i + rd/2 (pairing 0) or 2i with 2i + 1 (pairing 1)
 // by angle i of the token's position.
 // ---------------------------------------------------------------------------------------------
-// Element i of a part of which the first rd elements turn (i < rd): its partner, and the index of its angle.
-__device__ __forceinline__ void rope_pair(int i, int half, int pairing, int& partner, int& angle, bool& first) {
-    if (pairing) { partner = i ^ 1; angle = i >> 1; first = (i & 1) == 0; }
-    else { first = i < half; partner = first ? i + half : i - half; angle = first ? i : i - half; }
-}
-
 struct LatentPrepArgs {
     const float* proj;
     const float* wq;             // [qr]
@@ -476,6 +517,7 @@ struct MaskedAttnArgs {
     const int* block_table;
     int* status;
     const float* sinks;          // [nh] or null: exp(sinks[h]) joins the softmax's denominator, with no key and no value
+    const float* slopes;         // [nh] or null: slopes[h] * (position - key) is taken off the (scaled, capped) score
     int T, nh, nkv, d, dv, q_stride, q_head, ldk, ldv, gate_stride, page_size, max_pages, num_pages, window, keep_first;
     float scale, softcap;
     float out_scale;             // the stored result is multiplied by this (the mixer's weight in a sum of mixers)
@@ -502,6 +544,7 @@ __global__ void masked_attention_kernel(MaskedAttnArgs a) {
     int lo = a.window > 0 ? max(0, p - a.window + 1) : 0;
     int keep = a.window > 0 ? a.keep_first : 0;
     float inv_cap = a.softcap > 0.f ? 1.0f / a.softcap : 0.f;
+    const float slope = a.slopes ? a.slopes[h] : 0.f;
     float m_run = -INFINITY, l_run = 0.f;
     float acc[MA_MAX_ACC];
 #pragma unroll
@@ -525,6 +568,7 @@ __global__ void masked_attention_kernel(MaskedAttnArgs a) {
                 for (int j = 0; j < d; ++j) dot = fmaf(qs[j], CeType<T>::load(kr + j), dot);
                 s = dot * a.scale;
                 if (a.softcap > 0.f) s = a.softcap * tanhf(s * inv_cap);
+                s = fmaf(slope, (float)(key - p), s);
             }
         }
         float m_chunk = ce_block_max(s, scratch);
@@ -575,7 +619,8 @@ extern "C" int ce_masked_attention(const void* q, const void* k_pool, const void
                                    const int* positions, const int* seq_of_token, const int* seq_slot, const int* block_table,
                                    int* status, int T, int nh, int nkv, int d, int dv, int q_stride, int q_head, int ldk, int ldv,
                                    int gate_stride, int page_size, int max_pages, int num_pages, int window, int keep_first,
-                                   float scale, float softcap, const float* sinks, float out_scale, cudaStream_t stream) {
+                                   float scale, float softcap, const float* sinks, float out_scale, const float* slopes,
+                                   cudaStream_t stream) {
     if (T == 0) return CE_OK;
     if (!q || !k_pool || !v_pool || !out || !positions || !seq_of_token || !seq_slot || !block_table || !status)
         return ce_fail(CE_ERR_ARG, "ce_masked_attention: null pointer");
@@ -583,7 +628,7 @@ extern "C" int ce_masked_attention(const void* q, const void* k_pool, const void
         return ce_fail(CE_ERR_SIZE, "ce_masked_attention: head sizes %d / %d", d, dv);
     if (nkv <= 0 || nh % nkv != 0) return ce_fail(CE_ERR_SIZE, "ce_masked_attention: %d heads are not a multiple of %d kv heads", nh, nkv);
     if (ldk < d || ldv < dv || nh > 65535) return ce_fail(CE_ERR_SIZE, "ce_masked_attention: a pool's rows are shorter than a head");
-    MaskedAttnArgs a{q, k_pool, v_pool, gate, out, positions, seq_of_token, seq_slot, block_table, status, sinks, T, nh, nkv, d, dv,
+    MaskedAttnArgs a{q, k_pool, v_pool, gate, out, positions, seq_of_token, seq_slot, block_table, status, sinks, slopes, T, nh, nkv, d, dv,
                      q_stride, q_head, ldk, ldv, gate_stride, page_size, max_pages, num_pages, window, keep_first, scale, softcap,
                      out_scale};
     size_t smem = (d + MA_THREADS + 32) * sizeof(float) + MA_THREADS * sizeof(long long);

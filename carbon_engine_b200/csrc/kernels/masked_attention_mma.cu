@@ -1,6 +1,6 @@
 // Softmax attention over the paged cache in bfloat16 on the tensor cores (mma.sync m16n8k16), with the options of
 // masked_attention.cu, whose float32 kernel is its plain twin: key and value heads of different sizes, a tanh cap on the
-// scores, a sliding window that may keep the sequence's first tokens visible, a sigmoid gate per output element, and a
+// scores, a penalty per head that grows with a key's distance, a sliding window that may keep the sequence's first tokens visible, a sigmoid gate per output element, and a
 // value pool that may be the key pool itself (the values are then the leading part of every key row, and the key tile in
 // shared memory serves as the value tile too).
 //
@@ -42,6 +42,7 @@ struct MaskedMmaArgs {
     const int* tiles;            // (sequence, first token of the tile within the sequence's tokens of the step), 64 tokens a tile
     int* status;
     const float* sinks;          // [nh] or null: exp(sinks[h]) joins the softmax's denominator, with no key and no value
+    const float* slopes;         // [nh] or null: slopes[h] * (position - key) is taken off the (scaled, capped) score
     int nh, nkv, d, dv, q_stride, q_head, ldk, ldv, gate_stride, page_size, max_pages, num_pages, window, keep_first;
     int pack;                    // heads of one key head a block takes (a power of two up to 16 that divides nh / nkv)
     int slice;                   // value columns a block takes (a multiple of 16)
@@ -126,6 +127,10 @@ __global__ void __launch_bounds__(MM_THREADS, (DVT <= 16 ? 3 : 2)) masked_attent
     const float log2e = 1.4426950408889634f;
     const float scale2 = a.scale * log2e;
     const float cap2 = a.softcap * log2e, pre_cap = a.softcap > 0.f ? a.scale / a.softcap : 0.f;
+    // with a penalty on distance the scores are scaled (and capped) in a pass of their own, which the others do not run
+    const bool biased = a.slopes != nullptr;
+    const float slope_a = biased ? a.slopes[head0 + ra % pack] * log2e : 0.f, slope_b = biased ? a.slopes[head0 + rb % pack] * log2e : 0.f;
+    const float later_scale = biased ? 1.0f : scale2, later_cap = biased ? 0.f : a.softcap;
 
     auto page_of = [&](int k0, int r) -> int {
         int key = k0 + r;
@@ -196,6 +201,16 @@ __global__ void __launch_bounds__(MM_THREADS, (DVT <= 16 ? 3 : 2)) masked_attent
                     mm_mma(s[nt + 1], qf, b2, b3);
                 }
             }
+            if (biased) {
+#pragma unroll
+                for (int nt = 0; nt < MM_SUB / 8; ++nt)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) {
+                        int key = ks0 + nt * 8 + (lane & 3) * 2 + (e & 1);
+                        float v = a.softcap > 0.f ? cap2 * mm_tanh_fast(s[nt][e] * pre_cap) : s[nt][e] * scale2;
+                        s[nt][e] = fmaf(e < 2 ? slope_a : slope_b, (float)(key - (e < 2 ? pos_a : pos_b)), v);
+                    }
+            }
             // scale (and cap), mask, running maximum
             float mx_a = -INFINITY, mx_b = -INFINITY;
             const bool whole = rows_full && ks0 + MM_SUB - 1 <= warp_pos_first && ks0 >= warp_lo_last;
@@ -209,7 +224,7 @@ __global__ void __launch_bounds__(MM_THREADS, (DVT <= 16 ? 3 : 2)) masked_attent
                         int key = ks0 + nt * 8 + (lane & 3) * 2 + (e & 1);
                         see = upper ? (key <= pos_a && (key >= lo_a || key < keep)) : (key <= pos_b && (key >= lo_b || key < keep));
                     }
-                    float v = a.softcap > 0.f ? cap2 * mm_tanh_fast(s[nt][e] * pre_cap) : s[nt][e] * scale2;
+                    float v = later_cap > 0.f ? cap2 * mm_tanh_fast(s[nt][e] * pre_cap) : s[nt][e] * later_scale;
                     v = see ? v : -INFINITY;
                     s[nt][e] = v;
                     if (upper) mx_a = fmaxf(mx_a, v); else mx_b = fmaxf(mx_b, v);
@@ -443,7 +458,7 @@ extern "C" int ce_masked_attention_mma(const void* q, const void* k_pool, const 
                                        const int* tiles, int* status, int n_tiles, int n_tokens, int nh, int nkv, int d, int dv,
                                        int q_stride, int q_head, int ldk, int ldv, int gate_stride, int page_size, int max_pages,
                                        int num_pages, int window, int keep_first, float scale, float softcap, const float* sinks,
-                                       float out_scale, cudaStream_t stream) {
+                                       float out_scale, const float* slopes, cudaStream_t stream) {
     if (n_tiles == 0) return CE_OK;
     if (!q || !k_pool || !v_pool || !out || !positions || !seq_slot || !q_start || !block_table || !tiles || !status)
         return ce_fail(CE_ERR_ARG, "ce_masked_attention_mma: null pointer");
@@ -470,7 +485,7 @@ extern "C" int ce_masked_attention_mma(const void* q, const void* k_pool, const 
         if (mm_smem_bytes(d, slice, alias, 2) > 200 * 1024) slice = mm_slice(dv, 4);
     }
     MaskedMmaArgs a{(const __nv_bfloat16*)q, (const __nv_bfloat16*)k_pool, (const __nv_bfloat16*)v_pool, (const __nv_bfloat16*)gate,
-                    (__nv_bfloat16*)out, positions, seq_slot, q_start, block_table, tiles, status, sinks, nh, nkv, d, dv, q_stride, q_head,
+                    (__nv_bfloat16*)out, positions, seq_slot, q_start, block_table, tiles, status, sinks, slopes, nh, nkv, d, dv, q_stride, q_head,
                     ldk, ldv, gate_stride, page_size, max_pages, num_pages, window, keep_first, pack, slice, buffers == 4, scale, softcap,
                     out_scale};
     dim3 grid(n_tiles * pack, nh / pack, (dv + slice - 1) / slice);

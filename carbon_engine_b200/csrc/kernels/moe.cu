@@ -1,8 +1,8 @@
 // Mixture of experts: routing, the layout of a step's (token, expert) pairs by expert, the experts' two products as
 // grouped products over that layout, and the weighted sum back into token order.
 //
-//   route    z [T, ld] float32 router logits -> s = softmax(z[:E]) or sigmoid(z[:E]); choice scores c = s (+ a correction per
-//            expert); experts in `groups` equal groups of neighbours, a group's score the largest c in it or the sum of its two
+//   route    z [T, ld] float32 router logits (+ a bias per expert) -> s = softmax(z[:E]) or sigmoid(z[:E]), or, for a softmax over
+//            the chosen logits only, s = exp(z - max z) and choice by z itself; choice scores c = s (+ a correction per expert); experts in `groups` equal groups of neighbours, a group's score the largest c in it or the sum of its two
 //            largest, only the best `keep` groups' experts eligible; the `top` eligible experts with the largest c are chosen
 //            (ties: the lower index); weights s / (sum of the chosen s + 1e-20) * scale, or s * scale as they are.
 //            Column E of z, where there is one, is the logit of a shared expert's gate: sgate[t] = sigmoid(z[t, E]).
@@ -11,8 +11,8 @@
 //            padding row), pair_row[i] the row of pair i, tile_expert[j] the expert of tile j, n_tiles[0] their count.
 //            Nothing of it reaches the host: the products launch a grid for the most tiles a step of that size can have,
 //            and blocks past n_tiles leave at once, so a captured graph replays with any routing.
-//   products out[p] = act(in[row p's token, or p] W[e]^T), e = tile_expert[p / BM]; act = none, relu^2, or the clamped gated
-//            activation of row pairs (rows 2j and 2j + 1 of W[e] are feature j's gate and up).  Every output
+//   products out[p] = act(in[row p's token, or p] W[e]^T), e = tile_expert[p / BM]; act = none, relu^2, or a gated
+//            activation of row pairs (rows 2j and 2j + 1 of W[e] are feature j's gate and up): the clamped one, or silu(gate) up.  Every output
 //            element is a sum over k in a fixed order that depends on neither the row's place in its tile nor on the
 //            other rows, so a token's result does not depend on the batch.  float32 FMA for any size and both dtypes;
 //            bfloat16 on the tensor cores (wmma m16n16k16, float32 sums) for sizes in multiples of 16.
@@ -33,9 +33,10 @@ struct MoeRouteArgs {
     int T, ld, E, top, groups, keep;
     float scale;
     const float* correction;     // [E] or null: added to the scores for the choice, not for the weights
-    int scoring;                 // 0: softmax over the experts, 1: sigmoid
+    int scoring;                 // 0: softmax over the experts, 1: sigmoid, 2: softmax over the chosen logits
     int group_score;             // 0: a group's largest choice score, 1: the sum of its two largest
     int renormalize;             // 1: the weights are divided by the sum of the chosen scores
+    const float* bias;           // [E] or null: added to the logits
 };
 
 __device__ __forceinline__ void moe_warp_argmax(float& v, int& i) {
@@ -56,19 +57,21 @@ __global__ void __launch_bounds__(128) moe_route_kernel(MoeRouteArgs a) {
     float* c = s + a.E;                                      // choice scores; a chosen or barred expert's becomes -inf
     float* gs = c + a.E;                                     // the groups' scores; a kept group's becomes +inf
     const float* zr = a.z + (size_t)t * a.ld;
-    if (a.scoring == 0) {
+    for (int e = lane; e < a.E; e += 32) c[e] = a.bias ? zr[e] + a.bias[e] : zr[e];       // the logits (each lane its own experts')
+    if (a.scoring != 1) {
         float mx = -INFINITY;
-        for (int e = lane; e < a.E; e += 32) mx = fmaxf(mx, zr[e]);
+        for (int e = lane; e < a.E; e += 32) mx = fmaxf(mx, c[e]);
         for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
         float sum = 0.f;
-        for (int e = lane; e < a.E; e += 32) { float v = expf(zr[e] - mx); s[e] = v; sum += v; }
+        for (int e = lane; e < a.E; e += 32) { float v = expf(c[e] - mx); s[e] = v; sum += v; }
         for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
-        const float inv = 1.0f / sum;
+        const float inv = a.scoring == 0 ? 1.0f / sum : 1.0f;
         for (int e = lane; e < a.E; e += 32) s[e] *= inv;
     } else {
-        for (int e = lane; e < a.E; e += 32) s[e] = 1.0f / (1.0f + expf(-zr[e]));
+        for (int e = lane; e < a.E; e += 32) s[e] = 1.0f / (1.0f + expf(-c[e]));
     }
-    for (int e = lane; e < a.E; e += 32) c[e] = a.correction ? s[e] + a.correction[e] : s[e];
+    if (a.scoring != 2)
+        for (int e = lane; e < a.E; e += 32) c[e] = a.correction ? s[e] + a.correction[e] : s[e];
     __syncwarp();
     if (a.groups > 1 && a.keep < a.groups) {
         const int size = a.E / a.groups;
@@ -120,15 +123,17 @@ __global__ void __launch_bounds__(128) moe_route_kernel(MoeRouteArgs a) {
 
 extern "C" int ce_moe_route(const float* z, int* ids, float* weights, float* sgate, int T, int ld, int E, int top, int groups,
                             int keep, float scale, const float* correction, int scoring, int group_score, int renormalize,
-                            cudaStream_t stream) {
+                            const float* bias, cudaStream_t stream) {
     if (T == 0) return CE_OK;
     if (!z || !ids || !weights) return ce_fail(CE_ERR_ARG, "ce_moe_route: null pointer");
     if (E <= 0 || E > MOE_MAX_EXPERTS || top <= 0 || top > E || groups <= 0 || E % groups || keep <= 0 || keep > groups ||
         (long long)keep * (E / groups) < top || ld < E + (sgate ? 1 : 0))
         return ce_fail(CE_ERR_SIZE, "ce_moe_route: %d experts, top %d, %d groups of which %d are kept", E, top, groups, keep);
-    if (scoring < 0 || scoring > 1 || group_score < 0 || group_score > 1)
+    if (scoring == 2 && (correction || !renormalize))
+        return ce_fail(CE_ERR_ARG, "ce_moe_route: a softmax over the chosen logits takes no correction and sums to the scale");
+    if (scoring < 0 || scoring > 2 || group_score < 0 || group_score > 1)
         return ce_fail(CE_ERR_ARG, "ce_moe_route: scoring %d, group score %d", scoring, group_score);
-    MoeRouteArgs a{z, ids, weights, sgate, T, ld, E, top, groups, keep, scale, correction, scoring, group_score, renormalize};
+    MoeRouteArgs a{z, ids, weights, sgate, T, ld, E, top, groups, keep, scale, correction, scoring, group_score, renormalize, bias};
     size_t smem = (size_t)4 * 3 * E * sizeof(float);
     if (smem > 40 * 1024) cudaFuncSetAttribute(moe_route_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     ce_note("moe_route_kernel");
@@ -231,7 +236,8 @@ extern "C" int ce_moe_align(const int* ids, int n_pairs, int top, int E, int BM,
 // ---------------------------------------------------------------------------------------------
 // grouped products
 // ---------------------------------------------------------------------------------------------
-enum { MOE_ACT_NONE = 0, MOE_ACT_RELU2 = 1, MOE_ACT_CLAMPGLU = 2 };      // 2: of row pairs (gate, up), one output a pair
+enum { MOE_ACT_NONE = 0, MOE_ACT_RELU2 = 1, MOE_ACT_CLAMPGLU = 2, MOE_ACT_SILUGLU = 3 };      // 2, 3: of row pairs (gate, up), one output a pair
+#define MOE_GATED(act) ((act) == MOE_ACT_CLAMPGLU || (act) == MOE_ACT_SILUGLU)
 
 __device__ __forceinline__ float moe_act(int act, float v) {
     if (act == MOE_ACT_RELU2) { v = fmaxf(v, 0.f); return v * v; }
@@ -246,7 +252,7 @@ struct MoeMatmulArgs {
     const int* tile_expert;
     const int* n_tiles;          // or null: every tile of the grid
     int ldi, ldo, N, K, BM, act, n_rows;     // n_rows: rows of `in` when they are taken as they lie (later rows are padding)
-    float limit, alpha;          // act 2
+    float limit, alpha;          // the clamped activation's
 };
 
 #define MP_BN 64
@@ -299,12 +305,13 @@ __global__ void __launch_bounds__(256) moe_matmul_plain_kernel(MoeMatmulArgs a) 
 #pragma unroll
     for (int i = 0; i < RPT; ++i) {
         if (src[tm + i] < 0) continue;
-        if (a.act == MOE_ACT_CLAMPGLU) {
+        if (MOE_GATED(a.act)) {
 #pragma unroll
             for (int j = 0; j < 4; j += 2)
                 if (n0 + tn + j < a.N)
                     CeType<T>::store((T*)a.out + (size_t)(p0 + tm + i) * a.ldo + (n0 + tn + j) / 2,
-                                     ce_clamp_glu(acc[i][j], acc[i][j + 1], a.limit, a.alpha));
+                                     a.act == MOE_ACT_SILUGLU ? ce_silu_glu(acc[i][j], acc[i][j + 1])
+                                                              : ce_clamp_glu(acc[i][j], acc[i][j + 1], a.limit, a.alpha));
             continue;
         }
 #pragma unroll
@@ -370,9 +377,10 @@ __global__ void __launch_bounds__(128) moe_matmul_wmma_kernel(MoeMatmulArgs a) {
     for (int e = tid; e < BM * (MW_BN / 2); e += 128) {
         int r = e / (MW_BN / 2), c = (e % (MW_BN / 2)) * 2;
         if (src[r] < 0 || n0 + c >= a.N) continue;
-        if (a.act == MOE_ACT_CLAMPGLU) {
+        if (MOE_GATED(a.act)) {
             ((__nv_bfloat16*)a.out)[(size_t)(p0 + r) * a.ldo + (n0 + c) / 2] =
-                __float2bfloat16_rn(ce_clamp_glu_fast(Cs[r][c], Cs[r][c + 1], a.limit, a.alpha));
+                __float2bfloat16_rn(a.act == MOE_ACT_SILUGLU ? ce_silu_glu_fast(Cs[r][c], Cs[r][c + 1])
+                                                             : ce_clamp_glu_fast(Cs[r][c], Cs[r][c + 1], a.limit, a.alpha));
             continue;
         }
         __nv_bfloat162 v = __floats2bfloat162_rn(moe_act(a.act, Cs[r][c]), moe_act(a.act, Cs[r][c + 1]));
@@ -388,7 +396,7 @@ extern "C" int ce_moe_matmul(const void* in, const void* W, void* out, const int
     if (max_tiles == 0 || N == 0) return CE_OK;
     if (!in || !W || !out || K <= 0) return ce_fail(CE_ERR_ARG, "ce_moe_matmul: null pointer or K=%d", K);
     if ((BM != 16 && BM != 64) || max_tiles > 65535) return ce_fail(CE_ERR_SIZE, "ce_moe_matmul: tiles of %d rows, %d tiles", BM, max_tiles);
-    if (act < 0 || act > 2 || (act == MOE_ACT_CLAMPGLU && N % 2)) return ce_fail(CE_ERR_ARG, "ce_moe_matmul: activation %d of %d rows", act, N);
+    if (act < 0 || act > 3 || (MOE_GATED(act) && N % 2)) return ce_fail(CE_ERR_ARG, "ce_moe_matmul: activation %d of %d rows", act, N);
     MoeMatmulArgs a{in, W, out, row_token, tile_expert, n_tiles, ldi, ldo, N, K, BM, act, n_rows, limit, alpha};
     if (dtype == CE_BF16 && N % 16 == 0 && K % 16 == 0 && ldi % 8 == 0 && ldo % 2 == 0 &&
         ((((uintptr_t)in) & 15) == 0) && ((((uintptr_t)W) & 31) == 0) && ((((uintptr_t)out) & 3) == 0)) {

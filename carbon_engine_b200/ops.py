@@ -209,6 +209,21 @@ def embed(table: torch.Tensor, tokens: torch.Tensor, x: torch.Tensor, status: to
                            _ptr(status), float(scale), _stream()))
 
 
+def embed_norm(table: torch.Tensor, tokens: torch.Tensor, weight: torch.Tensor, x: torch.Tensor, status: torch.Tensor, eps: float,
+               scale: float = 1.0, rounded: Optional[torch.Tensor] = None) -> None:
+    """x[t, :] = rmsnorm(table[tokens[t], :] * scale) * weight as float32; ``rounded`` (bfloat16) receives the same rounded."""
+    _need(table, "table"); _need(tokens, "tokens", torch.int32); _need(x, "x", torch.float32); _need(weight, "weight", torch.float32)
+    T, H = x.shape
+    if table.shape[1] != H or weight.numel() != H:
+        raise KernelError("embed_norm: widths differ")
+    if rounded is not None:
+        _need(rounded, "rounded", torch.bfloat16)
+        if rounded.shape != x.shape:
+            raise KernelError("embed_norm: the rounded copy must have the shape of x")
+    _ok(kernels().ce_embed_norm(_ptr(table), dtype_code(table.dtype), _ptr(tokens), _ptr(weight), _ptr(x), _ptr(rounded), T, H,
+                                table.shape[0], _ptr(status), float(scale), float(eps), _stream()))
+
+
 def rmsnorm(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, eps: float,
             rows: Optional[torch.Tensor] = None) -> None:
     """out[r] = rmsnorm(x[rows[r]] or x[r]) * weight; x float32, out float32 or bfloat16."""
@@ -340,6 +355,37 @@ def rmsnorm_add_norm(y: torch.Tensor, weight: torch.Tensor, x: torch.Tensor, eps
                                       F32 if out is None else dtype_code(out.dtype), T, W, float(eps), float(next_eps), _stream()))
 
 
+def residual_norm(x: torch.Tensor, alpha: float, outputs: Sequence[torch.Tensor], weight: Optional[torch.Tensor], eps: float,
+                  bias: Optional[torch.Tensor] = None, member_weights: Sequence[torch.Tensor] = (), member_eps: float = 0.0,
+                  factor: float = 1.0, rounded: Optional[torch.Tensor] = None) -> None:
+    """x[t] = rmsnorm(alpha x[t] + s) * weight, all float32.  s is a sublayer's output: ``outputs`` is one tensor, to which
+    ``bias`` is added; or, with ``member_weights``, one or two tensors that are each normed with their weight and
+    ``member_eps`` and whose sum is multiplied by ``factor``.  ``weight`` None: no norm, x[t] = alpha x[t] + s (alpha 0: what x
+    held is not read).  ``rounded`` (bfloat16) receives the new x rounded."""
+    _need(x, "x", torch.float32)
+    T, W = x.shape
+    n = len(member_weights)
+    if len(outputs) != max(n, 1) or n > 2:
+        raise KernelError("residual_norm: one output, or one or two with a norm weight each")
+    for name, t in [("outputs", y) for y in outputs]:
+        _need(t, name, torch.float32)
+        if t.shape != x.shape:
+            raise KernelError("residual_norm: an output's shape differs from x's")
+    for name, t in [("weight", weight), ("bias", bias)] + [("member_weights", w) for w in member_weights]:
+        if t is not None:
+            _need(t, name, torch.float32)
+            if t.numel() != W:
+                raise KernelError(f"residual_norm: {name} must have the width of x")
+    if rounded is not None:
+        _need(rounded, "rounded", torch.bfloat16)
+        if rounded.shape != x.shape:
+            raise KernelError("residual_norm: the rounded copy must have the shape of x")
+    y1 = outputs[1] if len(outputs) > 1 else None
+    wm = list(member_weights) + [None, None]
+    _ok(kernels().ce_residual_norm(_ptr(outputs[0]), _ptr(y1), _ptr(wm[0]), _ptr(wm[1]), n, _ptr(bias), _ptr(weight), _ptr(x),
+                                   _ptr(rounded), T, W, float(alpha), float(factor), float(eps), float(member_eps), _stream()))
+
+
 def tanh_cap(x: torch.Tensor, cap: float) -> None:
     """x <- cap * tanh(x / cap) in place (float32)."""
     _need(x, "x", torch.float32)
@@ -435,25 +481,27 @@ def head_matmul(inp, in_head: int, w, out, out_head: int, heads: int, n: int, k:
 
 def masked_attention(q, q_head: int, k_pool, v_pool, ldk: int, ldv: int, gate, out, positions, seq_of_token, seq_slot,
                      block_table, status, nh: int, nkv: int, d: int, dv: int, page_size: int, window: int, keep_first: int,
-                     scale: float, softcap: float, sinks=None, out_scale: float = 1.0) -> None:
+                     scale: float, softcap: float, sinks=None, out_scale: float = 1.0, slopes=None) -> None:
     """Softmax attention in float32 arithmetic with separate key and value head sizes, a tanh cap on the scores
     (0: none), a window (0: none) that keeps the first ``keep_first`` keys visible, and an optional sigmoid gate per
     output element.  ``v_pool`` may be the key pool itself (``ldv`` = ``ldk``): the values are then the leading
-    ``dv`` elements of every key row.  ``sinks`` (float32 [nh]): exp(sinks[h]) is one more term of head h's denominator."""
+    ``dv`` elements of every key row.  ``sinks`` (float32 [nh]): exp(sinks[h]) is one more term of head h's denominator;
+    ``slopes`` (float32 [nh]): slopes[h] times the key's distance comes off the scaled and capped score."""
     _need(k_pool, "k_pool"); _need(out, "out", k_pool.dtype)
-    _check_sinks(sinks, nh)
+    check_head_numbers(sinks, nh, "sinks")
+    check_head_numbers(slopes, nh, "slopes")
     if q.dtype != k_pool.dtype or v_pool.dtype != k_pool.dtype:
         raise KernelError("masked_attention: q and the cache differ in dtype")
     _ok(kernels().ce_masked_attention(
         _ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(gate), _ptr(out), dtype_code(out.dtype), _ptr(positions), _ptr(seq_of_token),
         _ptr(seq_slot), _ptr(block_table), _ptr(status), out.shape[0], nh, nkv, d, dv, q.stride(0), int(q_head), int(ldk), int(ldv),
         gate.stride(0) if gate is not None else 0, page_size, block_table.shape[1], k_pool.shape[0], int(window), int(keep_first),
-        float(scale), float(softcap), _ptr(sinks), float(out_scale), _stream()))
+        float(scale), float(softcap), _ptr(sinks), float(out_scale), _ptr(slopes), _stream()))
 
 
-def _check_sinks(sinks, nh: int) -> None:
-    if sinks is not None and (sinks.dtype != torch.float32 or sinks.numel() != nh or not sinks.is_contiguous() or not sinks.is_cuda):
-        raise KernelError(f"attention sinks must be {nh} float32 numbers on the GPU")
+def check_head_numbers(t, nh: int, what: str) -> None:
+    if t is not None and (t.dtype != torch.float32 or t.numel() != nh or not t.is_contiguous() or not t.is_cuda):
+        raise KernelError(f"attention {what} must be {nh} float32 numbers on the GPU")
 
 
 def masked_attention_mma_supported(d: int, dv: int, q_stride: int, q_head: int, ldk: int, ldv: int, alias: bool) -> bool:
@@ -462,34 +510,44 @@ def masked_attention_mma_supported(d: int, dv: int, q_stride: int, q_head: int, 
 
 def masked_attention_mma(q, q_head: int, k_pool, v_pool, ldk: int, ldv: int, gate, out, positions, seq_slot, q_start, block_table,
                          tiles, n_tiles: int, status, nh: int, nkv: int, d: int, dv: int, page_size: int, window: int,
-                         keep_first: int, scale: float, softcap: float, sinks=None, out_scale: float = 1.0) -> None:
+                         keep_first: int, scale: float, softcap: float, sinks=None, out_scale: float = 1.0, slopes=None) -> None:
     """:func:`masked_attention` on the tensor cores (bfloat16) for tiles of 64 query tokens: ``tiles`` holds (sequence, first
     token within the sequence's tokens of the step) pairs.  ``gate`` holds bfloat16 logits."""
     _need(k_pool, "k_pool", torch.bfloat16); _need(out, "out", torch.bfloat16)
     if q.dtype != torch.bfloat16 or v_pool.dtype != torch.bfloat16 or (gate is not None and gate.dtype != torch.bfloat16):
         raise KernelError("masked_attention_mma: bfloat16 only")
-    _check_sinks(sinks, nh)
+    check_head_numbers(sinks, nh, "sinks")
+    check_head_numbers(slopes, nh, "slopes")
     _ok(kernels().ce_masked_attention_mma(
         _ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(gate), _ptr(out), _ptr(positions), _ptr(seq_slot), _ptr(q_start), _ptr(block_table),
         _ptr(tiles), _ptr(status), int(n_tiles), out.shape[0], nh, nkv, d, dv, q.stride(0), int(q_head), int(ldk), int(ldv),
         gate.stride(0) if gate is not None else 0, page_size, block_table.shape[1], k_pool.shape[0], int(window), int(keep_first),
-        float(scale), float(softcap), _ptr(sinks), float(out_scale), _stream()))
+        float(scale), float(softcap), _ptr(sinks), float(out_scale), _ptr(slopes), _stream()))
+
+
+#: how the heads of norm_rope_kvwrite are normed: not at all, before the rotation, or behind it
+HEAD_NORMS = {"none": 0, "before": 1, "after": 2}
 
 
 def norm_rope_kvwrite(proj, q_out, k_pool, v_pool, wq, wk, head_scale, cos, sin, positions, seq_of_token, seq_slot, block_table,
                       status, off_q: int, off_k: int, off_v: int, nh: int, nkv: int, d: int, dv: int, rotary_dim: int,
-                      page_size: int, eps: float, write_kv: bool = True) -> None:
+                      page_size: int, eps: float, write_kv: bool = True, norm: Optional[str] = None, pairing: str = "half",
+                      pos_scale=None) -> None:
     """Operands of attention with a norm per head, from float32 rows ``proj``: query heads (from ``off_q``) and key heads
-    (from ``off_k``) divided by their root mean square times ``wq`` / ``wk`` (None: no norm), rotated over their first
-    ``rotary_dim`` elements (element i with i + rotary_dim/2), queries times ``head_scale[h]`` (None: no factor) into
-    ``q_out`` [T, nh * d], keys and the values (``nkv`` heads of ``dv`` from ``off_v``; ``off_v`` = ``off_k``: the keys as
+    (from ``off_k``) divided by their root mean square, times ``wq`` / ``wk`` (None: no weight), before or behind the rotation
+    (``norm``: "before", "after", "none"; by default "before" with weights and "none" without), rotated over their first
+    ``rotary_dim`` elements (``pairing``: element i with i + rotary_dim/2, or 2i with 2i + 1), queries times ``head_scale[h]``
+    and ``pos_scale[position]`` (None: no factor) into ``q_out`` [T, nh * d], keys and the values (``nkv`` heads of ``dv`` from ``off_v``; ``off_v`` = ``off_k``: the keys as
     projected) into the pages."""
     _need(q_out, "q_out")
     if proj.dtype != torch.float32 or proj.stride(-1) != 1:
         raise KernelError("norm_rope_kvwrite: proj must be float32 rows")
-    for name, t in (("wq", wq), ("wk", wk), ("head_scale", head_scale), ("cos", cos), ("sin", sin)):
+    for name, t in (("wq", wq), ("wk", wk), ("head_scale", head_scale), ("pos_scale", pos_scale), ("cos", cos), ("sin", sin)):
         if t is not None:
             _need(t, name, torch.float32)
+    norm = norm or ("none" if wq is None else "before")
+    if norm not in HEAD_NORMS or pairing not in ROPE_PAIRINGS:
+        raise KernelError(f"norm_rope_kvwrite: norm '{norm}', pairing '{pairing}'")
     T = q_out.shape[0]
     if q_out.shape[1] != nh * d or (wq is not None and wq.numel() != d) or (wk is not None and wk.numel() != d) or \
             (head_scale is not None and head_scale.numel() != nh) or proj.shape[1] < max(off_q + nh * d, off_k + nkv * d, off_v + nkv * dv):
@@ -503,10 +561,11 @@ def norm_rope_kvwrite(proj, q_out, k_pool, v_pool, wq, wk, head_scale, cos, sin,
                               f"{nkv} x {d} keys and {nkv} x {dv} values in pages of {page_size}")
     _ok(kernels().ce_norm_rope_kvwrite(
         _ptr(proj), _ptr(q_out), _ptr(k_pool), _ptr(v_pool), dtype_code(q_out.dtype), _ptr(wq), _ptr(wk), _ptr(head_scale),
-        _ptr(cos), _ptr(sin), _ptr(positions), _ptr(seq_of_token), _ptr(seq_slot), _ptr(block_table), _ptr(status), T,
+        _ptr(pos_scale), _ptr(cos), _ptr(sin), _ptr(positions), _ptr(seq_of_token), _ptr(seq_slot), _ptr(block_table), _ptr(status), T,
         proj.stride(0), int(off_q), int(off_k), int(off_v), nh, nkv, d, dv, rotary_dim if cos is not None else 0, page_size,
         block_table.shape[1] if block_table is not None else 0, k_pool.shape[0] if k_pool is not None else 0,
-        cos.shape[0] if cos is not None else 0, 1 if write_kv else 0, float(eps), _stream()))
+        cos.shape[0] if cos is not None else 0, 1 if write_kv else 0, float(eps), HEAD_NORMS[norm], ROPE_PAIRINGS[pairing],
+        pos_scale.numel() if pos_scale is not None else 0, _stream()))
 
 
 DECAY_PER_CHANNEL, DECAY_PER_HEAD, DECAY_CONSTANT, DECAY_EXP_GATES = 0, 1, 2, 3
@@ -807,16 +866,19 @@ def general_delta(proj, zz, w0, a_bias, norm_w, prep, raw, state, out, seq_slot,
                                        proj.stride(0), off_r, off_k, off_v, off_a, off_g, heads, d, float(eps), stage, _stream()))
 
 
-#: "clamped_glu": an expert's rows are gate and up rows by turns (2j the gate of feature j, 2j + 1 its up); one output a pair
-MOE_ACTIVATIONS = {"none": 0, "relu2": 1, "clamped_glu": 2}
-MOE_SCORES = {"softmax": 0, "sigmoid": 1}
+#: the gated ones: an expert's rows are gate and up rows by turns (2j the gate of feature j, 2j + 1 its up); one output a pair
+MOE_ACTIVATIONS = {"none": 0, "relu2": 1, "clamped_glu": 2, "silu_glu": 3}
+MOE_GATED = ("clamped_glu", "silu_glu")
+#: "softmax_chosen": the logits themselves decide, and the weights are the softmax over the chosen ones
+MOE_SCORES = {"softmax": 0, "sigmoid": 1, "softmax_chosen": 2}
 MOE_GROUP_SCORES = {"max": 0, "top2": 1}
 
 
 def moe_route(z: torch.Tensor, experts: int, top: int, groups: int, keep: int, scale: float, ids: torch.Tensor,
               weights: torch.Tensor, sgate: Optional[torch.Tensor] = None, scoring: str = "softmax",
-              correction: Optional[torch.Tensor] = None, group_score: str = "max", renormalize: bool = True) -> None:
-    """Router logits z [T, >= experts (+1)] float32 -> the ``top`` experts of every token (``ids`` int32 [T, top], best
+              correction: Optional[torch.Tensor] = None, group_score: str = "max", renormalize: bool = True,
+              bias: Optional[torch.Tensor] = None) -> None:
+    """Router logits z [T, >= experts (+1)] float32 (plus ``bias`` [experts]) -> the ``top`` experts of every token (``ids`` int32 [T, top], best
     first) and their weights (float32 [T, top]): scores s = softmax over the experts or sigmoid, choice scores s +
     ``correction`` (float32 [experts]), experts in ``groups`` equal groups of neighbours of which the ``keep`` with the
     largest member (or, "top2", the largest sum of two members) stay eligible, weights = chosen s / their sum * scale, or s *
@@ -829,9 +891,13 @@ def moe_route(z: torch.Tensor, experts: int, top: int, groups: int, keep: int, s
         _need(correction, "correction", torch.float32)
         if correction.numel() != experts:
             raise KernelError("moe_route: one correction per expert")
+    if bias is not None:
+        _need(bias, "bias", torch.float32)
+        if bias.numel() < experts:
+            raise KernelError("moe_route: one bias per expert")
     _ok(kernels().ce_moe_route(_ptr(z), _ptr(ids), _ptr(weights), _ptr(sgate), T, z.stride(0), int(experts), int(top), int(groups),
                                int(keep), float(scale), _ptr(correction), MOE_SCORES[scoring], MOE_GROUP_SCORES[group_score],
-                               1 if renormalize else 0, _stream()))
+                               1 if renormalize else 0, _ptr(bias), _stream()))
 
 
 def moe_max_tiles(n_pairs: int, experts: int, tile: int) -> int:
@@ -856,10 +922,10 @@ def moe_matmul(inp: torch.Tensor, w: torch.Tensor, out: torch.Tensor, tile: int,
                tile_expert=None, n_tiles=None, limit: float = 0.0, alpha: float = 0.0) -> None:
     """out[p] = act(inp[row_token[p]] @ w[tile_expert[p // tile]].T) for the rows of the layout's tiles (``row_token``
     None: the input rows are the layout's rows already).  Without any table: out = act(inp @ w[0].T), row by row.
-    w [experts, N, K]; operands and output in one dtype.  "clamped_glu" (``limit``, ``alpha``): rows 2j and 2j + 1 of an expert
-    are feature j's gate and up, and ``out`` has N / 2 columns."""
+    w [experts, N, K]; operands and output in one dtype.  "clamped_glu" (``limit``, ``alpha``), "silu_glu": rows 2j and 2j + 1
+    of an expert are feature j's gate and up, and ``out`` has N / 2 columns."""
     _need(w, "w", inp.dtype); _need(out, "out", inp.dtype)
-    per = 2 if activation == "clamped_glu" else 1
+    per = 2 if activation in MOE_GATED else 1
     if inp.stride(-1) != 1 or w.dim() != 3 or inp.shape[1] != w.shape[2] or out.shape[1] * per != w.shape[1]:
         raise KernelError("moe_matmul: shapes do not fit")
     if tile_expert is None:

@@ -15,14 +15,14 @@ kernel_lib.declare("ce_attention_decode_scratch", _ll, [_i, _i, _i, _i])
 # q, k_pool, v_pool, out, scratch, counters, n_counters, positions, seq_slot, q_start, ctx_len, block_table, status,
 # n_seqs, nh, nkv, d, q_stride, page_size, max_pages, num_pages, window, scale, max_splits, stream
 kernel_lib.declare("ce_attention_decode_bf16", _i, [_p] * 6 + [_i] + [_p] * 6 + [_i] * 9 + [_f, _i, _p])
-# the same with, before the stream: sinks (float32 [nh] or null), out_scale
-kernel_lib.declare("ce_attention_decode_bf16_sink", _i, [_p] * 6 + [_i] + [_p] * 6 + [_i] * 9 + [_f, _i, _p, _f, _p])
+# the same with, before the stream: sinks (float32 [nh] or null), out_scale, slopes (float32 [nh] or null)
+kernel_lib.declare("ce_attention_decode_bf16_sink", _i, [_p] * 6 + [_i] + [_p] * 6 + [_i] * 9 + [_f, _i, _p, _f, _p, _p])
 kernel_lib.declare("ce_attention_decode_split", _i, [])
 kernel_lib.declare("ce_attention_decode_kernels", _i, [])
 # q, k_pool, v_pool, out, positions, seq_slot, q_start, ctx_len, block_table, tiles, status,
 # n_tiles, nh, nkv, d, q_stride, page_size, max_pages, num_pages, window, scale, stream
 kernel_lib.declare("ce_attention_prefill_bf16", _i, [_p] * 11 + [_i] * 9 + [_f, _p])
-kernel_lib.declare("ce_attention_prefill_bf16_sink", _i, [_p] * 11 + [_i] * 9 + [_f, _p, _f, _p])
+kernel_lib.declare("ce_attention_prefill_bf16_sink", _i, [_p] * 11 + [_i] * 9 + [_f, _p, _f, _p, _p])
 
 kernel_lib.declare("ce_gemm_tc_supported", _i, [_i, _i, _i, _i])
 kernel_lib.declare("ce_gemm_tc_scratch", _ll, [_i, _i, _i, _i])
@@ -45,7 +45,7 @@ kernel_lib.declare("ce_attention_prefill_tc_supported", _i, [_i, _i, _i])
 # q, k_pool, v_pool, out, seq_slot, q_start, ctx_len, block_table, tiles, status,
 # n_tiles, total_tokens, nh, nkv, d, q_stride, page_size, max_pages, num_pages, window, scale, stream
 kernel_lib.declare("ce_attention_prefill_tc", _i, [_p] * 10 + [_i] * 10 + [_f, _p])
-kernel_lib.declare("ce_attention_prefill_tc_sink", _i, [_p] * 10 + [_i] * 10 + [_f, _p, _f, _p])
+kernel_lib.declare("ce_attention_prefill_tc_sink", _i, [_p] * 10 + [_i] * 10 + [_f, _p, _f, _p, _p])
 
 #: set to False to keep portions of prompts off the tcgen05 attention kernel (the mma.sync one takes them)
 USE_TENSOR_ATTENTION = True
@@ -151,19 +151,21 @@ def attention_supported(d: int, q_stride: int) -> bool:
     return 16 <= d <= 256 and d % 16 == 0 and q_stride % 2 == 0
 
 
-def attention_bf16(ctx, plan, qkv, out, cache, table, nh, nkv, d, window, scale, sinks=None, out_scale: float = 1.0) -> bool:
+def attention_bf16(ctx, plan, qkv, out, cache, table, nh, nkv, d, window, scale, sinks=None, out_scale: float = 1.0,
+                   slopes=None) -> bool:
     """Decode kernel for the leading one-token sequences, flash kernel for the portions.  ``plan``: the
     step's tile lists and split bound (``parts.attention.AttentionPlan``).  ``qkv``: rows whose leading ``nh * d``
     columns are the query heads.  ``sinks`` (float32 [nh] or None): a number per head whose exponential joins the
-    softmax's denominator without a key or a value; ``out_scale`` multiplies what is stored."""
+    softmax's denominator without a key or a value; ``out_scale`` multiplies what is stored; ``slopes`` (float32 [nh] or None):
+    slope times the key's distance comes off a head's scaled scores."""
     if not attention_supported(d, qkv.shape[1]):
         return False
-    if sinks is not None and (sinks.dtype != torch.float32 or sinks.numel() != nh or not sinks.is_cuda or not sinks.is_contiguous()):
-        raise ops.KernelError(f"attention sinks must be {nh} float32 numbers on the GPU")
+    ops.check_head_numbers(sinks, nh, "sinks")
+    ops.check_head_numbers(slopes, nh, "slopes")
     k = kernels()
     stream = ops._stream()
     args = (cache.page_size, table.shape[1], cache.k_pool.shape[0], int(window), float(scale))
-    tail = (None if sinks is None else sinks.data_ptr(), float(out_scale), stream)
+    tail = (ops._ptr(sinks), float(out_scale), ops._ptr(slopes), stream)
     if ctx.n_decode > 0:
         splits = plan.decode_splits
         need = k.ce_attention_decode_scratch(ctx.n_decode, nh, d, splits)

@@ -72,6 +72,10 @@ class BundleCacheSpec:
     extra: Tuple[Tuple[str, StateCacheSpec], ...] = ()
 
 
+#: ``ctx.shared`` entry by which a kernel that wrote the residual hands on its bfloat16 rounding, for a sublayer that reads the
+#: residual itself: (rounded [T, width], the residual's data pointer)
+RESIDUAL_ROUNDED = "residual.rounded"
+
 CacheSpec = Union[PagedCacheSpec, StateCacheSpec, BundleCacheSpec, None]
 TensorGetter = Callable[[str], torch.Tensor]
 

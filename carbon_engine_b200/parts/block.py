@@ -1,6 +1,7 @@
 """Arrangements of parts in a layer.  Pre-norm: x += mixer(norm1(x)); x += ffn(norm2(x))
 (src/model/mod.rs:645-650).  Output-norm: x += norm1(mixer(x)); x += norm2(ffn(x)).  Sandwich-norm:
-x += norm1b(mixer(norm1(x))); x += norm2b(ffn(norm2(x))).  Parallel: h = norm1(x); x += mixer(h) + ffn(h)."""
+x += norm1b(mixer(norm1(x))); x += norm2b(ffn(norm2(x))).  Parallel: h = norm1(x); x += mixer(h) + ffn(h).
+Post-norm: x <- norm1(alpha x + mixer(x)); x <- norm2(alpha x + ffn(x))."""
 from __future__ import annotations
 
 from typing import List, Optional
@@ -8,8 +9,21 @@ from typing import List, Optional
 import torch
 
 from .. import ops
-from .base import Block, BundleCacheSpec, FeedForward, Mixer, Norm, Part
+from .base import RESIDUAL_ROUNDED, Block, BundleCacheSpec, FeedForward, Mixer, Norm, Part
+from .combine import NormedMixers
 from .norm import RMSNorm
+
+
+def read_residual(ctx, x: torch.Tensor) -> torch.Tensor:
+    """The residual as a sublayer's input: itself in float32, else its rounding, which the kernel that wrote it may have left."""
+    if ctx.dtype == torch.float32:
+        return x
+    left = ctx.shared.pop(RESIDUAL_ROUNDED, None)
+    if left is not None and left[1] == x.data_ptr() and left[0].shape == x.shape:
+        return left[0]
+    h = ctx.buffer(tuple(x.shape))
+    ops.copy_cols(x, 0, x.shape[1], h)
+    return h
 
 
 class PreNormBlock(Block):
@@ -87,19 +101,6 @@ class OutputNormBlock(Block):
         ffn = self.ffn.step_bytes(tokens, element_size) if self.ffn is not None else 0
         return tokens * self.width * (element_size + 4) + max(self.mixer.step_bytes(tokens, element_size), ffn)
 
-    #: what the norm before left in ``ctx.shared``: the residual rounded to bfloat16, and whose rounding it is
-    ROUNDED = "residual.rounded"
-
-    def _read(self, ctx, x: torch.Tensor) -> torch.Tensor:
-        if ctx.dtype == torch.float32:
-            return x
-        left = ctx.shared.pop(self.ROUNDED, None)
-        if left is not None and left[1] == x.data_ptr() and left[0].shape == x.shape:
-            return left[0]
-        h = ctx.buffer(tuple(x.shape))
-        ops.copy_cols(x, 0, x.shape[1], h)
-        return h
-
     def _add(self, ctx, norm: Norm, y: torch.Tensor, x: torch.Tensor) -> None:
         """x += norm(y); in bfloat16 the norm's kernel also leaves the new residual rounded for the sublayer that reads it
         next (this block's feed-forward, or the next block's mixer)."""
@@ -108,20 +109,70 @@ class OutputNormBlock(Block):
             return
         h = ctx.buffer(tuple(x.shape))
         norm.add_into(y, x, rounded=h)
-        ctx.shared[self.ROUNDED] = (h, x.data_ptr())
+        ctx.shared[RESIDUAL_ROUNDED] = (h, x.data_ptr())
 
     def forward(self, ctx, x: torch.Tensor, cache) -> None:
         y = ctx.buffer(tuple(x.shape), torch.float32)
-        owed = self.mixer.forward(ctx, self._read(ctx, x), y, cache, accumulate=False)
+        owed = self.mixer.forward(ctx, read_residual(ctx, x), y, cache, accumulate=False)
         if owed is not None:
             ops.add_bias(y, owed)
         self._add(ctx, self.mixer_norm, y, x)
         if self.ffn is None:
             return
-        owed = self.ffn.forward(ctx, self._read(ctx, x), y, accumulate=False)
+        owed = self.ffn.forward(ctx, read_residual(ctx, x), y, accumulate=False)
         if owed is not None:
             ops.add_bias(y, owed)
         self._add(ctx, self.ffn_norm, y, x)
+
+
+class PostNormBlock(Block):
+    """The norm is taken of the weighted residual plus the sublayer's output, and IS the new residual: x <- mixer_norm(alpha x +
+    mixer(x)); x <- ffn_norm(alpha x + ffn(x)).  The sublayers read the residual itself (rounded to the compute dtype) and STORE
+    their result in a float32 buffer (``can_store``); one kernel weighs, adds and norms, and leaves the new residual rounded for
+    the next sublayer.  The outputs of mixers side by side (:class:`NormedMixers`) are normed and added in that kernel too.
+    The norms are RMS norms.  ``ffn`` None: the layer has only the mixer."""
+
+    def __init__(self, width: int, alpha: float, mixer: Mixer, mixer_norm: RMSNorm, ffn: Optional[FeedForward] = None,
+                 ffn_norm: Optional[RMSNorm] = None):
+        if (ffn is None) != (ffn_norm is None):
+            raise ValueError("a feed-forward and its norm come together")
+        for part in (mixer, ffn):
+            if part is not None and not getattr(part, "can_store", False):
+                raise ValueError(f"{type(part).__name__} cannot store its output, which a norm of the sum needs")
+        for norm in (mixer_norm, ffn_norm):
+            if norm is not None and not isinstance(norm, RMSNorm):
+                raise ValueError(f"{type(norm).__name__}: this block's norms are RMS norms")
+        self.width, self.alpha = int(width), float(alpha)
+        self.mixer, self.mixer_norm, self.ffn, self.ffn_norm = mixer, mixer_norm, ffn, ffn_norm
+
+    def children(self) -> List[Part]:
+        return [p for p in (self.mixer, self.mixer_norm, self.ffn, self.ffn_norm) if p is not None]
+
+    def step_bytes(self, tokens: int, element_size: int) -> int:
+        ffn = self.ffn.step_bytes(tokens, element_size) if self.ffn is not None else 0
+        return tokens * self.width * (2 * element_size + 4) + max(self.mixer.step_bytes(tokens, element_size), ffn)
+
+    def _norm(self, ctx, x: torch.Tensor, outputs: List[torch.Tensor], norm: RMSNorm, **more) -> None:
+        rounded = ctx.buffer(tuple(x.shape)) if ctx.dtype == torch.bfloat16 else None
+        ops.residual_norm(x, self.alpha, outputs, norm.weight, norm.eps, rounded=rounded, **more)
+        if rounded is not None:
+            ctx.shared[RESIDUAL_ROUNDED] = (rounded, x.data_ptr())
+
+    def forward(self, ctx, x: torch.Tensor, cache) -> None:
+        h = read_residual(ctx, x)
+        if isinstance(self.mixer, NormedMixers):
+            m = self.mixer
+            self._norm(ctx, x, m.outputs(ctx, h, cache), self.mixer_norm, member_weights=[n.weight for n in m.norms],
+                       member_eps=m.norms[0].eps, factor=m.factor)
+        else:
+            y = ctx.buffer(tuple(x.shape), torch.float32)
+            owed = self.mixer.forward(ctx, h, y, cache, accumulate=False)
+            self._norm(ctx, x, [y], self.mixer_norm, bias=owed)
+        if self.ffn is None:
+            return
+        y = ctx.buffer(tuple(x.shape), torch.float32)
+        owed = self.ffn.forward(ctx, read_residual(ctx, x), y, accumulate=False)
+        self._norm(ctx, x, [y], self.ffn_norm, bias=owed)
 
 
 class SandwichNormBlock(Block):

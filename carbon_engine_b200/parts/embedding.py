@@ -12,23 +12,36 @@ from typing import List, Optional
 import torch
 
 from .. import ops
-from .base import Norm, Part, TensorGetter, TensorSpec, to_device
+from .base import RESIDUAL_ROUNDED, Norm, Part, TensorGetter, TensorSpec, to_device
 from .linear import STORE_F32, matmul_nt
+from .norm import RMSNorm
 
 
 class Embedding(Part):
-    def __init__(self, vocab: int, width: int, name: str, scale: float = 1.0):
-        """``scale`` multiplies every embedding row on its way into the residual stream."""
+    def __init__(self, vocab: int, width: int, name: str, scale: float = 1.0, norm: Optional[RMSNorm] = None,
+                 leave_rounded: bool = False):
+        """``scale`` multiplies every embedding row on its way into the residual stream; ``norm`` is taken of it then (in the same
+        kernel).  ``leave_rounded``, with a norm: the first block reads the residual itself, and finds it rounded."""
         self.vocab, self.width, self.name, self.scale = vocab, width, name, float(scale)
+        self.norm, self.leave_rounded = norm, bool(leave_rounded)
         self.weight: Optional[torch.Tensor] = None
 
     def tensor_specs(self) -> List[TensorSpec]:
         return [TensorSpec(self.name, (self.vocab, self.width), "embedding")]
 
+    def children(self) -> List[Part]:
+        return [self.norm] if self.norm is not None else []
+
     def load(self, get: TensorGetter, device, dtype) -> None:
         self.weight = to_device(get(self.name), device, dtype)
 
     def forward(self, ctx, x: torch.Tensor) -> None:
+        if self.norm is not None:
+            rounded = ctx.buffer(tuple(x.shape)) if self.leave_rounded and ctx.dtype == torch.bfloat16 else None
+            ops.embed_norm(self.weight, ctx.tokens, self.norm.weight, x, ctx.status, self.norm.eps, self.scale, rounded)
+            if rounded is not None:
+                ctx.shared[RESIDUAL_ROUNDED] = (rounded, x.data_ptr())
+            return
         ops.embed(self.weight, ctx.tokens, x, ctx.status, self.scale)
 
 

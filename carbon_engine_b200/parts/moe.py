@@ -1,12 +1,13 @@
 """Mixture-of-experts feed-forward: a router picks ``top`` of ``experts`` small feed-forward layers for every token, and
 their outputs are summed with the router's weights; a shared expert may run for every token beside them.
 
-    z = W_router h (float32);  s = softmax(z) over all experts, or sigmoid(z);  choice scores c = s, or s + a correction per expert
+    z = W_router h, or plus a bias per expert (float32);  s = softmax(z) over all experts, or sigmoid(z);  choice scores c = s, or s +
+    a correction per expert;  "softmax_chosen": s = exp(z), c = z, so that the weights below are a softmax over the chosen logits
     experts form ``groups`` equal groups of neighbours; a group's score is its largest c, or the sum of its two largest; only
     experts of the ``keep`` best groups are eligible; the ``top`` eligible experts with the largest c are chosen
     weight_e = s_e / (sum of the chosen s + 1e-20) * scale, or s_e * scale
     y = sum_e weight_e expert_e(h)  +  shared(h), optionally times sigmoid(W_sg h)
-    expert(h) = W_down relu(W_up h)^2, or W_down (g sigmoid(alpha g) (u + 1)), g = min(W_gate h, limit), u = W_up h within [-limit, limit]
+    expert(h) = W_down relu(W_up h)^2, W_down (silu(W_gate h) W_up h), or W_down (g sigmoid(alpha g) (u + 1)), g = min(W_gate h, limit), u = W_up h within [-limit, limit]
 
 The experts' matrices are held as two stacks [experts, ff, hidden] (gated experts: [experts, 2 ff, hidden], gate and up rows by
 turns, so that a feature's two values come out side by side and the product's epilogue is the activation) and
@@ -28,7 +29,7 @@ import torch
 
 from .. import ops, ops_tensor
 from .base import FeedForward, Part, TensorGetter, TensorSpec, register_init_kind, to_device
-from .linear import CLAMPGLU, RELU2, STORE, STORE_F32, Linear
+from .linear import CLAMPGLU, RELU2, STORE, STORE_F32, SWIGLU, Linear
 
 register_init_kind("correction", 0.0, 0.1, True)
 
@@ -41,9 +42,10 @@ class RoutedExperts(FeedForward):
     def __init__(self, hidden: int, experts: int, top: int, ff: int, prefix: str, groups: int = 1, keep_groups: int = 1,
                  scale: float = 1.0, activation: str = "relu2", shared_ff: int = 0, shared_gate: bool = True,
                  scoring: str = "softmax", correction: bool = False, group_score: str = "max", renormalize: bool = True,
-                 limit: float = 0.0, shared_limit: float = 0.0, alpha: float = 1.0):
-        """Tensors ``prefix.router`` [experts, hidden], ``prefix.e<i>.up`` [ff, hidden], ``prefix.e<i>.down`` [hidden, ff], with
-        the "clamped_glu" activation ``prefix.e<i>.gate``, with ``correction`` ``prefix.correction`` [experts] and,
+                 limit: float = 0.0, shared_limit: float = 0.0, alpha: float = 1.0, router_bias: bool = False):
+        """Tensors ``prefix.router`` [experts, hidden], with ``router_bias`` ``prefix.router.b`` [experts], ``prefix.e<i>.up`` [ff,
+        hidden], ``prefix.e<i>.down`` [hidden, ff], with the gated activations ("clamped_glu", "silu_glu") ``prefix.e<i>.gate``, with
+        ``correction`` ``prefix.correction`` [experts] and,
         with ``shared_ff`` > 0, ``prefix.shared.up`` / ``.down`` (``.gate``) and (with ``shared_gate``) ``prefix.shared.sg`` [1, hidden].
         ``limit``, ``shared_limit``, ``alpha``: the clamped activation's constants, of the experts and of the shared expert."""
         if activation not in ops.MOE_ACTIVATIONS:
@@ -55,8 +57,8 @@ class RoutedExperts(FeedForward):
         for table, value in ((ops.MOE_SCORES, scoring), (ops.MOE_GROUP_SCORES, group_score)):
             if value not in table:
                 raise ValueError(f"'{value}' is not supported ({', '.join(sorted(table))})")
-        self.gated = activation == "clamped_glu"
-        if self.gated and not (limit > 0.0 and (shared_ff == 0 or shared_limit > 0.0)):
+        self.gated = activation in ops.MOE_GATED
+        if activation == "clamped_glu" and not (limit > 0.0 and (shared_ff == 0 or shared_limit > 0.0)):
             raise ValueError(f"the clamped activation needs positive limits, got {limit} and {shared_limit}")
         self.scoring, self.correction, self.group_score, self.renormalize = scoring, bool(correction), group_score, bool(renormalize)
         self.limit, self.shared_limit, self.alpha = float(limit), float(shared_limit), float(alpha)
@@ -66,7 +68,8 @@ class RoutedExperts(FeedForward):
         sizes, names = [experts], [f"{prefix}.router"]
         if self.shared_gate:
             sizes.append(1); names.append(f"{prefix}.shared.sg")
-        self.router = Linear(hidden, sizes, names, pad_rows_to=4)
+        self.router = Linear(hidden, sizes, names, pad_rows_to=4,
+                             bias_names=[f"{prefix}.router.b"] + [None] * (len(names) - 1) if router_bias else None)
         self.up: Optional[torch.Tensor] = None            # [experts, ff, hidden]; gated: [experts, 2 ff, hidden], gate and up rows by turns
         self.down: Optional[torch.Tensor] = None          # [experts, hidden, ff]
         # the shared expert is two ordinary products (the activation is the first one's epilogue)
@@ -131,11 +134,11 @@ class RoutedExperts(FeedForward):
         T, E, top = h.shape[0], self.experts, self.top
         i32 = lambda n: ctx.buffer((n,), torch.int32)
         z = ctx.buffer((T, self.router.padded_out), torch.float32)
-        self.router.forward(h, z, STORE_F32)
+        self.router.forward(h, z, STORE_F32, add_bias=False)            # (the routing kernel adds the bias)
         ids, weights = ctx.buffer((T, top), torch.int32), ctx.buffer((T, top), torch.float32)
         sgate = ctx.buffer((T,), torch.float32) if self.shared_gate else None
         ops.moe_route(z, E, top, self.groups, self.keep_groups, self.scale, ids, weights, sgate, self.scoring, self.correction_w,
-                      self.group_score, self.renormalize)
+                      self.group_score, self.renormalize, self.router.bias)
         tile = self.tile_for(T, h.dtype)
         fast = self._fast(tile, h.dtype)
         tiles = ops.moe_max_tiles(T * top, E, tile)
@@ -153,7 +156,9 @@ class RoutedExperts(FeedForward):
         shared = None
         if self.shared_ff > 0:
             sact = ctx.buffer((T, self.shared_ff))
-            if self.gated:
+            if self.activation == "silu_glu":
+                self.shared_up.forward(h, sact, SWIGLU)
+            elif self.gated:
                 self.shared_up.forward(h, sact, CLAMPGLU, glu=ops.GluParams(self.shared_limit, self.alpha))
             else:
                 self.shared_up.forward(h, sact, RELU2 if self.activation == "relu2" else STORE)

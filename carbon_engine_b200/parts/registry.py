@@ -10,7 +10,7 @@ from typing import Callable, Dict
 from .attention import PagedAttention
 from .delta_rule import GeneralDeltaRule
 from .diff_attention import DifferentialAttention
-from .combine import SummedMixers
+from .combine import NormedMixers, SummedMixers
 from .gated_delta import ChannelGatedDelta, HeadGatedDelta
 from .latent_attention import LatentAttention
 from .masked_attention import GatedWindowAttention
@@ -62,6 +62,7 @@ register_mixer("head_gated_delta", HeadGatedDelta)
 register_mixer("retention", Retention)
 register_mixer("sink_attention", SinkAttention)
 register_mixer("summed_mixers", SummedMixers)
+register_mixer("normed_mixers", NormedMixers)
 register_mixer("state_space", StateSpace)
 register_mixer("matrix_memory", MatrixMemory)
 register_feed_forward("gated_mlp", GatedMLP)

@@ -113,3 +113,18 @@ class RotaryEmbedding(PositionEncoding):
 
 class NoPositionEncoding(PositionEncoding):
     """Attention without any rotation."""
+
+
+class QueryTemperature:
+    """A factor on the query that grows with its position p: 1 + coef ln(floor((p + 1) / every) + 1); a float32 table computed in
+    float64, read by the kernel that prepares the queries."""
+
+    def __init__(self, coef: float, every: float, max_positions: int):
+        if not every > 0:
+            raise ValueError(f"a query temperature that grows every {every} positions")
+        self.coef, self.every, self.max_positions = float(coef), float(every), int(max_positions)
+        self.table: Optional[torch.Tensor] = None      # float32 [max_positions]
+
+    def prepare(self, device: torch.device) -> None:
+        steps = torch.floor((torch.arange(self.max_positions, dtype=torch.float64) + 1.0) / self.every)
+        self.table = (1.0 + self.coef * torch.log(steps + 1.0)).to(torch.float32).to(device).contiguous()
