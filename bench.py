@@ -257,16 +257,38 @@ def rapovik_config(width, heads, kv_heads, ff, layers, vocab):
                                     "norm": {"eps": 1e-6}, "max_position_embeddings": 8192})
 
 
+def lanirax_config(width, heads, kv_heads, ff, layers, vocab):
+    """A Lanirax model of the usual proportions at the Qwen3 model's layer sizes: layers go the pair (attention with heads of 128
+    whose values are the projected keys, a window of 1,024, half of a head rotated, a sink per head, beside the delta rule with a
+    decay per head: state heads of 128 x 128 filling the width, half as many key heads, 4 taps) and attention (heads of 128 over
+    all keys, a penalty on distance) and again, each with a mixture of 32 gated experts, 4 per token, each an eighth of the dense
+    width: a token's products are half as wide as the dense layer's.  No layer shares weights."""
+    from carbon_engine_b200.config.lanirax import LaniraxConfig
+    n = width // 128
+    moe = {"kind": "moe", "expert": {"ff": ff // 8}, "router": {"experts": 32, "top": 4}}
+    pair = {"type": "parallel", "mlp": moe,
+            "mixer": {"left": {"heads": heads, "kv_heads": kv_heads, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": 1024},
+                               "rot": {"dims": 64, "base": 1e6, "scaling": {"factor": 4.0, "original": 2048, "fast": 32.0, "slow": 1.0}}},
+                      "right": {"heads": n, "kv_heads": max(1, n // 2), "dim": 128, "vdim": 128, "conv": 4}}}
+    attention = {"type": "attention", "mlp": moe,
+                 "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+                           "q_temp": {"coef": 0.1, "every": 1024}}}
+    kinds = (pair, attention)
+    return LaniraxConfig.from_dict({"architecture": "Lanirax", "vocab": vocab, "width": width,
+                                    "layers": [kinds[i % 2] for i in range(layers)], "norm": {"eps": 1e-6}, "postln_alpha": 1.5,
+                                    "max_position_embeddings": 8192})
+
+
 def compare_designs(args, BenchHarness, pk) -> int:
-    """Prefill and decode throughput of the engine's other designs (--designs: munizen, lunerax, vamadra, pugozen, rapovik) beside the Qwen3 dense
-    design at equal layer sizes (random weights, a few layers), with the kernels of each and their distance from the roofline."""
+    """Prefill and decode throughput of the engine's other designs (--designs: munizen, lunerax, vamadra, pugozen, rapovik, lanirax) beside the
+    Qwen3 dense design at equal layer sizes (random weights, a few layers), with the kernels of each and their distance from the roofline."""
     import torch
     makers = {"munizen": munizen_config, "lunerax": lunerax_config, "vamadra": vamadra_config, "pugozen": pugozen_config,
-              "rapovik": rapovik_config}
+              "rapovik": rapovik_config, "lanirax": lanirax_config}
     designs = [x for x in args.designs.split(",") if x != "qwen3"]
     for x in designs:
         if x not in makers:
-            raise SystemExit(f"--designs {x}: munizen, lunerax, vamadra, pugozen, rapovik and qwen3 are built")
+            raise SystemExit(f"--designs {x}: munizen, lunerax, vamadra, pugozen, rapovik, lanirax and qwen3 are built")
     layers = args.layers if args.layers != SIZES_8B["num_hidden_layers"] else 4
     vocab, out = 32768, {}
     for name in args.sizes.split(","):
@@ -325,7 +347,7 @@ def main() -> int:
     ap.add_argument("--sizes", default="1b,8b", help="with --workload compare-designs: which of the layer sizes "
                     "1b, 4b, 8b (width / heads / feed-forward of models of about that size), with commas between them")
     ap.add_argument("--designs", default="munizen,qwen3", help="with --workload compare-designs: the designs set beside one another "
-                    "(munizen, lunerax, vamadra, pugozen, rapovik; qwen3 is always the last)")
+                    "(munizen, lunerax, vamadra, pugozen, rapovik, lanirax; qwen3 is always the last)")
     ap.add_argument("--workload", default="decode", choices=["decode", "mixed-14b", "batch16-32b", "compare-designs"],
                     help="decode: the headline line (default).  mixed-14b: 32 requests with prompts of 128 to 3,072 tokens at "
                          "Qwen3-14B sizes, prompts cut under a 2,048-token step budget beside the decoding requests, 128 new "

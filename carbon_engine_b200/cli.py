@@ -112,8 +112,8 @@ def cmd_tiny_model(a) -> int:
     from . import models  # noqa: F401
     from .config.qwen3 import Qwen3Config
     from .weights.loader import write_random_model
-    if a.arch not in ("qwen3", "munizen", "lunerax", "vamadra", "pugozen", "rapovik"):
-        raise SystemExit(f"--arch {a.arch}: qwen3, munizen, lunerax, vamadra, pugozen and rapovik are built")
+    if a.arch not in ("qwen3", "munizen", "lunerax", "vamadra", "pugozen", "rapovik", "lanirax"):
+        raise SystemExit(f"--arch {a.arch}: qwen3, munizen, lunerax, vamadra, pugozen, rapovik and lanirax are built")
     heads = a.heads or 4
     head_dim = a.head_dim or 16
     store = {"f32": torch.float32, "bf16": torch.bfloat16}.get(a.dtype)
@@ -151,6 +151,15 @@ def cmd_tiny_model(a) -> int:
         cfg = sketch_config(a.vocab, a.hidden, a.layers, heads, head_dim, a.intermediate or 2 * a.hidden, window=a.mask_size,
                             experts=a.experts, top=a.top_experts, groups=(a.expert_groups, max(1, a.expert_groups // 2)), loop=loop,
                             max_positions=a.max_positions, eps=a.rms_norm_eps, rope_base=a.rope_theta)
+        print(f"wrote {write_random_model(cfg, a.out, seed=a.seed, store_dtype=store)}")
+        return 0
+    if a.arch == "lanirax":
+        # layers go parallel (attention with a window of --mask-size beside the delta rule), attention and again, every one with a
+        # mixture of experts; --shared-from: the layers from that index on run the weights of the layer that many places before them
+        from .config.lanirax import sketch_config
+        cfg = sketch_config(a.vocab, a.hidden, a.layers, heads, a.kv_heads or max(1, heads // 2), head_dim,
+                            a.intermediate or 2 * a.hidden, window=a.mask_size, experts=a.experts, top=a.top_experts,
+                            max_positions=a.max_positions, eps=a.rms_norm_eps, rope_base=a.rope_theta, shared_from=a.shared_from)
         print(f"wrote {write_random_model(cfg, a.out, seed=a.seed, store_dtype=store)}")
         return 0
     if a.arch == "vamadra":
@@ -223,17 +232,17 @@ def main(argv: Optional[List[str]] = None) -> int:
 
     t = sub.add_parser("tiny-model", help="write a small random model folder")
     t.add_argument("--out", required=True)
-    t.add_argument("--arch", default="qwen3", help="qwen3 | munizen | lunerax | vamadra | pugozen | rapovik")
+    t.add_argument("--arch", default="qwen3", help="qwen3 | munizen | lunerax | vamadra | pugozen | rapovik | lanirax")
     t.add_argument("--loop", default="", help="rapovik: START,STOP,TIMES: layers START..STOP-1 run TIMES times in a row")
     t.add_argument("--shared-from", type=int, default=0,
-                   help="pugozen: layers from this index on run the weights of the layer this many places before (0: none)")
-    t.add_argument("--experts", type=int, default=8, help="vamadra, rapovik: experts of a mixture layer")
-    t.add_argument("--top-experts", type=int, default=2, help="vamadra, rapovik: experts a token uses")
+                   help="pugozen, lanirax: layers from this index on run the weights of the layer this many places before (0: none)")
+    t.add_argument("--experts", type=int, default=8, help="vamadra, rapovik, lanirax: experts of a mixture layer")
+    t.add_argument("--top-experts", type=int, default=2, help="vamadra, rapovik, lanirax: experts a token uses")
     t.add_argument("--expert-groups", type=int, default=4, help="vamadra, rapovik: groups the experts form (half of them stay eligible)")
     t.add_argument("--yarn-factor", type=float, default=0.0, help="vamadra: stretch of the rotary frequencies (0: none)")
     t.add_argument("--side-dim", type=int, default=8, help="lunerax: width of the per-layer token input (0: none)")
     t.add_argument("--streams", type=int, default=2, help="munizen: residual streams (0: an ordinary residual)")
-    t.add_argument("--mask-size", type=int, default=256, help="munizen: positions in a block of the attention mask; lunerax, rapovik: the sliding window")
+    t.add_argument("--mask-size", type=int, default=256, help="munizen: positions in a block of the attention mask; lunerax, rapovik, lanirax: the sliding window")
     t.add_argument("--layers", type=int, default=4)
     t.add_argument("--hidden", type=int, default=64)
     t.add_argument("--heads", type=int, default=None)

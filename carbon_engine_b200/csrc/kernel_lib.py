@@ -46,6 +46,8 @@ _SIGNATURES = {
     "ce_rmsnorm_add_norm": (_i, [_p] * 6 + [_i] * 3 + [_f, _f, _p]),
     # y0, y1, wm0, wm1, members, bias, w, x, xb, T, H, alpha, c, eps, eps_m, stream
     "ce_residual_norm": (_i, [_p] * 4 + [_i] + [_p] * 4 + [_i] * 2 + [_f] * 4 + [_p]),
+    # rows, dtype, ld, pair_row, pick_w, top, w, x, xb, T, H, alpha, eps, stream
+    "ce_residual_norm_picks": (_i, [_p, _i, _i, _p, _p, _i] + [_p] * 3 + [_i] * 2 + [_f] * 2 + [_p]),
     # x, n, cap, stream
     "ce_tanh_cap": (_i, [_p, _ll, _f, _p]),
     # src, out, out_dtype, T, ld, off, L, stream
@@ -117,6 +119,10 @@ _SIGNATURES = {
     "ce_diff_attention_mma": (_i, [_p] * 11 + [_i] * 12 + [_f] * 4 + [_p]),
     # z, ids, weights, sgate, T, ld, E, top, groups, keep, scale, correction, scoring, group_score, renormalize, bias, stream
     "ce_moe_route": (_i, [_p] * 4 + [_i] * 6 + [_f, _p, _i, _i, _i, _p, _p]),
+    # N, K, ldh
+    "ce_moe_router_supported": (_i, [_i] * 3),
+    # h, ldh, W, N, K, ids, weights, sgate, T, E, top, groups, keep, scale, correction, scoring, group_score, renormalize, bias, stream
+    "ce_moe_router": (_i, [_p, _i, _p, _i, _i] + [_p] * 3 + [_i] * 5 + [_f, _p, _i, _i, _i, _p, _p]),
     "ce_moe_max_tiles": (_i, [_i, _i, _i]),
     # ids, n_pairs, top, E, BM, max_rows, row_token, pair_row, tile_expert, n_tiles, stream
     "ce_moe_align": (_i, [_p] + [_i] * 5 + [_p] * 5),

@@ -8,8 +8,9 @@
 // src/kernels/attention_tc.cu:682-807).  Each of the 4 warps takes 16 of every 64 staged keys and
 // keeps a running (max, sum, output); the warps are combined in shared memory and the block writes
 // one partial per split to scratch memory; a merge kernel combines the splits in split order
-// (src/kernels/attention_tc.cu:810-830).  Splits are cut at fixed positions, so a sequence's result
-// does not depend on the batch or on the longest sequence beside it.
+// (src/kernels/attention_tc.cu:810-830).  Splits are cut at fixed positions (under a window: counted from the
+// window's first run of AM_SPLIT positions), so a sequence's result does not depend on the batch or on the
+// longest sequence beside it.
 //
 // Prefill: one block per (tile of 64 new tokens of one sequence, query head); each warp owns 16
 // queries, keys are staged 64 at a time, causal and window limits are applied per row
@@ -75,6 +76,9 @@ struct MmaAttnArgs {
     const float* slopes;        // [nh] or null: slopes[h] * (position - key) is taken off head h's scaled scores
 };
 // The kernels that form scores are compiled apart (BIAS) for a penalty on distance, so that the plain scores carry nothing of it.
+
+// The position the splits of a sequence are counted from: under a window, its first run of AM_SPLIT positions.
+__device__ __forceinline__ int first_split_position(const MmaAttnArgs& a, int lo) { return a.window > 0 ? lo / AM_SPLIT * AM_SPLIT : 0; }
 
 // Stage keys [k0, k0 + AM_TILE) of one KV head into shared memory rows of d + AM_PAD elements.
 // Keys outside [lo, hi] are filled with zeros, so that a masked probability of 0 never meets a NaN.
@@ -256,8 +260,9 @@ __global__ void __launch_bounds__(AM_THREADS) attention_decode_kernel(MmaAttnArg
     int t = b;                                    // one-token sequences come first: sequence b brings token b
     int pos = a.positions[t];
     int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;
-    int k_begin = split * a.split, k_end = min(k_begin + a.split, pos + 1);
+    int k_begin = first_split_position(a, lo) + split * a.split, k_end = min(k_begin + a.split, pos + 1);
     if (k_begin > pos || k_end <= lo) return;     // the merge kernel skips these splits too
+    k_begin = max(k_begin, lo / AM_TILE * AM_TILE);      // whole tiles below the window are not even looked up
     const int* table = a.block_table + (size_t)a.seq_slot[b] * a.max_pages;
     int d = a.d, ld = d + AM_PAD;
     bf16* Ks = reinterpret_cast<bf16*>(smem_raw);
@@ -367,7 +372,7 @@ __global__ void __launch_bounds__(AM_THREADS) attention_decode_kernel(MmaAttnArg
     __shared__ int s_ticket;
     __threadfence();
     __syncthreads();
-    int s0 = lo / a.split, s1 = pos / a.split, ns = s1 - s0 + 1;       // the splits that hold visible keys
+    int p0 = first_split_position(a, lo), s0 = (lo - p0) / a.split, s1 = (pos - p0) / a.split, ns = s1 - s0 + 1;       // the splits that hold visible keys
     int cidx = (b * a.nkv + kvh) * gridDim.z + hg;
     if (threadIdx.x == 0) s_ticket = atomicAdd(&a.counters[cidx], 1);
     __syncthreads();
@@ -562,8 +567,9 @@ __global__ void __launch_bounds__(AMT_THREADS) attention_decode_tma_kernel(const
     int t = b;
     int pos = a.positions[t];
     int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;
-    int k_begin = split * a.split, k_end = min(k_begin + a.split, pos + 1);
+    int k_begin = first_split_position(a, lo) + split * a.split, k_end = min(k_begin + a.split, pos + 1);
     bool idle = k_begin > pos || k_end <= lo;     // no visible key in this split: the merge skips it
+    k_begin = max(k_begin, lo / AM_TILE * AM_TILE);      // whole tiles below the window are not even looked up
     if (idle && !a.cluster_merge) return;
     const int* table = a.block_table + (size_t)a.seq_slot[b] * a.max_pages;
     int d = a.d, panels = d >> 6;
@@ -791,7 +797,8 @@ __global__ void attention_merge_kernel(MmaAttnArgs a) {
     int t = a.q_start[b];
     int pos = a.positions[t];
     int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;
-    int s0 = lo / a.split, s1 = pos / a.split;                  // splits that hold visible keys
+    int p0 = first_split_position(a, lo);
+    int s0 = (lo - p0) / a.split, s1 = (pos - p0) / a.split;    // splits that hold visible keys
     int ns = s1 - s0 + 1;
     size_t base = ((size_t)b * a.nh + h) * a.max_splits + s0;
     if (threadIdx.x < 32) {
@@ -986,6 +993,10 @@ extern "C" int ce_attention_decode_bf16_sink(const void* q, const void* k_pool, 
     if (rc) return rc;
     if (max_splits <= 0 || (long long)n_seqs * max_splits > 2147483647LL)
         return ce_fail(CE_ERR_SIZE, "ce_attention_decode_bf16: %d sequences x %d splits", n_seqs, max_splits);
+    if (window > 0) {                    // a window spans at most this many runs of AM_SPLIT positions, whatever the context
+        long long runs = ((long long)window + 2 * AM_SPLIT - 2) / AM_SPLIT;
+        if (runs < max_splits) max_splits = (int)runs;
+    }
     MmaAttnArgs a{};
     a.q = (const bf16*)q; a.k_pool = (const bf16*)k_pool; a.v_pool = (const bf16*)v_pool; a.out = (bf16*)out;
     a.part_o = scratch; a.part_ml = scratch + (size_t)n_seqs * nh * max_splits * d;

@@ -151,7 +151,9 @@ struct TcAttnArgs {
     const float* slopes;        // [nh] or null: slopes[h] * (position - key) is taken off head h's scaled scores
 };
 
-// BIAS: a penalty that grows with a key's distance (``slopes``), compiled apart so that the plain scores carry nothing of it
+// BIAS: a penalty that grows with a key's distance (``slopes``), compiled apart so that the plain scores carry nothing of it.  The
+// key tiles are then walked from the nearest to the farthest: in the other order the penalty falls from tile to tile, a steep
+// head's running maximum would rise at every one, and each time the output accumulator would have to be rescaled.
 template <int D, bool BIAS>
 __global__ void __launch_bounds__(THREADS) attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
                                                                       const __grid_constant__ CUtensorMap map_k,
@@ -233,7 +235,7 @@ __global__ void __launch_bounds__(THREADS) attention_prefill_tc_kernel(const __g
             // one tile of K or V: pieces of a page, 64 columns a copy
             auto load_tile = [&](const CUtensorMap* map, unsigned char* dst, uint64_t* bar, int j) {
                 mbar_expect_tx(bar, K_BYTES);
-                int k0 = k_begin + j * BN;
+                int k0 = k_begin + (BIAS ? n_kv - 1 - j : j) * BN;
                 for (int r = 0; r < BN; r += box_rows) {
                     int key = k0 + r;
                     int page = key <= p_last ? table[key >> a.page_shift] : -1;
@@ -328,7 +330,7 @@ __global__ void __launch_bounds__(THREADS) attention_prefill_tc_kernel(const __g
         bool ok = true;
         int where = 66;                                        // 66..68: which wait of the softmax warps gave up
         for (int j = 0; j < n_kv; ++j) {
-            int k0 = k_begin + j * BN;
+            int k0 = k_begin + (BIAS ? n_kv - 1 - j : j) * BN;
             where = 66;
             if (!warp_wait(&s_full, j & 1)) { ok = false; break; }
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");

@@ -100,6 +100,27 @@ template <> struct CeType<__nv_bfloat16> {
     static __device__ __forceinline__ void store(__nv_bfloat16* p, float v) { *p = __float2bfloat16_rn(v); }
 };
 
+// four consecutive elements as float32
+__device__ __forceinline__ float4 ce_load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 ce_load4(const __nv_bfloat16* p) {
+    uint2 r = *reinterpret_cast<const uint2*>(p);
+    float2 lo = __bfloat1622float2(*reinterpret_cast<__nv_bfloat162*>(&r.x)), hi = __bfloat1622float2(*reinterpret_cast<__nv_bfloat162*>(&r.y));
+    return make_float4(lo.x, lo.y, hi.x, hi.y);
+}
+
+// Columns j .. j + 3 of a token's weighted sum of its experts' rows: sum_k weights[k] rows[pair_row[k]], in the order of k.
+template <typename T>
+__device__ __forceinline__ float4 ce_sum_picks4(const T* rows, int ld, const int* pair_row, const float* weights, int top, int j) {
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+    for (int k = 0; k < top; ++k) {
+        const float w = weights[k];
+        const float4 r = ce_load4(rows + (size_t)pair_row[k] * ld + j);
+        v.x = fmaf(w, r.x, v.x); v.y = fmaf(w, r.y, v.y); v.z = fmaf(w, r.z, v.z); v.w = fmaf(w, r.w, v.w);
+    }
+    return v;
+}
+
 // Sum over a block in a fixed order: warp shuffles down, then warp 0 adds the warp sums in index
 // order.  The result depends on blockDim only, never on the grid or on other rows.
 __device__ __forceinline__ float ce_block_sum(float v, float* scratch /* >= 32 floats */) {

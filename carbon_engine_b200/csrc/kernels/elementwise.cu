@@ -43,7 +43,8 @@ extern "C" int ce_embed(const void* table, int dtype, const int* tokens, float* 
 // Embedding gather with a norm: x[t, :] = v / sqrt(mean(v^2) + eps) * w,  v = table[tok[t], :] * scale.  xb (or null) receives
 // the row rounded to bfloat16 too, for a sublayer that reads the residual itself.
 // ---------------------------------------------------------------------------------------------
-template <typename T>
+#define EN_MAX 4
+template <typename T, bool VEC>
 __global__ void embed_norm_kernel(const T* __restrict__ table, const int* __restrict__ tokens, const float* __restrict__ w,
                                   float* __restrict__ x, __nv_bfloat16* __restrict__ xb, int H, int V, int* status, float scale, float eps) {
     ce_pdl_begin();
@@ -52,6 +53,32 @@ __global__ void embed_norm_kernel(const T* __restrict__ table, const int* __rest
     const bool there = tok >= 0 && tok < V;
     if (!there && threadIdx.x == 0) atomicExch(status, 1);
     const T* row = table + (size_t)(there ? tok : 0) * H;
+    if (VEC) {                           // four elements at a time, the row in registers
+        const int H4 = H >> 2;
+        float4 v[EN_MAX];
+        float ss = 0.f;
+#pragma unroll
+        for (int n = 0; n < EN_MAX; ++n) {
+            int j = threadIdx.x + n * blockDim.x;
+            v[n] = j < H4 ? ce_load4(row + 4 * j) : make_float4(0.f, 0.f, 0.f, 0.f);
+            v[n].x *= scale; v[n].y *= scale; v[n].z *= scale; v[n].w *= scale;
+            ss += (v[n].x * v[n].x + v[n].y * v[n].y) + (v[n].z * v[n].z + v[n].w * v[n].w);
+        }
+        const float inv = there ? 1.0f / sqrtf(ce_block_sum(ss, scratch) / (float)H + eps) : 0.f;
+#pragma unroll
+        for (int n = 0; n < EN_MAX; ++n) {
+            int j = threadIdx.x + n * blockDim.x;
+            if (j >= H4) continue;
+            const float4 ww = ce_load4(w + 4 * j);
+            const float4 o = make_float4(v[n].x * inv * ww.x, v[n].y * inv * ww.y, v[n].z * inv * ww.z, v[n].w * inv * ww.w);
+            *reinterpret_cast<float4*>(x + (size_t)t * H + 4 * j) = o;
+            if (xb) {
+                __nv_bfloat162 lo = __floats2bfloat162_rn(o.x, o.y), hi = __floats2bfloat162_rn(o.z, o.w);
+                *reinterpret_cast<uint2*>(xb + (size_t)t * H + 4 * j) = make_uint2(*reinterpret_cast<uint32_t*>(&lo), *reinterpret_cast<uint32_t*>(&hi));
+            }
+        }
+        return;
+    }
     float ss = 0.f;
     for (int j = threadIdx.x; j < H; j += blockDim.x) { float v = CeType<T>::load(row + j) * scale; ss = fmaf(v, v, ss); }
     float inv = 1.0f / sqrtf(ce_block_sum(ss, scratch) / (float)H + eps);
@@ -62,15 +89,24 @@ __global__ void embed_norm_kernel(const T* __restrict__ table, const int* __rest
     }
 }
 
+template <typename T>
+static void embed_norm_launch(const T* table, const int* tokens, const float* w, float* x, __nv_bfloat16* xb, int n, int H, int V, int* status,
+                              float scale, float eps, cudaStream_t stream) {
+    const int H4 = H / 4, vt = H4 >= 2048 ? 1024 : H4 >= 512 ? 512 : H4 >= 256 ? 256 : 128;
+    if (H % 4 == 0 && H4 <= vt * EN_MAX && ((((uintptr_t)table | (uintptr_t)w | (uintptr_t)x | (uintptr_t)xb) & 15) == 0))
+        ce_launch(embed_norm_kernel<T, true>, n, vt, 0, stream, table, tokens, w, x, xb, H, V, status, scale, eps);
+    else
+        ce_launch(embed_norm_kernel<T, false>, n, H >= 1024 ? 1024 : 256, 0, stream, table, tokens, w, x, xb, H, V, status, scale, eps);
+}
+
 extern "C" int ce_embed_norm(const void* table, int dtype, const int* tokens, const float* w, float* x, void* xb, int T, int H, int V,
                              int* status, float scale, float eps, cudaStream_t stream) {
     if (T == 0) return CE_OK;
     if (!table || !tokens || !w || !x || !status) return ce_fail(CE_ERR_ARG, "ce_embed_norm: null pointer");
     if (H <= 0 || V <= 0) return ce_fail(CE_ERR_SIZE, "ce_embed_norm: width %d, vocabulary %d", H, V);
-    int threads = H >= 1024 ? 1024 : 256;
     ce_note("embed_norm_kernel");
-    if (dtype == CE_F32) ce_launch(embed_norm_kernel<float>, T, threads, 0, stream, (const float*)table, tokens, w, x, (__nv_bfloat16*)xb, H, V, status, scale, eps);
-    else if (dtype == CE_BF16) ce_launch(embed_norm_kernel<__nv_bfloat16>, T, threads, 0, stream, (const __nv_bfloat16*)table, tokens, w, x, (__nv_bfloat16*)xb, H, V, status, scale, eps);
+    if (dtype == CE_F32) embed_norm_launch((const float*)table, tokens, w, x, (__nv_bfloat16*)xb, T, H, V, status, scale, eps, stream);
+    else if (dtype == CE_BF16) embed_norm_launch((const __nv_bfloat16*)table, tokens, w, x, (__nv_bfloat16*)xb, T, H, V, status, scale, eps, stream);
     else return ce_fail(CE_ERR_ARG, "ce_embed_norm: unknown dtype %d", dtype);
     return ce_check_launch("ce_embed_norm");
 }

@@ -253,6 +253,7 @@ extern "C" int ce_rmsnorm_add_norm(const float* y, const float* bias, const floa
 // ---------------------------------------------------------------------------------------------
 // The norm after the sum:  z = alpha x[t] + s,  x[t] = z / sqrt(mean(z^2) + eps) * w,  s the sublayer's output,
 //   NM 0  y0[t] (+ bias), as it is
+//   NM 3, 4  sum_k pick_w[t, k] rows[pair_row[t, k]], the weighted sum of a token's experts (rows float32 / bfloat16)
 //   NM 1, 2  c * sum_m y_m[t] / sqrt(mean(y_m[t]^2) + eps_m) * w_m: the outputs of mixers side by side, each normed over the width
 // store_only: s itself is stored in x (or, with alpha 1, added to it) and no norm is taken of the sum.
 // xb (or null) receives the new x rounded to bfloat16.  VEC: float4 accesses, a row in registers.
@@ -266,6 +267,10 @@ struct ResidualNormArgs {
     __nv_bfloat16* xb;
     int H;
     float alpha, c, eps, eps_m;
+    const void* rows;            // NM 3, 4: [*, ld]
+    const int* pair_row;         // [T, top]
+    const float* pick_w;         // [T, top]
+    int ld, top;
 };
 
 template <int NM, bool VEC>
@@ -273,7 +278,8 @@ __global__ void residual_norm_kernel(ResidualNormArgs a) {
     ce_pdl_begin();
     __shared__ float scratch[32];
     const int t = blockIdx.x, tid = threadIdx.x, H = a.H;
-    constexpr int NY = NM == 0 ? 1 : NM;
+    constexpr bool PICKS = NM >= 3;
+    constexpr int NY = NM == 2 ? 2 : 1;
     float inv_m[NY];
     if (VEC) {
         const int H4 = H >> 2;
@@ -284,14 +290,18 @@ __global__ void residual_norm_kernel(ResidualNormArgs a) {
 #pragma unroll
             for (int n = 0; n < LNV_MAX; ++n) {
                 int j = tid + n * blockDim.x;
-                v[m][n] = j < H4 ? reinterpret_cast<const float4*>(a.y[m] + (size_t)t * H)[j] : make_float4(0.f, 0.f, 0.f, 0.f);
+                v[m][n] = make_float4(0.f, 0.f, 0.f, 0.f);
+                if (j >= H4) continue;
+                if (NM == 3) v[m][n] = ce_sum_picks4((const float*)a.rows, a.ld, a.pair_row + (size_t)t * a.top, a.pick_w + (size_t)t * a.top, a.top, 4 * j);
+                else if (NM == 4) v[m][n] = ce_sum_picks4((const __nv_bfloat16*)a.rows, a.ld, a.pair_row + (size_t)t * a.top, a.pick_w + (size_t)t * a.top, a.top, 4 * j);
+                else v[m][n] = reinterpret_cast<const float4*>(a.y[m] + (size_t)t * H)[j];
             }
 #pragma unroll
         for (int n = 0; n < LNV_MAX; ++n) {
             int j = tid + n * blockDim.x;
             z[n] = j < H4 && a.alpha != 0.f ? xr[j] : make_float4(0.f, 0.f, 0.f, 0.f);
         }
-        if (NM > 0) {
+        if (NM > 0 && !PICKS) {
 #pragma unroll
             for (int m = 0; m < NY; ++m) {
                 float q = 0.f;
@@ -306,9 +316,9 @@ __global__ void residual_norm_kernel(ResidualNormArgs a) {
             int j = tid + n * blockDim.x;
             if (j >= H4) continue;
             float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
-            if (NM == 0) {
+            if (NM == 0 || PICKS) {
                 s = v[0][n];
-                if (a.bias) { float4 b = reinterpret_cast<const float4*>(a.bias)[j]; s.x += b.x; s.y += b.y; s.z += b.z; s.w += b.w; }
+                if (NM == 0 && a.bias) { float4 b = reinterpret_cast<const float4*>(a.bias)[j]; s.x += b.x; s.y += b.y; s.z += b.z; s.w += b.w; }
             } else {
 #pragma unroll
                 for (int m = 0; m < NY; ++m) {
@@ -340,7 +350,7 @@ __global__ void residual_norm_kernel(ResidualNormArgs a) {
         }
     } else {
         float* xr = a.x + (size_t)t * H;
-        if (NM > 0) {
+        if (NM > 0 && !PICKS) {
 #pragma unroll
             for (int m = 0; m < NY; ++m) {
                 float q = 0.f;
@@ -352,7 +362,12 @@ __global__ void residual_norm_kernel(ResidualNormArgs a) {
         for (int j = tid; j < H; j += blockDim.x) {
             float s = 0.f;
             if (NM == 0) s = a.y[0][(size_t)t * H + j] + (a.bias ? a.bias[j] : 0.f);
-            else {
+            else if (PICKS) {
+                for (int k = 0; k < a.top; ++k) {
+                    const size_t at = (size_t)a.pair_row[(size_t)t * a.top + k] * a.ld + j;
+                    s = fmaf(a.pick_w[(size_t)t * a.top + k], NM == 3 ? ((const float*)a.rows)[at] : __bfloat162float(((const __nv_bfloat16*)a.rows)[at]), s);
+                }
+            } else {
 #pragma unroll
                 for (int m = 0; m < NY; ++m) s += a.y[m][(size_t)t * H + j] * inv_m[m] * a.wm[m][j];
                 s *= a.c;
@@ -387,7 +402,7 @@ extern "C" int ce_residual_norm(const float* y0, const float* y1, const float* w
     if (!y0 || !x || members < 0 || members > 2 || (members > 0 && !wm0) || (members > 1 && (!wm1 || !y1)) || (members > 0 && bias))
         return ce_fail(CE_ERR_ARG, "ce_residual_norm: null pointer, or %d members", members);
     if (H <= 0) return ce_fail(CE_ERR_SIZE, "ce_residual_norm: width %d", H);
-    ResidualNormArgs a{{y0, y1}, {wm0, wm1}, bias, w, x, (__nv_bfloat16*)xb, H, alpha, c, eps, eps_m};
+    ResidualNormArgs a{{y0, y1}, {wm0, wm1}, bias, w, x, (__nv_bfloat16*)xb, H, alpha, c, eps, eps_m, nullptr, nullptr, nullptr, 0, 0};
     bool vec = H % 4 == 0 && H >= 256 && ((((uintptr_t)y0 | (uintptr_t)y1 | (uintptr_t)wm0 | (uintptr_t)wm1 | (uintptr_t)bias |
                                             (uintptr_t)w | (uintptr_t)x | (uintptr_t)xb) & 15) == 0);
     ce_note("residual_norm_kernel");
@@ -395,6 +410,22 @@ extern "C" int ce_residual_norm(const float* y0, const float* y1, const float* w
     else if (members == 1) residual_norm_launch<1>(a, T, vec, stream);
     else residual_norm_launch<2>(a, T, vec, stream);
     return ce_check_launch("ce_residual_norm");
+}
+
+// The same with the weighted sum of a token's experts as the sublayer's output: rows [*, ld] (float32 or bfloat16), pair_row and
+// pick_w [T, top] as ce_moe_combine takes them.
+extern "C" int ce_residual_norm_picks(const void* rows, int dtype, int ld, const int* pair_row, const float* pick_w, int top, const float* w,
+                                      float* x, void* xb, int T, int H, float alpha, float eps, cudaStream_t stream) {
+    if (T == 0) return CE_OK;
+    if (!rows || !pair_row || !pick_w || !w || !x) return ce_fail(CE_ERR_ARG, "ce_residual_norm_picks: null pointer");
+    if (H <= 0 || ld < H || top <= 0 || (dtype != CE_F32 && dtype != CE_BF16))
+        return ce_fail(CE_ERR_SIZE, "ce_residual_norm_picks: width %d, rows of %d, %d picks, dtype %d", H, ld, top, dtype);
+    ResidualNormArgs a{{nullptr, nullptr}, {nullptr, nullptr}, nullptr, w, x, (__nv_bfloat16*)xb, H, alpha, 1.0f, eps, 0.f, rows, pair_row, pick_w, ld, top};
+    bool vec = H % 4 == 0 && ld % 4 == 0 && H >= 256 && ((((uintptr_t)rows | (uintptr_t)w | (uintptr_t)x | (uintptr_t)xb) & 15) == 0);
+    ce_note("residual_norm_kernel (weighted sum of experts)");
+    if (dtype == CE_F32) residual_norm_launch<3>(a, T, vec, stream);
+    else residual_norm_launch<4>(a, T, vec, stream);
+    return ce_check_launch("ce_residual_norm_picks");
 }
 
 // xb (or null): receives the new x rounded to bfloat16, what a sublayer that reads the residual itself takes as its input

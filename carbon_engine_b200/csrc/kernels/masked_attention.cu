@@ -173,7 +173,7 @@ static void norm_rope_launch(const NormRopeArgs& a, dim3 grid, int threads, cuda
     if (a.d <= 64) ce_launch(norm_rope_kvwrite_kernel<T, 2>, grid, threads, 0, stream, a);
     else if (a.d <= 128) ce_launch(norm_rope_kvwrite_kernel<T, 4>, grid, threads, 0, stream, a);
     else if (a.d <= 256) ce_launch(norm_rope_kvwrite_kernel<T, 8>, grid, threads, 0, stream, a);
-    else ce_launch(norm_rope_kvwrite_kernel<T, 64>, grid, threads, 0, stream, a);
+    else ce_launch(norm_rope_kvwrite_kernel<T, 32>, grid, threads, 0, stream, a);
 }
 
 extern "C" int ce_norm_rope_kvwrite(const float* proj, void* q_out, void* k_pool, void* v_pool, int dtype, const float* wq,
@@ -187,7 +187,7 @@ extern "C" int ce_norm_rope_kvwrite(const float* proj, void* q_out, void* k_pool
     if (write_kv && (!k_pool || !v_pool || !block_table)) return ce_fail(CE_ERR_ARG, "ce_norm_rope_kvwrite: no cache to write to");
     if (rd < 0 || rd > d || rd % 2) return ce_fail(CE_ERR_SIZE, "ce_norm_rope_kvwrite: %d rotated elements of %d", rd, d);
     if (rd > 0 && (!cos_table || !sin_table)) return ce_fail(CE_ERR_ARG, "ce_norm_rope_kvwrite: no rotation tables");
-    if (nh <= 0 || nkv <= 0 || d <= 0 || d > 2048 || dv <= 0) return ce_fail(CE_ERR_SIZE, "ce_norm_rope_kvwrite: sizes");
+    if (nh <= 0 || nkv <= 0 || d <= 0 || d > 1024 || dv <= 0) return ce_fail(CE_ERR_SIZE, "ce_norm_rope_kvwrite: sizes");
     if (norm_mode < 0 || norm_mode > 2 || (norm_mode == 1 && (!wq || !wk)) || (pairing != 0 && pairing != 1))
         return ce_fail(CE_ERR_ARG, "ce_norm_rope_kvwrite: norm mode %d, pairing %d", norm_mode, pairing);
     NormRopeArgs a{proj, q_out, k_pool, v_pool, wq, wk, head_scale, pos_scale, rd > 0 ? cos_table : nullptr, sin_table, positions,

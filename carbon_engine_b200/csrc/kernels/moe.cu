@@ -2,19 +2,21 @@
 // grouped products over that layout, and the weighted sum back into token order.
 //
 //   route    z [T, ld] float32 router logits (+ a bias per expert) -> s = softmax(z[:E]) or sigmoid(z[:E]), or, for a softmax over
-//            the chosen logits only, s = exp(z - max z) and choice by z itself; choice scores c = s (+ a correction per expert); experts in `groups` equal groups of neighbours, a group's score the largest c in it or the sum of its two
-//            largest, only the best `keep` groups' experts eligible; the `top` eligible experts with the largest c are chosen
+//            the chosen logits only, s = exp(z - max z) and choice by z itself; choice scores c = s (+ a correction per expert);
+//            experts in `groups` equal groups of neighbours, a group's score the largest c in it or the sum of its two largest,
+//            only the best `keep` groups' experts eligible; the `top` eligible experts with the largest c are chosen
 //            (ties: the lower index); weights s / (sum of the chosen s + 1e-20) * scale, or s * scale as they are.
 //            Column E of z, where there is one, is the logit of a shared expert's gate: sgate[t] = sigmoid(z[t, E]).
+//            In bfloat16, for routers of up to 128 rows, the product that gives z is part of the kernel.
 //   align    the T*top pairs sorted by expert into rows of a padded layout: every expert's rows start at a multiple of
 //            the tile height BM, so a tile of BM rows belongs to ONE expert.  row_token[p] is the token of row p (-1: a
 //            padding row), pair_row[i] the row of pair i, tile_expert[j] the expert of tile j, n_tiles[0] their count.
 //            Nothing of it reaches the host: the products launch a grid for the most tiles a step of that size can have,
 //            and blocks past n_tiles leave at once, so a captured graph replays with any routing.
 //   products out[p] = act(in[row p's token, or p] W[e]^T), e = tile_expert[p / BM]; act = none, relu^2, or a gated
-//            activation of row pairs (rows 2j and 2j + 1 of W[e] are feature j's gate and up): the clamped one, or silu(gate) up.  Every output
-//            element is a sum over k in a fixed order that depends on neither the row's place in its tile nor on the
-//            other rows, so a token's result does not depend on the batch.  float32 FMA for any size and both dtypes;
+//            activation of row pairs (rows 2j and 2j + 1 of W[e] are feature j's gate and up): the clamped one, or
+//            silu(gate) up.  Every output element is a sum over k in a fixed order that depends on neither the row's place in
+//            its tile nor on the other rows, so a token's result does not depend on the batch.  float32 FMA for any size and both dtypes;
 //            bfloat16 on the tensor cores (wmma m16n16k16, float32 sums) for sizes in multiples of 16.
 //   combine  y[t] (+)= sum_k weight[t, k] out[pair_row[t*top + k]] + sgate[t] shared[t], in the order of k, float32.
 #include "common.cuh"
@@ -47,16 +49,9 @@ __device__ __forceinline__ void moe_warp_argmax(float& v, int& i) {
     }
 }
 
-__global__ void __launch_bounds__(128) moe_route_kernel(MoeRouteArgs a) {
-    ce_pdl_begin();
-    extern __shared__ float moe_route_smem[];
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int t = blockIdx.x * 4 + warp;
-    if (t >= a.T) return;
-    float* s = moe_route_smem + (size_t)warp * 3 * a.E;      // scores
-    float* c = s + a.E;                                      // choice scores; a chosen or barred expert's becomes -inf
-    float* gs = c + a.E;                                     // the groups' scores; a kept group's becomes +inf
-    const float* zr = a.z + (size_t)t * a.ld;
+// One token, one warp.  zr: the token's logits; s, c, gs: E floats of shared memory each: the scores; the choice scores (a chosen
+// or barred expert's becomes -inf); the groups' scores (a kept group's becomes +inf).
+__device__ __forceinline__ void moe_route_token(const MoeRouteArgs& a, int t, int lane, const float* zr, float* s, float* c, float* gs) {
     for (int e = lane; e < a.E; e += 32) c[e] = a.bias ? zr[e] + a.bias[e] : zr[e];       // the logits (each lane its own experts')
     if (a.scoring != 1) {
         float mx = -INFINITY;
@@ -121,24 +116,131 @@ __global__ void __launch_bounds__(128) moe_route_kernel(MoeRouteArgs a) {
     if (a.sgate && lane == 0) a.sgate[t] = 1.0f / (1.0f + expf(-zr[a.E]));
 }
 
+__global__ void __launch_bounds__(128) moe_route_kernel(MoeRouteArgs a) {
+    ce_pdl_begin();
+    extern __shared__ float moe_route_smem[];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int t = blockIdx.x * 4 + warp;
+    if (t >= a.T) return;
+    float* s = moe_route_smem + (size_t)warp * 3 * a.E;
+    moe_route_token(a, t, lane, a.z + (size_t)t * a.ld, s, s + a.E, s + 2 * a.E);
+}
+
+// The router's product and the routing in one kernel (bfloat16): a block of 16 warps takes 16 tokens; the warps share K in runs of
+// 32, each a product of the 16 tokens with all experts (mma.sync m16n8k16), and the partial logits are added in the warps' order
+// (float32): a token's logits depend on neither its place nor on the other tokens.  Within a run the elements of K are dealt to the
+// products so that every lane reads 16 consecutive bytes of a row (the same for both operands).  Then a warp routes a token.
+#define MR_WARPS 16
+struct MoeRouterArgs {
+    const __nv_bfloat16* h;      // [T, ldh]
+    const __nv_bfloat16* W;      // [N, K]: the experts' rows, then the shared expert's gate row where there is one
+    int ldh, N, K;
+};
+
+template <int NT>
+__global__ void __launch_bounds__(32 * MR_WARPS) moe_router_kernel(MoeRouterArgs r, MoeRouteArgs a) {
+    ce_pdl_begin();
+    extern __shared__ float moe_router_smem[];
+    constexpr int NE = NT * 8;
+    float* part = moe_router_smem;                           // [warps][16][NE]; the routing's work space afterwards
+    float* z = part + MR_WARPS * 16 * NE;                    // [16][NE]
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, grp = lane >> 2, quad = lane & 3;
+    const int t0 = blockIdx.x * 16;
+    const __nv_bfloat16* ha = r.h + (size_t)min(t0 + grp, a.T - 1) * r.ldh + quad * 8;
+    const __nv_bfloat16* hb = r.h + (size_t)min(t0 + grp + 8, a.T - 1) * r.ldh + quad * 8;
+    float acc[NT][4];
+#pragma unroll
+    for (int n = 0; n < NT; ++n) acc[n][0] = acc[n][1] = acc[n][2] = acc[n][3] = 0.f;
+#pragma unroll 2
+    for (int k0 = warp * 32; k0 < r.K; k0 += MR_WARPS * 32) {
+        const uint4 x = *reinterpret_cast<const uint4*>(ha + k0), y = *reinterpret_cast<const uint4*>(hb + k0);
+#pragma unroll
+        for (int n = 0; n < NT; ++n) {
+            const uint4 w = *reinterpret_cast<const uint4*>(r.W + (size_t)min(n * 8 + grp, r.N - 1) * r.K + quad * 8 + k0);
+            asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                         : "+f"(acc[n][0]), "+f"(acc[n][1]), "+f"(acc[n][2]), "+f"(acc[n][3]) : "r"(x.x), "r"(y.x), "r"(x.y), "r"(y.y), "r"(w.x), "r"(w.y));
+            asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                         : "+f"(acc[n][0]), "+f"(acc[n][1]), "+f"(acc[n][2]), "+f"(acc[n][3]) : "r"(x.z), "r"(y.z), "r"(x.w), "r"(y.w), "r"(w.z), "r"(w.w));
+        }
+    }
+#pragma unroll
+    for (int n = 0; n < NT; ++n) {
+        float* p = part + (warp * 16 + grp) * NE + n * 8 + 2 * quad;
+        p[0] = acc[n][0]; p[1] = acc[n][1];
+        p[8 * NE] = acc[n][2]; p[8 * NE + 1] = acc[n][3];
+    }
+    __syncthreads();
+    for (int e = threadIdx.x; e < 16 * NE; e += blockDim.x) {
+        float v = 0.f;
+#pragma unroll
+        for (int w = 0; w < MR_WARPS; ++w) v += part[w * 16 * NE + e];
+        z[e] = v;
+    }
+    __syncthreads();
+    if (t0 + warp >= a.T) return;
+    float* s = part + (size_t)warp * 3 * a.E;                // (16 warps x 3 E floats: less than the partial logits took)
+    moe_route_token(a, t0 + warp, lane, z + warp * NE, s, s + a.E, s + 2 * a.E);
+}
+
+static int check_route(const char* who, const int* ids, const float* weights, int E, int top, int groups, int keep, int columns, bool gate,
+                       const float* correction, int scoring, int group_score, int renormalize) {
+    if (!ids || !weights) return ce_fail(CE_ERR_ARG, "%s: null pointer", who);
+    if (E <= 0 || E > MOE_MAX_EXPERTS || top <= 0 || top > E || groups <= 0 || E % groups || keep <= 0 || keep > groups ||
+        (long long)keep * (E / groups) < top || columns < E + (gate ? 1 : 0))
+        return ce_fail(CE_ERR_SIZE, "%s: %d experts, top %d, %d groups of which %d are kept", who, E, top, groups, keep);
+    if (scoring == 2 && (correction || !renormalize))
+        return ce_fail(CE_ERR_ARG, "%s: a softmax over the chosen logits takes no correction and sums to the scale", who);
+    if (scoring < 0 || scoring > 2 || group_score < 0 || group_score > 1)
+        return ce_fail(CE_ERR_ARG, "%s: scoring %d, group score %d", who, scoring, group_score);
+    return CE_OK;
+}
+
 extern "C" int ce_moe_route(const float* z, int* ids, float* weights, float* sgate, int T, int ld, int E, int top, int groups,
                             int keep, float scale, const float* correction, int scoring, int group_score, int renormalize,
                             const float* bias, cudaStream_t stream) {
     if (T == 0) return CE_OK;
-    if (!z || !ids || !weights) return ce_fail(CE_ERR_ARG, "ce_moe_route: null pointer");
-    if (E <= 0 || E > MOE_MAX_EXPERTS || top <= 0 || top > E || groups <= 0 || E % groups || keep <= 0 || keep > groups ||
-        (long long)keep * (E / groups) < top || ld < E + (sgate ? 1 : 0))
-        return ce_fail(CE_ERR_SIZE, "ce_moe_route: %d experts, top %d, %d groups of which %d are kept", E, top, groups, keep);
-    if (scoring == 2 && (correction || !renormalize))
-        return ce_fail(CE_ERR_ARG, "ce_moe_route: a softmax over the chosen logits takes no correction and sums to the scale");
-    if (scoring < 0 || scoring > 2 || group_score < 0 || group_score > 1)
-        return ce_fail(CE_ERR_ARG, "ce_moe_route: scoring %d, group score %d", scoring, group_score);
+    if (!z) return ce_fail(CE_ERR_ARG, "ce_moe_route: null pointer");
+    int rc = check_route("ce_moe_route", ids, weights, E, top, groups, keep, ld, sgate != nullptr, correction, scoring, group_score, renormalize);
+    if (rc) return rc;
     MoeRouteArgs a{z, ids, weights, sgate, T, ld, E, top, groups, keep, scale, correction, scoring, group_score, renormalize, bias};
     size_t smem = (size_t)4 * 3 * E * sizeof(float);
     if (smem > 40 * 1024) cudaFuncSetAttribute(moe_route_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     ce_note("moe_route_kernel");
     ce_launch(moe_route_kernel, (T + 3) / 4, 128, smem, stream, a);
     return ce_check_launch("ce_moe_route");
+}
+
+// rows of W (experts, and the gate) and elements of W that ce_moe_router takes: all of W passes through every block
+extern "C" int ce_moe_router_supported(int N, int K, int ldh) {
+    return N > 0 && N <= 128 && K >= 32 && K % 32 == 0 && ldh % 8 == 0 && (long long)N * K <= (1 << 20);
+}
+
+template <int NT>
+static void moe_router_launch(const MoeRouterArgs& r, const MoeRouteArgs& a, cudaStream_t stream) {
+    size_t smem = (size_t)(MR_WARPS + 1) * 16 * NT * 8 * sizeof(float);
+    if (smem > 40 * 1024) cudaFuncSetAttribute(moe_router_kernel<NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    ce_launch(moe_router_kernel<NT>, (a.T + 15) / 16, 32 * MR_WARPS, smem, stream, r, a);
+}
+
+// ce_moe_route with the router's product in the same kernel: h [T, ldh] bf16, W [>= N, K] bf16, N = E (+ 1 with sgate)
+extern "C" int ce_moe_router(const void* h, int ldh, const void* W, int N, int K, int* ids, float* weights, float* sgate, int T, int E,
+                             int top, int groups, int keep, float scale, const float* correction, int scoring, int group_score,
+                             int renormalize, const float* bias, cudaStream_t stream) {
+    if (T == 0) return CE_OK;
+    if (!h || !W) return ce_fail(CE_ERR_ARG, "ce_moe_router: null pointer");
+    if (!ce_moe_router_supported(N, K, ldh) || ldh < K || (((uintptr_t)h | (uintptr_t)W) & 15))
+        return ce_fail(CE_ERR_SIZE, "ce_moe_router: %d rows of %d, row stride %d", N, K, ldh);
+    int rc = check_route("ce_moe_router", ids, weights, E, top, groups, keep, N, sgate != nullptr, correction, scoring, group_score, renormalize);
+    if (rc) return rc;
+    MoeRouterArgs r{(const __nv_bfloat16*)h, (const __nv_bfloat16*)W, ldh, N, K};
+    MoeRouteArgs a{nullptr, ids, weights, sgate, T, N, E, top, groups, keep, scale, correction, scoring, group_score, renormalize, bias};
+    ce_note("moe_router_kernel");
+    if (N <= 8) moe_router_launch<1>(r, a, stream);
+    else if (N <= 16) moe_router_launch<2>(r, a, stream);
+    else if (N <= 32) moe_router_launch<4>(r, a, stream);
+    else if (N <= 64) moe_router_launch<8>(r, a, stream);
+    else moe_router_launch<16>(r, a, stream);
+    return ce_check_launch("ce_moe_router");
 }
 
 // ---------------------------------------------------------------------------------------------
@@ -468,7 +570,7 @@ __global__ void moe_combine_kernel(const T* __restrict__ rows, int ld, const int
                                    int W, int accumulate) {
     ce_pdl_begin();
     const int t = blockIdx.x;
-    for (int j = threadIdx.x; j < W; j += blockDim.x) {
+    for (int j = blockIdx.y * blockDim.x + threadIdx.x; j < W; j += blockDim.x * gridDim.y) {
         float v = 0.f;
         for (int k = 0; k < top; ++k)
             v = fmaf(weights[(size_t)t * top + k], CeType<T>::load(rows + (size_t)pair_row[(size_t)t * top + k] * ld + j), v);
@@ -478,14 +580,43 @@ __global__ void moe_combine_kernel(const T* __restrict__ rows, int ld, const int
     }
 }
 
+// The same with four columns a thread (W and ld in multiples of 4, rows aligned): the same sums in the same order.
+template <typename T>
+__global__ void moe_combine_vec_kernel(const T* __restrict__ rows, int ld, const int* __restrict__ pair_row, const float* __restrict__ weights,
+                                       const T* __restrict__ shared, const float* __restrict__ sgate, float* __restrict__ y, int top,
+                                       int W, int accumulate) {
+    ce_pdl_begin();
+    const int t = blockIdx.x;
+    const int j = 4 * (blockIdx.y * blockDim.x + threadIdx.x);
+    if (j >= W) return;
+    float4 v = ce_sum_picks4(rows, ld, pair_row + (size_t)t * top, weights + (size_t)t * top, top, j);
+    if (shared) {
+        const float g = sgate ? sgate[t] : 1.0f;
+        const float4 s = ce_load4(shared + (size_t)t * W + j);
+        v.x = fmaf(g, s.x, v.x); v.y = fmaf(g, s.y, v.y); v.z = fmaf(g, s.z, v.z); v.w = fmaf(g, s.w, v.w);
+    }
+    float4* o = reinterpret_cast<float4*>(y + (size_t)t * W + j);
+    if (accumulate) { const float4 p = *o; v.x = p.x + v.x; v.y = p.y + v.y; v.z = p.z + v.z; v.w = p.w + v.w; }
+    *o = v;
+}
+
 extern "C" int ce_moe_combine(const void* rows, int dtype, int ld, const int* pair_row, const float* weights, const void* shared,
                               const float* sgate, float* y, int T, int top, int W, int accumulate, cudaStream_t stream) {
     if (T == 0 || W == 0) return CE_OK;
     if (!rows || !pair_row || !weights || !y) return ce_fail(CE_ERR_ARG, "ce_moe_combine: null pointer");
-    int threads = W >= 1024 ? 256 : 128;
+    const size_t el = dtype == CE_F32 ? 4 : 2;
+    const int threads = 128;
     ce_note("moe_combine_kernel");
-    if (dtype == CE_F32) ce_launch(moe_combine_kernel<float>, T, threads, 0, stream, (const float*)rows, ld, pair_row, weights, (const float*)shared, sgate, y, top, W, accumulate);
-    else if (dtype == CE_BF16) ce_launch(moe_combine_kernel<__nv_bfloat16>, T, threads, 0, stream, (const __nv_bfloat16*)rows, ld, pair_row, weights, (const __nv_bfloat16*)shared, sgate, y, top, W, accumulate);
+    if (W % 4 == 0 && ld % 4 == 0 && ((uintptr_t)y & 15) == 0 && (((uintptr_t)rows | (uintptr_t)shared) & (4 * el - 1)) == 0) {
+        dim3 grid(T, (W / 4 + threads - 1) / threads);
+        if (dtype == CE_F32) ce_launch(moe_combine_vec_kernel<float>, grid, threads, 0, stream, (const float*)rows, ld, pair_row, weights, (const float*)shared, sgate, y, top, W, accumulate);
+        else if (dtype == CE_BF16) ce_launch(moe_combine_vec_kernel<__nv_bfloat16>, grid, threads, 0, stream, (const __nv_bfloat16*)rows, ld, pair_row, weights, (const __nv_bfloat16*)shared, sgate, y, top, W, accumulate);
+        else return ce_fail(CE_ERR_ARG, "ce_moe_combine: unknown dtype %d", dtype);
+        return ce_check_launch("ce_moe_combine");
+    }
+    dim3 grid(T, (W + 4 * threads - 1) / (4 * threads));
+    if (dtype == CE_F32) ce_launch(moe_combine_kernel<float>, grid, threads, 0, stream, (const float*)rows, ld, pair_row, weights, (const float*)shared, sgate, y, top, W, accumulate);
+    else if (dtype == CE_BF16) ce_launch(moe_combine_kernel<__nv_bfloat16>, grid, threads, 0, stream, (const __nv_bfloat16*)rows, ld, pair_row, weights, (const __nv_bfloat16*)shared, sgate, y, top, W, accumulate);
     else return ce_fail(CE_ERR_ARG, "ce_moe_combine: unknown dtype %d", dtype);
     return ce_check_launch("ce_moe_combine");
 }

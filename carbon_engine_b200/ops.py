@@ -386,6 +386,24 @@ def residual_norm(x: torch.Tensor, alpha: float, outputs: Sequence[torch.Tensor]
                                    _ptr(rounded), T, W, float(alpha), float(factor), float(eps), float(member_eps), _stream()))
 
 
+def residual_norm_picks(x: torch.Tensor, alpha: float, rows: torch.Tensor, pair_row: torch.Tensor, weights: torch.Tensor,
+                        weight: torch.Tensor, eps: float, rounded: Optional[torch.Tensor] = None) -> None:
+    """:func:`residual_norm` with the weighted sum of a token's experts as the sublayer's output (:func:`moe_combine` without a
+    shared expert, in the same order): x[t] = rmsnorm(alpha x[t] + sum_k weights[t, k] rows[pair_row[t * top + k]]) * weight."""
+    _need(x, "x", torch.float32); _need(weight, "weight", torch.float32); _need(weights, "weights", torch.float32)
+    _need(pair_row, "pair_row", torch.int32)
+    T, W = x.shape
+    top = weights.shape[1]
+    if weights.shape[0] != T or pair_row.numel() < T * top or rows.shape[1] != W or rows.stride(-1) != 1 or weight.numel() != W:
+        raise KernelError("residual_norm_picks: sizes do not fit")
+    if rounded is not None:
+        _need(rounded, "rounded", torch.bfloat16)
+        if rounded.shape != x.shape:
+            raise KernelError("residual_norm_picks: the rounded copy must have the shape of x")
+    _ok(kernels().ce_residual_norm_picks(_ptr(rows), dtype_code(rows.dtype), rows.stride(0), _ptr(pair_row), _ptr(weights), top, _ptr(weight),
+                                         _ptr(x), _ptr(rounded), T, W, float(alpha), float(eps), _stream()))
+
+
 def tanh_cap(x: torch.Tensor, cap: float) -> None:
     """x <- cap * tanh(x / cap) in place (float32)."""
     _need(x, "x", torch.float32)
@@ -898,6 +916,35 @@ def moe_route(z: torch.Tensor, experts: int, top: int, groups: int, keep: int, s
     _ok(kernels().ce_moe_route(_ptr(z), _ptr(ids), _ptr(weights), _ptr(sgate), T, z.stride(0), int(experts), int(top), int(groups),
                                int(keep), float(scale), _ptr(correction), MOE_SCORES[scoring], MOE_GROUP_SCORES[group_score],
                                1 if renormalize else 0, _ptr(bias), _stream()))
+
+
+def moe_router_supported(h: torch.Tensor, w: torch.Tensor, rows: int) -> bool:
+    """Whether :func:`moe_router` takes the router ``w`` [>= rows, K] (bfloat16, up to 128 rows that fit a block's reading)."""
+    return h.dtype == torch.bfloat16 and w.dtype == h.dtype and h.stride(-1) == 1 and w.is_contiguous() and \
+        not (h.data_ptr() | w.data_ptr()) & 15 and bool(kernels().ce_moe_router_supported(int(rows), w.shape[1], h.stride(0)))
+
+
+def moe_router(h: torch.Tensor, w: torch.Tensor, experts: int, top: int, groups: int, keep: int, scale: float, ids: torch.Tensor,
+               weights: torch.Tensor, sgate: Optional[torch.Tensor] = None, scoring: str = "softmax",
+               correction: Optional[torch.Tensor] = None, group_score: str = "max", renormalize: bool = True,
+               bias: Optional[torch.Tensor] = None) -> None:
+    """:func:`moe_route` with the router's product in the same kernel: z = h @ w[:experts (+1)].T in float32."""
+    _need(ids, "ids", torch.int32); _need(weights, "weights", torch.float32)
+    T, rows = h.shape[0], experts + (1 if sgate is not None else 0)
+    if ids.shape != (T, top) or weights.shape != (T, top) or (sgate is not None and (sgate.dtype != torch.float32 or sgate.numel() != T)) \
+            or w.shape[0] < rows or w.shape[1] != h.shape[1] or not moe_router_supported(h, w, rows):
+        raise KernelError("moe_router: sizes do not fit")
+    for name, t in (("correction", correction), ("bias", bias)):
+        if t is not None:
+            _need(t, name, torch.float32)
+            if t.numel() < experts:
+                raise KernelError(f"moe_router: one {name} per expert")
+    prof = profiling()
+    if prof is not None:
+        prof.note_work((T + rows) * h.shape[1] * 2, 2 * T * rows * h.shape[1])
+    _ok(kernels().ce_moe_router(_ptr(h), h.stride(0), _ptr(w), rows, w.shape[1], _ptr(ids), _ptr(weights), _ptr(sgate), T, int(experts),
+                                int(top), int(groups), int(keep), float(scale), _ptr(correction), MOE_SCORES[scoring],
+                                MOE_GROUP_SCORES[group_score], 1 if renormalize else 0, _ptr(bias), _stream()))
 
 
 def moe_max_tiles(n_pairs: int, experts: int, tile: int) -> int:

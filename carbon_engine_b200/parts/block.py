@@ -11,6 +11,7 @@ import torch
 from .. import ops
 from .base import RESIDUAL_ROUNDED, Block, BundleCacheSpec, FeedForward, Mixer, Norm, Part
 from .combine import NormedMixers
+from .moe import RoutedExperts
 from .norm import RMSNorm
 
 
@@ -129,7 +130,8 @@ class PostNormBlock(Block):
     """The norm is taken of the weighted residual plus the sublayer's output, and IS the new residual: x <- mixer_norm(alpha x +
     mixer(x)); x <- ffn_norm(alpha x + ffn(x)).  The sublayers read the residual itself (rounded to the compute dtype) and STORE
     their result in a float32 buffer (``can_store``); one kernel weighs, adds and norms, and leaves the new residual rounded for
-    the next sublayer.  The outputs of mixers side by side (:class:`NormedMixers`) are normed and added in that kernel too.
+    the next sublayer.  The outputs of mixers side by side (:class:`NormedMixers`) are normed and added in that kernel too, and so
+    are a token's experts (:class:`RoutedExperts` without a shared expert) summed.
     The norms are RMS norms.  ``ffn`` None: the layer has only the mixer."""
 
     def __init__(self, width: int, alpha: float, mixer: Mixer, mixer_norm: RMSNorm, ffn: Optional[FeedForward] = None,
@@ -152,9 +154,12 @@ class PostNormBlock(Block):
         ffn = self.ffn.step_bytes(tokens, element_size) if self.ffn is not None else 0
         return tokens * self.width * (2 * element_size + 4) + max(self.mixer.step_bytes(tokens, element_size), ffn)
 
-    def _norm(self, ctx, x: torch.Tensor, outputs: List[torch.Tensor], norm: RMSNorm, **more) -> None:
+    def _norm(self, ctx, x: torch.Tensor, outputs, norm: RMSNorm, picks=None, **more) -> None:
         rounded = ctx.buffer(tuple(x.shape)) if ctx.dtype == torch.bfloat16 else None
-        ops.residual_norm(x, self.alpha, outputs, norm.weight, norm.eps, rounded=rounded, **more)
+        if picks is not None:
+            ops.residual_norm_picks(x, self.alpha, *picks, norm.weight, norm.eps, rounded)
+        else:
+            ops.residual_norm(x, self.alpha, outputs, norm.weight, norm.eps, rounded=rounded, **more)
         if rounded is not None:
             ctx.shared[RESIDUAL_ROUNDED] = (rounded, x.data_ptr())
 
@@ -170,8 +175,13 @@ class PostNormBlock(Block):
             self._norm(ctx, x, [y], self.mixer_norm, bias=owed)
         if self.ffn is None:
             return
+        h = read_residual(ctx, x)
+        if isinstance(self.ffn, RoutedExperts) and self.ffn.shared_ff == 0:
+            rows, pair_row, weights, _ = self.ffn.picks(ctx, h)
+            self._norm(ctx, x, None, self.ffn_norm, picks=(rows, pair_row, weights))
+            return
         y = ctx.buffer(tuple(x.shape), torch.float32)
-        owed = self.ffn.forward(ctx, read_residual(ctx, x), y, accumulate=False)
+        owed = self.ffn.forward(ctx, h, y, accumulate=False)
         self._norm(ctx, x, [y], self.ffn_norm, bias=owed)
 
 

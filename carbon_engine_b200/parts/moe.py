@@ -18,7 +18,8 @@ the host, so a step of a given size launches the same grids whatever the router 
 In bfloat16, with sizes the kernel takes, the products run on the tcgen05 grouped kernel of ``gemm_tc.cu`` (tiles of 16 rows
 in steps of single tokens, of 64 or 128 rows in steps of many); it loads its rows by TMA, so the tokens' rows are first
 copied into the layout's order.  Other sizes and float32 take the kernels of ``moe.cu``, which read the tokens' rows where
-they lie.  The shared expert is two ordinary products.
+they lie.  The shared expert is two ordinary products.  In bfloat16 the router's product is part of the routing kernel (routers of
+up to 128 rows); a block that norms the sum of the residual and the experts' outputs takes the rows and sums them itself (``picks``).
 Where there is a gate on the shared expert, the router's product also yields the shared expert's gate logit (its row is appended to the router's).
 """
 from __future__ import annotations
@@ -130,15 +131,21 @@ class RoutedExperts(FeedForward):
             return
         ops.moe_matmul(x, w, out, tile, activation, row_token, tile_expert, n_tiles, self.limit, self.alpha)
 
-    def forward(self, ctx, h: torch.Tensor, x: torch.Tensor, accumulate: bool = True) -> None:
+    def picks(self, ctx, h: torch.Tensor):
+        """Route the tokens and run their experts: (rows [*, hidden] over the layout by expert, the row of every (token, pick)
+        pair, the picks' weights [T, top], the shared expert's gate [T] or None)."""
         T, E, top = h.shape[0], self.experts, self.top
         i32 = lambda n: ctx.buffer((n,), torch.int32)
-        z = ctx.buffer((T, self.router.padded_out), torch.float32)
-        self.router.forward(h, z, STORE_F32, add_bias=False)            # (the routing kernel adds the bias)
         ids, weights = ctx.buffer((T, top), torch.int32), ctx.buffer((T, top), torch.float32)
         sgate = ctx.buffer((T,), torch.float32) if self.shared_gate else None
-        ops.moe_route(z, E, top, self.groups, self.keep_groups, self.scale, ids, weights, sgate, self.scoring, self.correction_w,
-                      self.group_score, self.renormalize, self.router.bias)
+        options = (E, top, self.groups, self.keep_groups, self.scale, ids, weights, sgate, self.scoring, self.correction_w,
+                   self.group_score, self.renormalize, self.router.bias)
+        if ops.moe_router_supported(h, self.router.weight, E + (1 if self.shared_gate else 0)):
+            ops.moe_router(h, self.router.weight, *options)
+        else:
+            z = ctx.buffer((T, self.router.padded_out), torch.float32)
+            self.router.forward(h, z, STORE_F32, add_bias=False)            # (the routing kernel adds the bias)
+            ops.moe_route(z, *options)
         tile = self.tile_for(T, h.dtype)
         fast = self._fast(tile, h.dtype)
         tiles = ops.moe_max_tiles(T * top, E, tile)
@@ -153,6 +160,11 @@ class RoutedExperts(FeedForward):
             self._product(h, self.up, act, tile, self.activation, False, row_token, tile_expert, n_tiles)
         rows = ctx.buffer((tiles * tile, self.hidden))
         self._product(act, self.down, rows, tile, "none", fast, None, tile_expert, n_tiles)
+        return rows, pair_row, weights, sgate
+
+    def forward(self, ctx, h: torch.Tensor, x: torch.Tensor, accumulate: bool = True) -> None:
+        T = h.shape[0]
+        rows, pair_row, weights, sgate = self.picks(ctx, h)
         shared = None
         if self.shared_ff > 0:
             sact = ctx.buffer((T, self.shared_ff))

@@ -155,7 +155,10 @@ class SinkAttention(Mixer):
                 for b in range(ctx.B):
                     n, before = ctx.h_q_start[b + 1] - ctx.h_q_start[b], ctx.h_ctx_before[b]
                     keys += before + n if self.window <= 0 else min(before + n, self.window - 1 + n)
-                    pairs += sum(min(p + 1, self.window) if self.window > 0 else p + 1 for p in range(before, before + n))
+                    pairs += n * before + n * (n + 1) // 2
+                    if self.window > 0:                       # less the keys that have left the window
+                        out0, out1 = max(0, before - self.window), max(0, before + n - self.window)
+                        pairs -= out1 * (out1 + 1) // 2 - out0 * (out0 + 1) // 2
                 prof.note_work((2 * keys * G * d + 2 * ctx.T * H * d) * 2, 4 * pairs * H * d)
             if ops_tensor.attention_bf16(ctx, plan, q, out, cache, table, H, G, d, self.window, self.scale, sinks=self.sinks,
                                          out_scale=self.out_scale, slopes=self.slopes):

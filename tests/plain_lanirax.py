@@ -159,7 +159,8 @@ def tied_window_attention(w: Weights, p: str, m: dict, h: torch.Tensor, eps: flo
     T, H, G, d = h.shape[0], int(m["heads"]), int(m["kv_heads"]), int(m["dim"])
     q = (h @ w[f"{p}.q"].T).reshape(T, H, d)
     v = (h @ w[f"{p}.k"].T).reshape(T, G, d)
-    q, k = unit_rms(rotate_neighbours(q, m["rot"]), eps), unit_rms(rotate_neighbours(v, m["rot"]), eps)
+    turn = lambda x: rotate_neighbours(x, m["rot"]) if m.get("rot") else x
+    q, k = unit_rms(turn(q), eps), unit_rms(turn(v), eps)
     window = int(m["mask"]["size"]) if m.get("mask") else 0
     out = softmax_attention(q, k, v, float(m["scale"]), window=window, sink=w[f"{p}.sink"])
     return out.reshape(T, H * d) @ w[f"{p}.o"].T
@@ -220,10 +221,14 @@ def expert(w: Weights, p: str, h: torch.Tensor) -> torch.Tensor:
     return (silu(h @ w[f"{p}.gate"].T) * (h @ w[f"{p}.up"].T)) @ w[f"{p}.down"].T
 
 
-def mixture(w: Weights, p: str, mlp: dict, h: torch.Tensor) -> torch.Tensor:
+def mixture(w: Weights, p: str, mlp: dict, h: torch.Tensor, margins: Optional[list] = None) -> torch.Tensor:
+    """``margins`` receives, per token, the gap between the last logit chosen and the first one not."""
     top = int(mlp["router"]["top"])
     z = h @ w[f"{p}.router"].T + w[f"{p}.router.b"]
     out = torch.zeros_like(h)
+    if margins is not None:
+        ranked = torch.sort(z, dim=-1, descending=True).values
+        margins.append((ranked[:, top - 1] - ranked[:, top]).tolist() if top < z.shape[1] else [float("inf")] * h.shape[0])
     for t in range(h.shape[0]):
         chosen = torch.sort(z[t], descending=True, stable=True).indices[:top]
         weight = torch.exp(z[t][chosen] - z[t][chosen].max())
@@ -245,9 +250,11 @@ def owner(layers: list, i: int) -> int:
     return i
 
 
-def forward(cfg: dict, weights: Weights, tokens: List[int], layers_out: Optional[list] = None, rounding=None) -> torch.Tensor:
-    """Logits [T, vocab] of one sequence; ``layers_out`` receives the residual after every layer.  ``rounding``: a function
-    applied to what every sublayer reads (to see how far rounding alone moves the result)."""
+def forward(cfg: dict, weights: Weights, tokens: List[int], layers_out: Optional[list] = None, rounding=None,
+            margins: Optional[list] = None) -> torch.Tensor:
+    """Logits [T, vocab] of one sequence; ``layers_out`` receives the residual after every layer, ``margins`` the routers' (see
+    :func:`mixture`).  ``rounding``: a function applied to what every sublayer reads (to see how far rounding alone moves the
+    result)."""
     w = {k: v.to(F) if v.is_floating_point() else v for k, v in weights.items()}
     read = rounding if rounding is not None else lambda x: x
     eps, alpha = float(cfg["norm"]["eps"]), float(cfg["postln_alpha"])
@@ -256,7 +263,7 @@ def forward(cfg: dict, weights: Weights, tokens: List[int], layers_out: Optional
         p = f"l{owner(cfg['layers'], i)}"
         x = rms_norm(alpha * x + MIXERS[layer["type"]](w, f"{p}.mix", layer["mixer"], read(x), eps), w[f"{p}.norm1"], eps)
         if layer.get("mlp") is not None:
-            x = rms_norm(alpha * x + mixture(w, f"{p}.mlp", layer["mlp"], read(x)), w[f"{p}.norm2"], eps)
+            x = rms_norm(alpha * x + mixture(w, f"{p}.mlp", layer["mlp"], read(x), margins), w[f"{p}.norm2"], eps)
         if layers_out is not None:
             layers_out.append(x.clone())
     return read(rms_norm(x, w["final.norm"], eps)) @ w["head"].T
