@@ -194,22 +194,27 @@ __global__ void gated_delta_prepare_kernel(GatedDeltaArgs a) {
     }
 }
 
-// The same for operands 2 (nothing couples the channels): a thread takes one channel of GD_CONV_TOKENS tokens, so that a token's input
-// is read once and not K times, and the channel's taps once for all of them.
+// The same for operands 2 (nothing couples the channels) and, with key heads of 32, 64, 128 or 256 (UNIT), for operands 0: a thread
+// takes one channel of GD_CONV_TOKENS tokens, so that a token's input is read once and not K times, and the channel's taps once for
+// all of them.  UNIT: a key head's channels lie in one block of 256; its sum of squares is a butterfly over each warp's 32 channels
+// and the warps' sums in order, whatever the tile.
 #define GD_CONV_TOKENS 8
-template <int K>
+template <int K, bool UNIT>
 __global__ void __launch_bounds__(256) gated_delta_conv_kernel(GatedDeltaArgs a, int T, int tile) {
     ce_pdl_begin();
+    __shared__ float squares[UNIT ? GD_CONV_TOKENS : 1][8];
     const int C = 2 * a.G * a.d + a.H * a.dv, H = a.H;
     const int t0 = blockIdx.x * tile, nt = min(tile, T - t0), c = blockIdx.y * 256 + threadIdx.x;
     const int b0 = a.seq_of_token[t0], rel0 = t0 - a.q_start[b0];
+    float y[GD_CONV_TOKENS];
+#pragma unroll
+    for (int i = 0; i < GD_CONV_TOKENS; ++i) y[i] = 0.f;
     if (c < C) {
         float w[K];
 #pragma unroll
         for (int j = 0; j < K; ++j) w[j] = a.taps[(size_t)c * K + j];
         const float bias = a.conv_bias ? a.conv_bias[c] : 0.f;
         const float* in = a.proj + a.off_conv + c;
-        auto out = [&](int t, float y) { a.prep[(size_t)t * a.P + c] = y / (1.0f + expf(-y)); };
         if (nt == GD_CONV_TOKENS && a.seq_of_token[t0 + nt - 1] == b0) {
             const float* kept = a.kept + (size_t)a.seq_slot[b0] * (K - 1) * C + c;
             float x[GD_CONV_TOKENS + K - 1];          // the tile's inputs, after the K - 1 before it
@@ -220,35 +225,75 @@ __global__ void __launch_bounds__(256) gated_delta_conv_kernel(GatedDeltaArgs a,
             for (int i = 0; i < GD_CONV_TOKENS; ++i) x[K - 1 + i] = in[(size_t)(t0 + i) * a.ld];
 #pragma unroll
             for (int i = 0; i < GD_CONV_TOKENS; ++i) {
-                float y = bias;
+                y[i] = bias;
 #pragma unroll
-                for (int j = 0; j < K; ++j) y = fmaf(w[j], x[i + j], y);
-                out(t0 + i, y);
+                for (int j = 0; j < K; ++j) y[i] = fmaf(w[j], x[i + j], y[i]);
             }
         } else {
-            for (int t = t0; t < t0 + nt; ++t) {
-                const int b = a.seq_of_token[t], rel = t - a.q_start[b];
+#pragma unroll
+            for (int i = 0; i < GD_CONV_TOKENS; ++i) {
+                if (i >= nt) break;
+                const int t = t0 + i, b = a.seq_of_token[t], rel = t - a.q_start[b];
                 float* kept = a.kept + (size_t)a.seq_slot[b] * (K - 1) * C + c;
-                float y = bias, x[K];
+                float x[K];
+                y[i] = bias;
 #pragma unroll
                 for (int j = 0; j < K; ++j) {
                     const int back = K - 1 - j;
                     x[j] = back <= rel ? in[(size_t)(t - back) * a.ld] : kept[(size_t)(K - 1 + rel - back) * C];
                 }
 #pragma unroll
-                for (int j = 0; j < K; ++j) y = fmaf(w[j], x[j], y);
+                for (int j = 0; j < K; ++j) y[i] = fmaf(w[j], x[j], y[i]);
                 if (a.single) {                       // the kept rows move up by one
 #pragma unroll
                     for (int j = 1; j < K; ++j) kept[(size_t)(j - 1) * C] = x[j];
                 }
-                out(t, y);
             }
+        }
+#pragma unroll
+        for (int i = 0; i < GD_CONV_TOKENS; ++i) y[i] = y[i] / (1.0f + expf(-y[i]));
+    }
+    if (UNIT) {
+        const int warp = threadIdx.x >> 5;
+        const bool key = c < 2 * a.G * a.d;          // (the same for a whole warp: heads are made of whole warps)
+        if (key) {
+#pragma unroll
+            for (int i = 0; i < GD_CONV_TOKENS; ++i) {
+                if (i >= nt) break;
+                float ss = __fmul_rn(y[i], y[i]);
+                for (int o = 16; o > 0; o >>= 1) ss = __fadd_rn(ss, __shfl_xor_sync(0xffffffffu, ss, o));
+                if ((threadIdx.x & 31) == 0) squares[i][warp] = ss;
+            }
+        }
+        __syncthreads();
+        if (key) {
+            const int per = a.d >> 5, first = warp / per * per;
+            const float scale = c < a.G * a.d ? rsqrtf((float)a.d) : 1.0f;
+#pragma unroll
+            for (int i = 0; i < GD_CONV_TOKENS; ++i) {
+                if (i >= nt) break;
+                float ss = 0.f;
+                for (int n = 0; n < per; ++n) ss = __fadd_rn(ss, squares[i][first + n]);
+                y[i] *= 1.0f / sqrtf(ss + 1e-6f) * scale;
+            }
+        }
+    }
+    if (c < C) {
+#pragma unroll
+        for (int i = 0; i < GD_CONV_TOKENS; ++i) if (i < nt) a.prep[(size_t)(t0 + i) * a.P + c] = y[i];
+    }
+    if (a.decay_mode == 0) {                         // a decay per key channel: dealt to all blocks of the tile
+        const int n = H * a.d;
+        for (int e = blockIdx.y * 256 + threadIdx.x; e < nt * n; e += 256 * gridDim.y) {
+            const int t = t0 + e / n, i = e % n;
+            a.prep[(size_t)t * a.P + C + i] = expf(-expf(a.a_log[i / a.d]) * gd_softplus(a.dec[(size_t)t * a.ld_dec + i] + a.dt_bias[i]));
         }
     }
     if (blockIdx.y == gridDim.y - 1) {
         for (int e = threadIdx.x; e < nt * H; e += 256) {
             const int t = t0 + e / H, h = e % H;
             float* gates = a.prep + (size_t)t * a.P + C;
+            if (a.decay_mode == 0) { gates[H * a.d + h] = gd_sigmoid(a.proj[(size_t)t * a.ld + a.off_b + h]); continue; }
             float step = a.decay_mode == 1 ? gd_softplus(a.dec[(size_t)t * a.ld_dec + h] + a.dt_bias[h]) : 0.f;
             gates[h] = a.decay_mode == 1 ? expf(-expf(a.a_log[h]) * step) : a.a_log[h];
             gates[H + h] = a.write_mode == 1 ? step : gd_sigmoid(a.proj[(size_t)t * a.ld + a.off_b + h]);
@@ -851,17 +896,23 @@ extern "C" int ce_gated_delta(const float* proj, const float* dec, const float* 
                      write_mode, ones, norm_all, parts, T == B ? 1 : 0};
     int heads = 2 * G + H;
     int threads = heads >= 8 ? 256 : 32 * heads;
-    if (stage == 1 && operands == 2 && K <= 5 && decay_mode != 0) {
+    const bool unit = operands == 0 && (d == 32 || d == 64 || d == 128 || d == 256);
+    if (stage == 1 && K <= 5 && (unit || (operands == 2 && decay_mode != 0))) {
         const int C = 2 * G * d + H * dv, tile = T >= 4 * GD_CONV_TOKENS ? GD_CONV_TOKENS : 1;
         dim3 grid((T + tile - 1) / tile, (C + 255) / 256);
         ce_note("gated_delta_conv_kernel");
+#define GD_CONV_CASE(KK)                                                                                       \
+        if (unit) ce_launch(gated_delta_conv_kernel<KK, true>, grid, 256, 0, stream, a, T, tile);              \
+        else ce_launch(gated_delta_conv_kernel<KK, false>, grid, 256, 0, stream, a, T, tile);                  \
+        break;
         switch (K) {
-            case 1: ce_launch(gated_delta_conv_kernel<1>, grid, 256, 0, stream, a, T, tile); break;
-            case 2: ce_launch(gated_delta_conv_kernel<2>, grid, 256, 0, stream, a, T, tile); break;
-            case 3: ce_launch(gated_delta_conv_kernel<3>, grid, 256, 0, stream, a, T, tile); break;
-            case 4: ce_launch(gated_delta_conv_kernel<4>, grid, 256, 0, stream, a, T, tile); break;
-            default: ce_launch(gated_delta_conv_kernel<5>, grid, 256, 0, stream, a, T, tile); break;
+            case 1: GD_CONV_CASE(1)
+            case 2: GD_CONV_CASE(2)
+            case 3: GD_CONV_CASE(3)
+            case 4: GD_CONV_CASE(4)
+            default: GD_CONV_CASE(5)
         }
+#undef GD_CONV_CASE
     } else if (stage == 1) {
         ce_note("gated_delta_prepare_kernel");
         int per_block = threads / 32, want = (heads + per_block - 1) / per_block, room = 4 * 148 / T;

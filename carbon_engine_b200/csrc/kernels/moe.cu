@@ -130,14 +130,26 @@ __global__ void __launch_bounds__(128) moe_route_kernel(MoeRouteArgs a) {
 // 32, each a product of the 16 tokens with all experts (mma.sync m16n8k16), and the partial logits are added in the warps' order
 // (float32): a token's logits depend on neither its place nor on the other tokens.  Within a run the elements of K are dealt to the
 // products so that every lane reads 16 consecutive bytes of a row (the same for both operands).  Then a warp routes a token.
+// In a step of few tokens one block would read the whole router by itself: with CLUSTER > 1 that many blocks share K for the same 16
+// tokens, and the first adds their logits up through distributed shared memory and routes.
 #define MR_WARPS 16
+__device__ __forceinline__ void moe_cluster_sync() {
+    asm volatile("barrier.cluster.arrive.release.aligned;\nbarrier.cluster.wait.acquire.aligned;" ::: "memory");
+}
+__device__ __forceinline__ float moe_ld_cluster(const float* mine, int rank) {
+    unsigned at = (unsigned)__cvta_generic_to_shared(mine), there;
+    float v;
+    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(there) : "r"(at), "r"(rank));
+    asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(there) : "memory");
+    return v;
+}
 struct MoeRouterArgs {
     const __nv_bfloat16* h;      // [T, ldh]
     const __nv_bfloat16* W;      // [N, K]: the experts' rows, then the shared expert's gate row where there is one
     int ldh, N, K;
 };
 
-template <int NT>
+template <int NT, int CLUSTER>
 __global__ void __launch_bounds__(32 * MR_WARPS) moe_router_kernel(MoeRouterArgs r, MoeRouteArgs a) {
     ce_pdl_begin();
     extern __shared__ float moe_router_smem[];
@@ -145,14 +157,14 @@ __global__ void __launch_bounds__(32 * MR_WARPS) moe_router_kernel(MoeRouterArgs
     float* part = moe_router_smem;                           // [warps][16][NE]; the routing's work space afterwards
     float* z = part + MR_WARPS * 16 * NE;                    // [16][NE]
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, grp = lane >> 2, quad = lane & 3;
-    const int t0 = blockIdx.x * 16;
+    const int t0 = blockIdx.x / CLUSTER * 16, rank = blockIdx.x % CLUSTER;
     const __nv_bfloat16* ha = r.h + (size_t)min(t0 + grp, a.T - 1) * r.ldh + quad * 8;
     const __nv_bfloat16* hb = r.h + (size_t)min(t0 + grp + 8, a.T - 1) * r.ldh + quad * 8;
     float acc[NT][4];
 #pragma unroll
     for (int n = 0; n < NT; ++n) acc[n][0] = acc[n][1] = acc[n][2] = acc[n][3] = 0.f;
-#pragma unroll 2
-    for (int k0 = warp * 32; k0 < r.K; k0 += MR_WARPS * 32) {
+#pragma unroll (NT >= 16 ? 1 : 4)
+    for (int k0 = (rank * MR_WARPS + warp) * 32; k0 < r.K; k0 += CLUSTER * MR_WARPS * 32) {
         const uint4 x = *reinterpret_cast<const uint4*>(ha + k0), y = *reinterpret_cast<const uint4*>(hb + k0);
 #pragma unroll
         for (int n = 0; n < NT; ++n) {
@@ -175,6 +187,20 @@ __global__ void __launch_bounds__(32 * MR_WARPS) moe_router_kernel(MoeRouterArgs
 #pragma unroll
         for (int w = 0; w < MR_WARPS; ++w) v += part[w * 16 * NE + e];
         z[e] = v;
+    }
+    if (CLUSTER > 1) {
+        moe_cluster_sync();                                  // every block's logits are there
+        float* total = part;                                 // (its partial logits are used up)
+        if (rank == 0)
+            for (int e = threadIdx.x; e < 16 * NE; e += blockDim.x) {
+                float v = z[e];
+#pragma unroll
+                for (int w = 1; w < CLUSTER; ++w) v += moe_ld_cluster(z + e, w);
+                total[e] = v;
+            }
+        moe_cluster_sync();                                  // no block's shared memory goes away while it may still be read
+        if (rank != 0) return;
+        for (int e = threadIdx.x; e < 16 * NE; e += blockDim.x) z[e] = total[e];
     }
     __syncthreads();
     if (t0 + warp >= a.T) return;
@@ -216,10 +242,31 @@ extern "C" int ce_moe_router_supported(int N, int K, int ldh) {
 }
 
 template <int NT>
-static void moe_router_launch(const MoeRouterArgs& r, const MoeRouteArgs& a, cudaStream_t stream) {
+static int moe_router_launch(const MoeRouterArgs& r, const MoeRouteArgs& a, cudaStream_t stream) {
     size_t smem = (size_t)(MR_WARPS + 1) * 16 * NT * 8 * sizeof(float);
-    if (smem > 40 * 1024) cudaFuncSetAttribute(moe_router_kernel<NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    ce_launch(moe_router_kernel<NT>, (a.T + 15) / 16, 32 * MR_WARPS, smem, stream, r, a);
+    const int blocks = (a.T + 15) / 16;
+    if (blocks > 8 || r.K < 4 * MR_WARPS * 32) {
+        if (smem > 40 * 1024) cudaFuncSetAttribute(moe_router_kernel<NT, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        ce_launch(moe_router_kernel<NT, 1>, blocks, 32 * MR_WARPS, smem, stream, r, a);
+        return ce_check_launch("ce_moe_router");
+    }
+    constexpr int CLUSTER = 8;
+    if (smem > 40 * 1024) cudaFuncSetAttribute(moe_router_kernel<NT, CLUSTER>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = dim3(blocks * CLUSTER);
+    cfg.blockDim = dim3(32 * MR_WARPS);
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = stream;
+    cudaLaunchAttribute attr[2];
+    attr[0].id = cudaLaunchAttributeClusterDimension;
+    attr[0].val.clusterDim.x = CLUSTER; attr[0].val.clusterDim.y = 1; attr[0].val.clusterDim.z = 1;
+    attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[1].val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs = attr;
+    cfg.numAttrs = ce_pdl_enabled() ? 2 : 1;
+    cudaError_t e = cudaLaunchKernelEx(&cfg, moe_router_kernel<NT, CLUSTER>, r, a);
+    if (e != cudaSuccess) return ce_fail(CE_ERR_CUDA, "ce_moe_router: %s", cudaGetErrorString(e));
+    return ce_check_launch("ce_moe_router");
 }
 
 // ce_moe_route with the router's product in the same kernel: h [T, ldh] bf16, W [>= N, K] bf16, N = E (+ 1 with sgate)
@@ -235,12 +282,11 @@ extern "C" int ce_moe_router(const void* h, int ldh, const void* W, int N, int K
     MoeRouterArgs r{(const __nv_bfloat16*)h, (const __nv_bfloat16*)W, ldh, N, K};
     MoeRouteArgs a{nullptr, ids, weights, sgate, T, N, E, top, groups, keep, scale, correction, scoring, group_score, renormalize, bias};
     ce_note("moe_router_kernel");
-    if (N <= 8) moe_router_launch<1>(r, a, stream);
-    else if (N <= 16) moe_router_launch<2>(r, a, stream);
-    else if (N <= 32) moe_router_launch<4>(r, a, stream);
-    else if (N <= 64) moe_router_launch<8>(r, a, stream);
-    else moe_router_launch<16>(r, a, stream);
-    return ce_check_launch("ce_moe_router");
+    if (N <= 8) return moe_router_launch<1>(r, a, stream);
+    if (N <= 16) return moe_router_launch<2>(r, a, stream);
+    if (N <= 32) return moe_router_launch<4>(r, a, stream);
+    if (N <= 64) return moe_router_launch<8>(r, a, stream);
+    return moe_router_launch<16>(r, a, stream);
 }
 
 // ---------------------------------------------------------------------------------------------

@@ -227,10 +227,10 @@ def test_attention_kernels_with_a_penalty_on_distance(H, G, d, dv, window, cap, 
 
 
 @pytest.mark.parametrize("E, top, K, gate", [(5, 2, 64, False), (8, 8, 96, True), (16, 4, 352, False), (33, 3, 512, True), (64, 6, 128, False),
-                                             (100, 33, 64, False), (127, 5, 2048, True)])
+                                             (100, 33, 64, False), (127, 5, 2048, True), (32, 4, 4096, False), (7, 2, 2080, True)])
 def test_router_with_its_product_in_one_kernel(E, top, K, gate):
-    """Against the plain router and against the product and the routing in two kernels, for every scoring, over full and part-filled
-    blocks of tokens; a token's picks do not depend on the others."""
+    """Against the plain router for every scoring, over full and part-filled blocks of tokens (with K of 2,048 and more and few tokens:
+    several blocks that share K); a token's picks do not depend on the others."""
     from carbon_engine_b200 import ops
     g = torch.Generator().manual_seed(E + K)
     T, rows = 37, E + (1 if gate else 0)
@@ -265,6 +265,73 @@ def test_router_with_its_product_in_one_kernel(E, top, K, gate):
         for sel in (slice(0, 1), slice(17, 20), slice(36, 37)):
             a = run(sel, **kw)
             assert torch.equal(a[0], ids[sel]) and torch.equal(a[1], wts[sel])
+
+
+@pytest.mark.parametrize("channel_decay", [False, True])
+@pytest.mark.parametrize("H, G, d, dv, K", [(4, 2, 32, 24, 4), (2, 1, 64, 40, 5), (3, 3, 128, 16, 2), (2, 1, 256, 12, 3), (6, 2, 32, 7, 1)])
+def test_delta_rule_kernels_with_key_heads_of_whole_warps(H, G, d, dv, K, channel_decay):
+    """The convolution kernel that also makes unit keys: two sequences of 39 and 1 tokens in one step, then single tokens, then
+    another portion; a token has the same bits however it was cut, and the values are right (decays per head and per channel)."""
+    from carbon_engine_b200 import ops
+    g = torch.Generator().manual_seed(H * 100 + d)
+    n, C = 60, 2 * G * d + H * dv
+    n_dec = H * d if channel_decay else H
+    ld = (C + H + n_dec + H * dv + 3) // 4 * 4
+    taps = torch.randn(C, K, generator=g) * 0.5
+    a_log, dt_bias = torch.randn(H, generator=g) * 0.5, torch.randn(n_dec, generator=g) * 0.3
+    norm_w = 1 + 0.1 * torch.randn(dv, generator=g)
+    rows = [torch.randn(n, ld, generator=g) for _ in range(2)]
+    mode = ops.DECAY_PER_CHANNEL if channel_decay else ops.DECAY_PER_HEAD
+
+    def run(cuts):
+        """cuts: per step, the tokens each sequence brings (0: left out)."""
+        state = torch.zeros(3, H, d, dv, device="cuda")
+        kept = torch.zeros(3, max(K - 1, 1), C, device="cuda")
+        at, got = [0, 0], [[], []]
+        for cut in cuts:
+            who = [b for b in (0, 1) if cut[b]]
+            lengths = [cut[b] for b in who]
+            T = sum(lengths)
+            seq = torch.tensor([i for i, m in enumerate(lengths) for _ in range(m)], dtype=torch.int32, device="cuda")
+            starts = torch.tensor(np.concatenate([[0], np.cumsum(lengths)]), dtype=torch.int32, device="cuda")
+            slots = torch.tensor([(2, 0)[b] for b in who], dtype=torch.int32, device="cuda")
+            proj = torch.cat([rows[b][at[b]:at[b] + cut[b]] for b in who]).cuda()
+            prep = torch.empty(T, ops.gated_delta_prep_width(H, G, d, dv, mode), device="cuda")
+            raw, out = torch.empty(T, H * dv, device="cuda"), torch.empty(T, H * dv, device="cuda")
+            ops.gated_delta(proj, proj[:, C + H:C + H + n_dec], proj[:, C + H + n_dec:C + H + n_dec + H * dv], taps.cuda(), a_log.cuda(),
+                            dt_bias.cuda(), norm_w.cuda(), prep, raw, state, kept if K > 1 else None, out, seq, slots, starts, len(who), 0, C,
+                            H, G, d, dv, K, 1e-5, decay=mode, gate=ops.GATE_SILU)
+            i = 0
+            for b in who:
+                got[b].append(out[i:i + cut[b]].cpu())
+                at[b] += cut[b]
+                i += cut[b]
+        return [torch.cat(x) for x in got]
+    ops.reset_kernel_counts()
+    a = run([(39, 1), (1, 1), (1, 0), (19, 58)])
+    assert ops.kernel_counts()["gated_delta_conv_kernel"] == 4 and "gated_delta_prepare_kernel" not in ops.kernel_counts()
+    b = run([(60, 0), (0, 60)])
+    c = run([(2, 7), (5, 31), *[(1, 1)] * 22, (31, 0)])
+    for i in range(2):
+        assert torch.equal(a[i], b[i]) and torch.equal(a[i], c[i])
+        x = rows[i].double()
+        conv = plain.silu(plain.short_convolution(x[:, :C], taps.double()))
+        q = plain.unit_length(conv[:, :G * d].reshape(n, G, d)) * d ** -0.5
+        k = plain.unit_length(conv[:, G * d:2 * G * d].reshape(n, G, d))
+        v, beta = conv[:, 2 * G * d:].reshape(n, H, dv), torch.sigmoid(x[:, C:C + H])
+        dec = plain.softplus(x[:, C + H:C + H + n_dec] + dt_bias.double()).reshape(n, H, -1)
+        dec = torch.exp(-torch.exp(a_log.double())[None, :, None] * dec).expand(n, H, d)
+        want = torch.zeros(n, H, dv, dtype=torch.float64)
+        for h in range(H):
+            S = torch.zeros(d, dv, dtype=torch.float64)
+            for t in range(n):
+                S = dec[t, h][:, None] * S
+                kk = k[t, h // (H // G)]
+                S = S + torch.outer(kk, beta[t, h] * (v[t, h] - kk @ S))
+                want[t, h] = q[t, h // (H // G)] @ S
+        gate = plain.silu(x[:, C + H + n_dec:C + H + n_dec + H * dv])
+        want = plain.rms_norm(want, norm_w.double(), 1e-5).reshape(n, -1) * gate
+        assert rel_err(a[i].numpy(), want.numpy()) < 2e-5
 
 
 def test_routing_with_a_bias_far_from_zero_and_equal_logits():
