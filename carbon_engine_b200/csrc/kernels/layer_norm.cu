@@ -388,7 +388,10 @@ __global__ void residual_norm_kernel(ResidualNormArgs a) {
 
 template <int NM>
 static void residual_norm_launch(const ResidualNormArgs& a, int T, bool vec, cudaStream_t stream) {
-    int H4 = a.H / 4, vt = H4 >= 2048 ? 1024 : H4 >= 512 ? 512 : H4 >= 256 ? 256 : 128;
+    // Four float4s a thread: with fewer a block would take an SM's registers for threads that hold little of the row.  A bfloat16 step
+    // of few tokens takes more threads a row instead, for its latency (in float32 the order of a row's sums must not depend on T).
+    int H4 = a.H / 4, vt = H4 > 2048 ? 1024 : H4 > 1024 ? 512 : H4 > 512 ? 256 : 128;
+    if (a.xb && T <= 64) vt = H4 >= 2048 ? 1024 : H4 >= 512 ? 512 : H4 >= 256 ? 256 : 128;
     if (vec && H4 <= vt * LNV_MAX) ce_launch(residual_norm_kernel<NM, true>, T, vt, 0, stream, a);
     else ce_launch(residual_norm_kernel<NM, false>, T, a.H >= 4096 ? 512 : a.H >= 1024 ? 256 : 128, 0, stream, a);
 }

@@ -168,6 +168,111 @@ __global__ void norm_rope_kvwrite_kernel(NormRopeArgs a) {
     }
 }
 
+// The same for heads of 64, 128 and 256 whose elements come in aligned runs: a lane holds V = d / 32 neighbouring elements, so rows are
+// read and written in vectors; neighbouring pairs turn within a lane, the halves' pairs lie rd / 2 / V lanes apart.
+template <int V> __device__ __forceinline__ void nr_load(float (&v)[V], const float* p) {
+    if (V == 2) { float2 x = *reinterpret_cast<const float2*>(p); v[0] = x.x; v[1] = x.y; return; }
+#pragma unroll
+    for (int i = 0; i + 3 < V; i += 4) { float4 x = ce_load4(p + i); v[i] = x.x; v[i + 1] = x.y; v[i + 2] = x.z; v[i + 3] = x.w; }
+}
+template <int V> __device__ __forceinline__ void nr_store(float* p, const float (&v)[V]) {
+    if (V == 2) { *reinterpret_cast<float2*>(p) = make_float2(v[0], v[1]); return; }
+#pragma unroll
+    for (int i = 0; i + 3 < V; i += 4) *reinterpret_cast<float4*>(p + i) = make_float4(v[i], v[i + 1], v[i + 2], v[i + 3]);
+}
+template <int V> __device__ __forceinline__ void nr_store(__nv_bfloat16* p, const float (&v)[V]) {
+#pragma unroll
+    for (int i = 0; i < V; i += 2) *reinterpret_cast<__nv_bfloat162*>(p + i) = __floats2bfloat162_rn(v[i], v[i + 1]);
+}
+
+template <typename T, int V>
+__global__ void norm_rope_kvwrite_vec_kernel(NormRopeArgs a) {
+    ce_pdl_begin();
+    const int t = blockIdx.x, lane = threadIdx.x & 31, nwarp = (blockDim.x >> 5) * gridDim.y;
+    const int warp = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    constexpr int d = 32 * V;
+    const int half = a.rd / 2, p = a.positions[t], j0 = lane * V;
+    const float* row = a.proj + (size_t)t * a.ld;
+    const bool rotate = a.cos_table != nullptr && half > 0;
+    if ((rotate && (p < 0 || p >= a.max_pos)) || (a.pos_scale && (p < 0 || p >= a.max_pos_scale))) {
+        if (threadIdx.x == 0) atomicExch(a.status, 3);
+        return;
+    }
+    int page = -1, off = 0;
+    if (a.write_kv) {
+        int slot = a.seq_slot[a.seq_of_token[t]];
+        page = a.block_table[(size_t)slot * a.max_pages + p / a.page_size];
+        off = p % a.page_size;
+        if (page < 0 || page >= a.num_pages) {
+            if (threadIdx.x == 0) atomicExch(a.status, 2);
+            page = -1;
+        }
+    }
+    // this lane's cosines and sines: one per pair (neighbours), or one per element (halves)
+    float cs[V], sn[V];
+#pragma unroll
+    for (int i = 0; i < V; ++i) { cs[i] = 1.f; sn[i] = 0.f; }
+    if (rotate && j0 < a.rd) {
+        const float* ct = a.cos_table + (size_t)p * half;
+        const float* st = a.sin_table + (size_t)p * half;
+#pragma unroll
+        for (int i = 0; i < V; ++i) {
+            if (j0 + i >= a.rd) break;
+            int partner, angle;
+            bool first;
+            rope_pair(j0 + i, half, a.pairing, partner, angle, first);
+            cs[i] = ct[angle];
+            sn[i] = first ? -st[angle] : st[angle];
+        }
+    }
+    const int hop = a.pairing ? 0 : half / V;                // lanes between the two of a pair of the halves
+    const int other = j0 < half ? lane + hop : lane - hop;
+    const float ps = a.pos_scale ? a.pos_scale[p] : 1.0f;
+    for (int hh = warp; hh < a.nh + 2 * a.nkv; hh += nwarp) {
+        float v[V];
+        if (hh >= a.nh + a.nkv) {                            // a value head of the keys' size, as it is
+            if (page < 0) continue;
+            const int h = hh - a.nh - a.nkv;
+            nr_load<V>(v, row + a.off_v + h * d + j0);
+            nr_store<V>((T*)a.v_pool + (((size_t)page * a.nkv + h) * a.page_size + off) * d + j0, v);
+            continue;
+        }
+        const bool is_q = hh < a.nh;
+        const float* w = a.norm_mode ? (is_q ? a.wq : a.wk) : nullptr;
+        T* dst;
+        if (is_q) dst = (T*)a.q_out + ((size_t)t * a.nh + hh) * d;
+        else {
+            if (page < 0) continue;
+            dst = (T*)a.k_pool + (((size_t)page * a.nkv + (hh - a.nh)) * a.page_size + off) * d;
+        }
+        nr_load<V>(v, row + (is_q ? a.off_q + hh * d : a.off_k + (hh - a.nh) * d) + j0);
+        float wv[V];
+        if (w) nr_load<V>(wv, w + j0);
+        auto norm = [&]() {
+            float ss = 0.f;
+#pragma unroll
+            for (int i = 0; i < V; ++i) ss = fmaf(v[i], v[i], ss);
+            for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+            const float inv = 1.0f / sqrtf(ss / (float)d + a.eps);
+#pragma unroll
+            for (int i = 0; i < V; ++i) v[i] = w ? v[i] * inv * wv[i] : v[i] * inv;
+        };
+        if (a.norm_mode == 1) norm();
+        if (rotate) {
+            float y[V];
+#pragma unroll
+            for (int i = 0; i < V; ++i) y[i] = a.pairing ? v[i ^ 1] : __shfl_sync(0xffffffffu, v[i], other & 31);
+#pragma unroll
+            for (int i = 0; i < V; ++i) if (j0 + i < a.rd) v[i] = v[i] * cs[i] + y[i] * sn[i];
+        }
+        if (a.norm_mode == 2) norm();
+        const float hs = is_q ? (a.head_scale ? a.head_scale[hh] * ps : ps) : 1.0f;
+#pragma unroll
+        for (int i = 0; i < V; ++i) v[i] *= hs;
+        nr_store<V>(dst + j0, v);
+    }
+}
+
 template <typename T>
 static void norm_rope_launch(const NormRopeArgs& a, dim3 grid, int threads, cudaStream_t stream) {
     if (a.d <= 64) ce_launch(norm_rope_kvwrite_kernel<T, 2>, grid, threads, 0, stream, a);
@@ -200,6 +305,23 @@ extern "C" int ce_norm_rope_kvwrite(const float* proj, void* q_out, void* k_pool
     int per_block = threads / 32, want = (heads + per_block - 1) / per_block, room = 4 * 148 / T;
     int split = want < room ? want : room;
     dim3 grid(T, split < 1 ? 1 : split);
+    const int V = d / 32;
+    const bool vec = (d == 64 || d == 128 || d == 256) && dv == d && ld % 4 == 0 && off_q % 4 == 0 && off_k % 4 == 0 && off_v % 4 == 0 &&
+                     (rd == 0 || pairing == 1 || (rd / 2) % V == 0) && (dtype == CE_F32 || dtype == CE_BF16) &&
+                     ((((uintptr_t)proj | (uintptr_t)q_out | (uintptr_t)k_pool | (uintptr_t)v_pool | (uintptr_t)wq | (uintptr_t)wk) & 15) == 0);
+    if (vec) {
+        heads = nh + 2 * nkv;
+        want = (heads + per_block - 1) / per_block;
+        split = want < room ? want : room;
+        grid.y = split < 1 ? 1 : split;
+        ce_note("norm_rope_kvwrite_vec_kernel");
+#define NR_CASE(VV)                                                                                               \
+        if (dtype == CE_F32) ce_launch(norm_rope_kvwrite_vec_kernel<float, VV>, grid, threads, 0, stream, a);      \
+        else ce_launch(norm_rope_kvwrite_vec_kernel<__nv_bfloat16, VV>, grid, threads, 0, stream, a);
+        if (V == 2) { NR_CASE(2) } else if (V == 4) { NR_CASE(4) } else { NR_CASE(8) }
+#undef NR_CASE
+        return ce_check_launch("ce_norm_rope_kvwrite");
+    }
     ce_note("norm_rope_kvwrite_kernel");
     if (dtype == CE_F32) norm_rope_launch<float>(a, grid, threads, stream);
     else if (dtype == CE_BF16) norm_rope_launch<__nv_bfloat16>(a, grid, threads, stream);

@@ -124,7 +124,9 @@ def _paged(n, page, table_pages):
 
 @pytest.mark.parametrize("norm, weighted", [("before", True), ("after", False), ("after", True), ("none", False)])
 @pytest.mark.parametrize("H, G, d, rd, pairing", [(4, 2, 16, 6, "interleaved"), (3, 1, 20, 20, "half"), (9, 3, 136, 70, "interleaved"),
-                                                  (2, 2, 300, 34, "half"), (2, 1, 64, 0, "half")])
+                                                  (2, 2, 300, 34, "half"), (2, 1, 64, 0, "half"), (4, 2, 64, 28, "half"), (3, 1, 64, 30, "half"),
+                                                  (2, 2, 64, 22, "interleaved"), (5, 1, 128, 128, "half"), (2, 2, 128, 72, "interleaved"),
+                                                  (3, 3, 256, 96, "half"), (2, 1, 256, 90, "interleaved")])
 def test_attention_operands(H, G, d, rd, pairing, norm, weighted):
     """Norm before and behind the rotation in both pairings, a factor per head and one per position, tied values."""
     from carbon_engine_b200 import ops
